@@ -60,6 +60,8 @@ class StepContext:
     max_ctx_len: int = 0
     logits_out: Optional[torch.Tensor] = None   # where the head writes, if preallocated
     plans: Dict = field(default_factory=dict)    # launch plans that parts share within the step
+    # activations of the step's tokens that a layer's part leaves for parts of later layers (name -> tensor)
+    carried: Dict[str, torch.Tensor] = field(default_factory=dict)
     # True while a step of a fixed shape is recorded into a graph that later steps of other makeups
     # replay: launch plans must then hold for every batch of num_tokens tokens in num_seqs requests
     # (the host lists above describe no particular batch)

@@ -130,19 +130,15 @@ class Model:
                 self.stream_steps.add(residual, e.add_step)     # (sums commute: the pending delta is added by the next norm)
             if not getattr(block, "takes_pending", False):
                 delta = resolve(delta)      # (a block may hand its last product on unrun)
-            if scale != 1.0 and delta is not None:
-                if hasattr(block, "delta_scale"):
-                    delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache, delta_scale=scale)
-                else:
-                    raise ValueError("a block that scales its output is followed by one that cannot take the factor")
+            if hasattr(block, "delta_scale"):
+                delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache, delta_scale=scale)
+            elif scale != 1.0 and delta is not None:
+                raise ValueError("a block that scales its output is followed by one that cannot take the factor")
             else:
                 delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache)
             scale = getattr(block, "delta_scale", 1.0)
-        if isinstance(delta, NormedDelta) and getattr(self.final_norm, "fuses_products", False) and scale == 1.0:
-            y = self.final_norm.add_norm(residual, delta, "norm.final", step.logits_rows, step.num_logits_rows)
-        elif scale != 1.0:
-            y = self.final_norm.add_norm(residual, resolve(delta), "norm.final", step.logits_rows,
-                                         step.num_logits_rows, delta_scale=scale)
-        else:
-            y = self.final_norm.add_norm(residual, resolve(delta), "norm.final", step.logits_rows, step.num_logits_rows)
+        if not (isinstance(delta, NormedDelta) and getattr(self.final_norm, "fuses_products", False)):
+            delta = resolve(delta)
+        kw = {"delta_scale": scale} if scale != 1.0 else {}
+        y = self.final_norm.add_norm(residual, delta, "norm.final", step.logits_rows, step.num_logits_rows, **kw)
         return self.lm_head.forward(y, step.logits_out)

@@ -60,7 +60,17 @@ _SIGNATURES = {
     "atom_embedding": [_vp, _vp, _i, _vp, _i, _i, _i, _f, _vp],
     "atom_pair_embedding": [_vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i64, _i64, _f, _i, _vp],
     "atom_add_row": [_vp, _vp, _i, _i, _i, _vp],
-    "atom_normed_add_rmsnorm": [_vp, _i, _vp, _vp, _vp, _f, _vp, _i, _f, _vp, _i, _i, _vp],
+    "atom_normed_add_rmsnorm": [_vp, _i, _vp, _vp, _vp, _f, _vp, _i, _f, _vp, _i, _i, _f, _vp],
+    "atom_add_layernorm": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _f, _f, _vp, _vp, _i, _f, _vp, _i, _i, _vp],
+    "atom_layernorm": [_vp, _vp, _i, _vp, _vp, _vp, _i, _f, _i, _i, _vp],
+    "atom_clamped_mul": [_vp, _vp, _i, _i, _i, _f, _vp],
+    "atom_scale_softcap": [_vp, _i64, _f, _f, _vp],
+    "atom_ssm_supports": [_i, _i],
+    "atom_ssm_conv_updates_state": [_i],
+    "atom_ssm_conv": [_vp, _vp, _i, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "atom_ssm_step": [_vp, _vp, _vp, _i, _i64, _vp, _vp, _i, _i, _i, _vp],
+    "atom_ssm_scan": [_vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "atom_ssm_gate_norm": [_vp, _i, _i64, _vp, _vp, _i64, _vp, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "atom_head_gate": [_vp, _vp, _i, _i64, _i, _i, _i, _vp],
     "atom_gla_supports": [_i, _i],
     "atom_gla_scan": [_vp, _vp, _vp, _vp, _i, _i64, _vp, _i64, _vp, _i, _f, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
@@ -101,17 +111,18 @@ _SIGNATURES = {
     "atom_gemm_bf16_batched": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i64, _i64, _i64, _i64, _i64, _vp, _sz, _vp],
     "atom_relu2": [_vp, _i, _i64, _vp],
     "atom_conv_rope_write": [_vp, _vp, _i, _i64, _i, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i,
-                             _i, _vp, _vp, _i64, _vp, _vp],
+                             _i, _vp, _vp, _i64, _vp, _vp, _i, _i, _f, _vp, _f, _vp, _vp],
     "atom_conv_state_update": [_vp, _vp, _i, _i64, _i, _i, _vp, _vp, _i, _vp],
-    "atom_window_attention_merge": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _vp],
-    "atom_window_attention": [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _i, _vp],
+    "atom_window_attention_merge": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i64, _f, _i64, _vp],
+    "atom_window_attention": [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _i, _vp, _vp,
+                              _i64, _f, _i64, _vp],
     "atom_lightning_supports": [_i, _i],
     "atom_lightning_scan": [_vp, _vp, _i, _i64, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "atom_lightning_gate_norm": [_vp, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _f, _vp, _vp],
-    "atom_moe_route": [_vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
+    "atom_moe_route": [_vp, _i64, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp],
     "atom_moe_place": [_vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp],
-    "atom_moe_gemm": [_vp, _vp, _i, _i64, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "atom_moe_combine": [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _i64, _i, _i, _vp, _vp],
+    "atom_moe_gemm": [_vp, _vp, _i, _i64, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "atom_moe_combine": [_vp, _vp, _i, _vp, _vp, _i, _vp, _vp, _i64, _i, _i, _vp, _vp, _i64, _vp, _i, _vp],
     "atom_rmsnorm": [_vp, _vp, _i, _vp, _i, _f, _i, _i, _vp],
     "atom_silu_mul": [_vp, _vp, _i, _i, _i, _vp],
     "atom_qknorm_rope_kvwrite": [_vp, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _vp, _i, _i, _vp, _vp,
@@ -125,7 +136,7 @@ _SIGNATURES = {
     "atom_gemm_rows": [_vp, _i, _vp, _vp],
     "atom_gemm_rows_grid": [],
     "atom_gemm_rows_supports": [_i, _i, _i, _i64],
-    "atom_gemm_pairs": [_vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _vp, _vp],
+    "atom_gemm_pairs": [_vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _f, _vp, _vp],
     "atom_gemm_pairs_resident": [],
     "atom_gemm_pairs_supports": [_i, _i, _i, _i64, _i64],
     "atom_set_option": [_i, _i],
@@ -230,7 +241,9 @@ def _cuda(*tensors) -> None:
 
 # --------------------------------------------------------------------------- wrappers
 
-GATE_ACTS = {"silu": 1, "gelu_tanh": 2}      # the activation on the gate of a gated product (gemm_rows, gemm_pairs)
+# the activation of a gated product (gemm_rows, gemm_pairs; moe_gemm: silu and clamped): "clamped" takes a limit,
+# g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1)
+GATE_ACTS = {"silu": 1, "gelu_tanh": 2, "clamped": 3}
 
 
 def embedding(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: float = 1.0) -> None:
@@ -787,6 +800,22 @@ def gelu_mul(out: torch.Tensor, gate_up: torch.Tensor) -> None:
     _check(lib().atom_gelu_mul(out.data_ptr(), gate_up.data_ptr(), dtype_code(out.dtype), T, I, _stream()), "gelu_mul")
 
 
+def clamped_mul(out: torch.Tensor, gate_up: torch.Tensor, limit: float) -> None:
+    """out = g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit) of gate_up = [gate | up]."""
+    _cuda(out, gate_up)
+    T, I = out.shape
+    assert gate_up.shape == (T, 2 * I) and gate_up.is_contiguous() and out.is_contiguous() and out.dtype == gate_up.dtype
+    _check(lib().atom_clamped_mul(out.data_ptr(), gate_up.data_ptr(), dtype_code(out.dtype), T, I, float(limit),
+                                  _stream()), "clamped_mul")
+
+
+def scale_softcap_(x: torch.Tensor, scale: float, cap: float) -> None:
+    """x = cap * tanh(x * scale / cap) in place (cap 0: x * scale); float32."""
+    _cuda(x)
+    assert x.is_contiguous() and x.dtype == torch.float32
+    _check(lib().atom_scale_softcap(x.data_ptr(), x.numel(), float(scale), float(cap), _stream()), "scale_softcap")
+
+
 def relu2_(x: torch.Tensor) -> None:
     """x = relu(x)^2 in place."""
     _cuda(x)
@@ -798,13 +827,22 @@ def conv_rope_write(q_out: torch.Tensor, qkv: torch.Tensor, H: int, G: int, dk: 
                     conv_w: Optional[torch.Tensor], conv_state: Optional[torch.Tensor], freq: Optional[torch.Tensor],
                     rot_dims: int, positions: torch.Tensor, seq_of_token: torch.Tensor, cu_q: torch.Tensor,
                     state_slots: torch.Tensor, block_table: torch.Tensor, page_size: int,
-                    k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], status: torch.Tensor) -> None:
+                    k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], status: torch.Tensor,
+                    bias: Optional[torch.Tensor] = None, neighbours: bool = False, magnitude: float = 1.0,
+                    v_first: Optional[torch.Tensor] = None, v_mix: float = 0.0,
+                    v_keep: Optional[torch.Tensor] = None) -> None:
     """Per token of the packed projection [q (H dk) | k (G dk) | v (G dv)]: the short causal convolution over time on
     every channel (conv_w [C, taps]; rows before the step from conv_state [slots, taps - 1, C], which is only read),
     rotation of the first rot_dims numbers of every query and key head by position * freq, queries to q_out
-    [T, H dk], keys and values to their pages (csrc/window_attention.cu).  conv_w None: no convolution."""
+    [T, H dk], keys and values to their pages (csrc/window_attention.cu).  conv_w None: no convolution.  bias [C] is
+    added to the projected channels (only without a convolution); neighbours: rotated pairs are (2i, 2i + 1) instead of
+    (i, i + rot_dims / 2); magnitude: factor on cos and sin; v_first [T, G dv] dense: values become
+    (1 - v_mix) v + v_mix v_first; v_keep [T, G dv] takes a copy of the values."""
     _cuda(q_out, qkv, conv_w, conv_state, freq, positions, seq_of_token, cu_q, state_slots, block_table, k_pages,
-          v_pages, status)
+          v_pages, status, bias, v_first, v_keep)
+    assert bias is None or (conv_w is None and bias.numel() >= (H + G) * dk + G * dv and bias.is_contiguous())
+    for vt in (v_first, v_keep):
+        assert vt is None or (vt.is_contiguous() and vt.dtype == qkv.dtype and vt.shape == (qkv.shape[0], G * dv))
     T = qkv.shape[0]
     C = (H + G) * dk + G * dv
     taps = 0 if conv_w is None else conv_w.shape[1]
@@ -822,7 +860,9 @@ def conv_rope_write(q_out: torch.Tensor, qkv: torch.Tensor, H: int, G: int, dk: 
         dtype_code(conv_w.dtype) if conv_w is not None else F32, taps, _ptr(conv_state) if taps > 1 else None,
         _ptr(freq), rot_dims, positions.data_ptr(), seq_of_token.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(),
         block_table.data_ptr(), block_table.shape[1], page_size, _ptr(k_pages), _ptr(v_pages),
-        k_pages.shape[0] if k_pages is not None else 0, status.data_ptr(), _stream()), "conv_rope_write")
+        k_pages.shape[0] if k_pages is not None else 0, status.data_ptr(), _ptr(bias),
+        dtype_code(bias.dtype) if bias is not None else F32, int(neighbours), float(magnitude), _ptr(v_first),
+        float(v_mix), _ptr(v_keep), _stream()), "conv_rope_write")
 
 
 def conv_state_update(conv_state: torch.Tensor, qkv: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
@@ -838,28 +878,38 @@ def conv_state_update(conv_state: torch.Tensor, qkv: torch.Tensor, cu_q: torch.T
 
 def window_attention(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                      block_table: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor, nh: int, nkv: int,
-                     dk: int, dv: int, scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0) -> None:
+                     dk: int, dv: int, scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0,
+                     sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                     out_scale: float = 1.0) -> None:
     """Causal paged attention, key j seen from position p if j <= p and (p - j < window or j < keep_first); scores
-    scale * q.k, then softcap * tanh(score / softcap) if softcap > 0.  q [T, nh dk], out [T, nh dv], any sizes, both
-    precisions (csrc/window_attention.cu)."""
-    _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token)
+    scale * q.k, then softcap * tanh(score / softcap) if softcap > 0.  q [T, nh dk], out [T, nh dv] (rows may lie further
+    apart), any sizes, both precisions (csrc/window_attention.cu).  sink [nh] float32: exp(sink_h) is added to the
+    denominator; gate [T, nh] (a view, activation type): the output times sigmoid(gate); out_scale: times a constant."""
+    _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token, sink, gate)
+    _attention_extras(sink, gate, nh, q)
     T = q.shape[0]
     page_size = k_pages.shape[2]
-    assert q.is_contiguous() and out.is_contiguous() and q.shape == (T, nh * dk) and out.shape == (T, nh * dv)
+    assert q.is_contiguous() and out.stride(1) == 1 and q.shape == (T, nh * dk) and out.shape == (T, nh * dv)
     assert out.dtype == q.dtype == k_pages.dtype == v_pages.dtype and k_pages.is_contiguous() and v_pages.is_contiguous()
     assert tuple(k_pages.shape[1:]) == (nkv, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
     assert block_table.dtype == torch.int32 and block_table.is_contiguous()
     _check(lib().atom_window_attention(
         out.data_ptr(), q.data_ptr(), dtype_code(q.dtype), k_pages.data_ptr(), v_pages.data_ptr(),
         block_table.data_ptr(), block_table.shape[1], page_size, positions.data_ptr(), seq_of_token.data_ptr(), T, nh,
-        nkv, dk, dv, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first), _stream()),
-        "window_attention")
+        nkv, dk, dv, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first), _ptr(sink), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), _stream()), "window_attention")
+
+
+def _attention_extras(sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], nh: int, q: torch.Tensor) -> None:
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh)
+    assert gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], nh) and gate.stride(1) == 1)
 
 
 # ---- the same attention on the tensor cores (csrc/window_attention_tc.cu), compiled per (key size, value size) on
 # first use
 _watc_libs = {}
-_WATC_SIG = [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _i, _vp]
+_WATC_SIG = [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _i, _vp,
+             _vp, _i64, _f, _i64, _vp]
 WINDOW_TC = True     # False: the plain kernel also where the tensor-core kernel takes the sizes (measurements, tests)
 WINDOW_TC_ROWS = 64  # query rows of a tile
 
@@ -893,16 +943,19 @@ def window_attention_tc(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tenso
                         block_table: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
                         cu_q: torch.Tensor, num_seqs: int, nh: int, nkv: int, dk: int, dv: int, scale: float,
                         softcap: float = 0.0, window: int = 0, keep_first: int = 0, nsplit: int = 1,
-                        scratch: Optional[torch.Tensor] = None, heads_rows: bool = False) -> None:
+                        scratch: Optional[torch.Tensor] = None, heads_rows: bool = False,
+                        sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                        out_scale: float = 1.0) -> None:
     """``window_attention`` on the tensor cores: tiles of 64 consecutive tokens of a request and one head (cu_q:
     [num_seqs + 1] first token row of every request); with nsplit > 1 a tile's keys are shared out among nsplit
     CTAs and put together by a merge kernel.  heads_rows (only for steps in which every request brings ONE token, and
     at most 64 query heads to a key head): a CTA's rows are the query heads of one key head for one token, so the
     keys and values are read once per key head.  Sizes as ``window_attention_tc_supports``."""
-    _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token, cu_q, scratch)
+    _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token, cu_q, scratch, sink, gate)
+    _attention_extras(sink, gate, nh, q)
     T = q.shape[0]
     page_size = k_pages.shape[2]
-    assert q.stride(1) == 1 and q.shape[1] == nh * dk and out.is_contiguous() and out.shape == (T, nh * dv)
+    assert q.stride(1) == 1 and q.shape[1] == nh * dk and out.stride(1) == 1 and out.shape == (T, nh * dv)
     assert out.dtype == q.dtype == k_pages.dtype == v_pages.dtype == torch.bfloat16
     assert tuple(k_pages.shape[1:]) == (nkv, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
     assert k_pages.is_contiguous() and v_pages.is_contiguous() and cu_q.numel() >= num_seqs + 1
@@ -915,11 +968,13 @@ def window_attention_tc(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tenso
         out.data_ptr(), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0],
         block_table.data_ptr(), block_table.shape[1], page_size, positions.data_ptr(), seq_of_token.data_ptr(),
         cu_q.data_ptr(), num_seqs, units, nh, nkv, float(scale), float(softcap or 0.0), int(window or 0),
-        int(keep_first), int(nsplit), _ptr(scratch) if nsplit > 1 else None, int(heads_rows), _stream()),
-        "window_attention_tc")
+        int(keep_first), int(nsplit), _ptr(scratch) if nsplit > 1 else None, int(heads_rows), _ptr(sink), _ptr(gate),
+        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), _stream()), "window_attention_tc")
     if nsplit > 1:
         _check(lib().atom_window_attention_merge(out.data_ptr(), dtype_code(out.dtype), scratch.data_ptr(),
-                                                 seq_of_token.data_ptr(), T, nh, dv, nsplit, _stream()),
+                                                 seq_of_token.data_ptr(), T, nh, dv, nsplit, _ptr(sink), _ptr(gate),
+                                                 gate.stride(0) if gate is not None else 0, float(out_scale),
+                                                 out.stride(0), _stream()),
                "window_attention_merge")
 
 
@@ -976,23 +1031,31 @@ def lightning_gate_norm(y: torch.Tensor, o: torch.Tensor, g: torch.Tensor, w: to
 
 
 def moe_route(logits: torch.Tensor, E: int, top: int, score: str, renormalize: bool, seq_of_token: torch.Tensor,
-              ids: torch.Tensor, wts: torch.Tensor, counts: torch.Tensor) -> None:
+              ids: torch.Tensor, wts: torch.Tensor, counts: torch.Tensor, identity: int = 0, sum_eps: float = 0.0,
+              factor: float = 1.0, correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1) -> None:
     """Per row: the ``top`` experts with the largest scores (sigmoid or softmax of logits[:, :E], float32), their
-    scores as weights (divided by their sum if renormalize), and the experts' row counts added to ``counts``."""
-    _cuda(logits, seq_of_token, ids, wts, counts)
+    scores as weights (divided by their sum + sum_eps if renormalize; times ``factor``), and the experts' row counts
+    added to ``counts``.  The last ``identity`` of the E outputs are identity experts (no row counts); ``correction`` [E]
+    is added to the scores for the choice only; of ``groups`` groups of neighbours only the ``keep`` groups with the
+    largest choice score in them can be chosen from."""
+    _cuda(logits, seq_of_token, ids, wts, counts, correction)
     T = logits.shape[0]
     assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= E
     assert ids.dtype == counts.dtype == torch.int32 and wts.dtype == torch.float32 and ids.is_contiguous()
     assert wts.is_contiguous() and ids.shape == wts.shape == (T, top) and counts.numel() >= E
-    _check(lib().atom_moe_route(logits.data_ptr(), logits.stride(0), T, E, top, int(score == "softmax"),
-                                int(renormalize), seq_of_token.data_ptr(), ids.data_ptr(), wts.data_ptr(),
-                                counts.data_ptr(), _stream()), "moe_route")
+    assert correction is None or (correction.numel() == E and correction.is_contiguous())
+    _check(lib().atom_moe_route(logits.data_ptr(), logits.stride(0), T, E, int(identity), top, int(score == "softmax"),
+                                int(renormalize), float(sum_eps), float(factor), _ptr(correction),
+                                dtype_code(correction.dtype) if correction is not None else F32, int(groups), int(keep),
+                                seq_of_token.data_ptr(), ids.data_ptr(), wts.data_ptr(), counts.data_ptr(), _stream()),
+           "moe_route")
 
 
 def moe_place(ids: torch.Tensor, wts: torch.Tensor, E: int, counts: torch.Tensor, offsets: torch.Tensor,
               row_token: torch.Tensor, row_w: torch.Tensor, pair_pos: torch.Tensor) -> None:
     """Sorts the (row, choice) pairs by expert: offsets [E + 1] (first place of every expert), for every place the
-    row it came from and its weight, for every pair its place.  ``counts`` goes back to zero."""
+    row it came from and its weight, for every pair its place (-1: a pair without a row, as those of identity experts,
+    whose numbers lie from E on).  ``counts`` goes back to zero."""
     _cuda(ids, wts, counts, offsets, row_token, row_w, pair_pos)
     pairs, top = ids.numel(), ids.shape[1]
     assert offsets.numel() >= E + 1 and row_token.numel() >= pairs and row_w.numel() >= pairs and pair_pos.numel() >= pairs
@@ -1005,10 +1068,11 @@ MOE_TC = True        # False: the plain product also in bfloat16 (measurements, 
 
 
 def moe_gemm(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, offsets: torch.Tensor, gated: bool = False,
-             row_token: Optional[torch.Tensor] = None, row_w: Optional[torch.Tensor] = None) -> None:
-    """out[r] = A[r] w[e]^T for the places r of every expert e (offsets [E + 1]); w [E, N or 2 N, K].  With row_token
-    and row_w, A[r] = row_w[r] * a[row_token[r]] (rows picked from the step's rows, weighted on the way in); else
-    A = a by place.  gated: w[e] = [gate ; up], out = silu(gate) * up.  bfloat16 with K and the row stride in steps
+             row_token: Optional[torch.Tensor] = None, row_w: Optional[torch.Tensor] = None, act: str = "silu",
+             limit: float = 0.0) -> None:
+    """out[r] = A[r] w[e]^T for the places r of every expert e (offsets [E + 1]); w [E, N or 2 N, K].  With row_token,
+    A[r] = a[row_token[r]] (rows picked from the step's rows), with row_w weighted on the way in by row_w[r]; else
+    A = a by place.  gated: w[e] = [gate ; up], out = silu(gate) * up or the clamped form (GATE_ACTS).  bfloat16 with K and the row stride in steps
     of 8 runs on the tensor cores, everything else on plain FMAs."""
     _cuda(out, a, w, offsets, row_token, row_w)
     R, N = out.shape
@@ -1016,15 +1080,20 @@ def moe_gemm(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, offsets: torch
     assert w.shape[1] == (2 * N if gated else N) and w.is_contiguous() and out.is_contiguous() and a.stride(1) == 1
     assert a.shape[1] == K and out.dtype == a.dtype == w.dtype and (row_token is not None or a.shape[0] >= R)
     _check(lib().atom_moe_gemm(out.data_ptr(), a.data_ptr(), dtype_code(a.dtype), a.stride(0), w.data_ptr(),
-                               offsets.data_ptr(), _ptr(row_token), _ptr(row_w), R, E, N, K, int(gated),
-                               int(row_token is not None), int(MOE_TC), _stream()), "moe_gemm")
+                               offsets.data_ptr(), _ptr(row_token), _ptr(row_w), R, E, N, K,
+                               GATE_ACTS[act] if gated else 0, int(row_token is not None), int(MOE_TC), float(limit),
+                               _stream()), "moe_gemm")
 
 
 def moe_combine(out: torch.Tensor, y: torch.Tensor, pair_pos: torch.Tensor, top: int,
                 pair_w: Optional[torch.Tensor], shared: Optional[torch.Tensor], gate: Optional[torch.Tensor],
-                seq_of_token: torch.Tensor) -> None:
+                seq_of_token: torch.Tensor, x: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                identity_from: int = 0) -> None:
     """out[t] = sum over t's choices k of (pair_w[t, k] *) y[pair_pos[t, k]] (+ sigmoid(gate[t]) * shared[t]);
-    gate: a float32 column view (one logit per row) or None (the shared part is added as it is)."""
+    gate: a float32 column view (one logit per row) or None (the shared part is added as it is).  With x [T, n] and ids
+    [T, top]: + x[t] times the weights of those choices whose expert number is at least identity_from."""
+    assert x is None or (ids is not None and ids.dtype == torch.int32 and ids.is_contiguous() and x.dtype == out.dtype
+                         and x.stride(1) == 1 and x.shape == out.shape)
     _cuda(out, y, pair_pos, pair_w, shared, gate, seq_of_token)
     T, n = out.shape
     assert out.is_contiguous() and y.is_contiguous() and y.shape[1] == n and out.dtype == y.dtype
@@ -1032,7 +1101,8 @@ def moe_combine(out: torch.Tensor, y: torch.Tensor, pair_pos: torch.Tensor, top:
     assert gate is None or (gate.dtype == torch.float32 and gate.shape[0] == T)
     _check(lib().atom_moe_combine(out.data_ptr(), y.data_ptr(), dtype_code(out.dtype), pair_pos.data_ptr(),
                                   _ptr(pair_w), top, _ptr(shared), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                  T, n, seq_of_token.data_ptr(), _stream()), "moe_combine")
+                                  T, n, seq_of_token.data_ptr(), _ptr(x), x.stride(0) if x is not None else 0, _ptr(ids),
+                                  int(identity_from), _stream()), "moe_combine")
 
 
 _device_flags = {}
@@ -1085,7 +1155,7 @@ class _RowsOpC(ctypes.Structure):
                 ("bias", _vp), ("bias_dtype", _i), ("N", _i), ("K", _i), ("gated", _i),
                 ("ssq_in", _vp), ("ssq_parts", _i), ("norm_size", _i), ("norm_eps", _f),
                 ("residual", _vp), ("norm_w", _vp), ("norm_w_dtype", _i), ("xout", _vp), ("ssq_out", _vp),
-                ("res_scale", _f)]
+                ("res_scale", _f), ("limit", _f)]
 
 
 ROWS_M = 16     # rows up to which the weight-streaming product is used (parts/linear.py: streams)
@@ -1104,10 +1174,11 @@ def gemm_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
               bias: Optional[torch.Tensor] = None, gated: bool = False, ssq_in: Optional[torch.Tensor] = None,
               norm_size: int = 0, norm_eps: float = 0.0, residual: Optional[torch.Tensor] = None,
               norm_w: Optional[torch.Tensor] = None, xout: Optional[torch.Tensor] = None,
-              ssq_out: Optional[torch.Tensor] = None, act: str = "silu", res_scale: float = 1.0) -> None:
+              ssq_out: Optional[torch.Tensor] = None, act: str = "silu", res_scale: float = 1.0,
+              limit: float = 0.0) -> None:
     """out[M, N] = x[M, K] w[N, K]^T for at most 16 rows of bf16 x, with one of the epilogues of
-    csrc/gemm_rows.h: plain (+ bias; out bf16 or float32); ``gated`` (w = [gate ; up] of 2N rows, ``act`` "silu" or
-    "gelu_tanh" on the gate);
+    csrc/gemm_rows.h: plain (+ bias; out bf16 or float32); ``gated`` (w = [gate ; up] of 2N rows, ``act`` of
+    GATE_ACTS, ``limit`` of its clamped form);
     ``residual`` (float32 [M, N], += ``res_scale`` * product in place, with ``xout`` = bf16(residual * norm_w) and the CTAs'
     sums of squares in ``ssq_out`` [gemm_rows_grid(), 16]).  ``ssq_in`` (such sums, of ``norm_size`` columns):
     every output row is first multiplied by its rstd."""
@@ -1139,7 +1210,7 @@ def gemm_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
     c.residual, c.norm_w = _ptr(residual), _ptr(norm_w)
     c.norm_w_dtype = dtype_code(norm_w.dtype) if norm_w is not None else F32
     c.xout, c.ssq_out = _ptr(xout), _ptr(ssq_out)
-    c.res_scale = float(res_scale)
+    c.res_scale, c.limit = float(res_scale), float(limit)
     _check(lib().atom_gemm_rows(ctypes.byref(c), M, error_flag(x.device).data_ptr(), _stream()), "gemm_rows")
 
 
@@ -1171,16 +1242,18 @@ def gemm_pairs_waves(M: int, N: int, gated: bool) -> float:
     return tiles / (waves * pairs)
 
 
-def gemm_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = False, act: str = "silu") -> None:
+def gemm_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool = False, act: str = "silu",
+               limit: float = 0.0) -> None:
     """out[M, N] = x[M, K] w[N, K]^T in bf16 on tcgen05 with two CTAs to a tile; ``gated``: w = [gate ; up]
-    of 2N rows, out = act(x gate^T) * (x up^T), ``act`` "silu" or "gelu_tanh" (csrc/gemm_pairs.cu)."""
+    of 2N rows, out = act(x gate^T) * (x up^T), ``act`` of GATE_ACTS, ``limit`` of its clamped form (csrc/gemm_pairs.cu)."""
     M, K = x.shape
     N = out.shape[1]
     _cuda(x, w, out)
     assert x.dtype == w.dtype == out.dtype == torch.bfloat16 and w.shape[1] == K and w.is_contiguous()
     assert x.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == M and w.shape[0] == (2 * N if gated else N)
     _check(lib().atom_gemm_pairs(x.data_ptr(), x.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), M, N, K,
-                                 GATE_ACTS[act] if gated else 0, error_flag(x.device).data_ptr(), _stream()), "gemm_pairs")
+                                 GATE_ACTS[act] if gated else 0, float(limit), error_flag(x.device).data_ptr(), _stream()),
+           "gemm_pairs")
 
 
 def add_bias(out: torch.Tensor, bias: torch.Tensor) -> None:
@@ -1414,8 +1487,8 @@ def add_row(residual: torch.Tensor, vec: torch.Tensor) -> None:
 
 def normed_add_rmsnorm(out: torch.Tensor, residual: torch.Tensor, delta: torch.Tensor, delta_weight: torch.Tensor,
                        delta_eps: float, weight: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None,
-                       n_rows: Optional[int] = None) -> None:
-    """residual += rmsnorm(delta; delta_weight); out = rmsnorm(residual; weight), one kernel, 32-bit.  With ``rows``
+                       n_rows: Optional[int] = None, delta_scale: float = 1.0) -> None:
+    """residual += delta_scale * rmsnorm(delta; delta_weight); out = rmsnorm(residual; weight), one kernel, 32-bit.  With ``rows``
     only those rows, written densely, and residual is left as it is."""
     _cuda(out, residual, delta, delta_weight, weight, rows)
     H = residual.shape[-1]
@@ -1425,8 +1498,42 @@ def normed_add_rmsnorm(out: torch.Tensor, residual: torch.Tensor, delta: torch.T
     n = (rows.numel() if n_rows is None else n_rows) if rows is not None else residual.shape[0]
     _check(lib().atom_normed_add_rmsnorm(out.data_ptr(), dtype_code(out.dtype), residual.data_ptr(), delta.data_ptr(),
                                          delta_weight.data_ptr(), float(delta_eps), weight.data_ptr(),
-                                         dtype_code(weight.dtype), float(eps), _ptr(rows), n, H, _stream()),
+                                         dtype_code(weight.dtype), float(eps), _ptr(rows), n, H, float(delta_scale), _stream()),
            "normed_add_rmsnorm")
+
+
+def add_layernorm(out: torch.Tensor, residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor,
+                  bias: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None,
+                  delta_scale: float = 1.0, delta_bias: Optional[torch.Tensor] = None,
+                  delta_norm: Optional[tuple] = None) -> None:
+    """residual (+= delta_scale * d); out = layernorm(residual; weight, bias), one kernel, 32-bit, with
+    d = delta (+ delta_bias), or layernorm(delta (+ delta_bias); w, b, eps) for delta_norm = (w, b, eps).  With ``rows``
+    only those rows, written densely, and residual is left as it is.  All vectors have one type."""
+    wd, bd, eps_d = delta_norm if delta_norm is not None else (None, None, 0.0)
+    _cuda(out, residual, delta, weight, bias, rows, delta_bias, wd, bd)
+    H = residual.shape[-1]
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and out.is_contiguous() and out.shape[-1] == H
+    assert delta is None or (delta.dtype == out.dtype and delta.is_contiguous() and delta.shape[-1] == H)
+    for t in (weight, bias, wd, bd, delta_bias):
+        assert t is None or (t.numel() == H and t.dtype == weight.dtype and t.is_contiguous())
+    n = (rows.numel() if n_rows is None else n_rows) if rows is not None else residual.shape[0]
+    assert out.shape[0] >= n
+    _check(lib().atom_add_layernorm(out.data_ptr(), dtype_code(out.dtype), residual.data_ptr(), _ptr(delta),
+                                    _ptr(delta_bias), _ptr(wd), _ptr(bd), float(eps_d), float(delta_scale),
+                                    weight.data_ptr(), bias.data_ptr(), dtype_code(weight.dtype), float(eps), _ptr(rows),
+                                    n, H, _stream()), "add_layernorm")
+
+
+def layernorm(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float,
+              x_bias: Optional[torch.Tensor] = None) -> None:
+    """out = layernorm(x (+ x_bias); weight, bias) of dense rows."""
+    _cuda(out, x, weight, bias, x_bias)
+    H = x.shape[-1]
+    assert x.is_contiguous() and out.is_contiguous() and out.dtype == x.dtype and weight.dtype == bias.dtype
+    assert weight.numel() == bias.numel() == H and (x_bias is None or (x_bias.dtype == weight.dtype and x_bias.numel() == H))
+    _check(lib().atom_layernorm(out.data_ptr(), x.data_ptr(), dtype_code(x.dtype), _ptr(x_bias), weight.data_ptr(),
+                                bias.data_ptr(), dtype_code(weight.dtype), float(eps), x.numel() // H, H, _stream()),
+           "layernorm")
 
 
 def head_gate(x: torch.Tensor, g: torch.Tensor) -> None:
@@ -1503,6 +1610,98 @@ def gla_gate_norm(y: torch.Tensor, o: torch.Tensor, g: torch.Tensor, w: torch.Te
     _check(lib().atom_gla_gate_norm(y.data_ptr(), o.data_ptr(), g.data_ptr(), dtype_code(y.dtype), g.stride(0),
                                     w.data_ptr(), dtype_code(w.dtype), T, H, dv, float(eps), seq_of_token.data_ptr(),
                                     _stream()), "gla_gate_norm")
+
+
+# ------------------------------------------------------------------ state-space duality (Mamba-2)
+
+def ssm_supports(N: int, P: int) -> bool:
+    return bool(lib().atom_ssm_supports(N, P))
+
+
+SSM_RUN = 64        # rows per run of the scan in steps of more rows than this
+
+
+def ssm_run(T: int) -> int:
+    """Rows per run for a step of T rows (0: every request is walked once)."""
+    if T <= SSM_RUN:
+        return 0
+    return SSM_RUN if T <= 64 * SSM_RUN else -(-T // 64)
+
+
+def ssm_scratch_elems(T: int, num_seqs: int, H: int, N: int, P: int):
+    """(floats of the runs' sums, floats of the runs' decays)."""
+    run = ssm_run(T)
+    if run == 0:
+        return 0, 0
+    slots = -(-T // run) + num_seqs
+    return slots * H * N * P, slots * H
+
+
+def ssm_conv(u: torch.Tensor, xbc: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: Optional[torch.Tensor],
+             seq_of_token: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, num_seqs: int,
+             write_state: bool = True) -> None:
+    """u [T, C] = silu(causal convolution of xbc's C channels with w [C, taps], + b) within each request; rows before the
+    step come from state [slots, taps - 1, C] (None for one tap), which takes the request's last taps - 1 rows."""
+    _cuda(u, xbc, w, b, state, seq_of_token, cu_q, state_slots)
+    T, C = u.shape
+    taps = w.shape[1]
+    assert xbc.shape == (T, C) and xbc.stride(1) == 1 and u.is_contiguous() and u.dtype == xbc.dtype
+    assert w.shape == (C, taps) and w.is_contiguous() and b.numel() == C and b.dtype == w.dtype
+    assert taps == 1 or (state.is_contiguous() and state.dtype == u.dtype and tuple(state.shape[1:]) == (taps - 1, C))
+    _check(lib().atom_ssm_conv(u.data_ptr(), xbc.data_ptr(), dtype_code(u.dtype), xbc.stride(0), w.data_ptr(), b.data_ptr(),
+                               dtype_code(w.dtype), _ptr(state) if taps > 1 else None, taps, seq_of_token.data_ptr(),
+                               cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, C, int(write_state), _stream()),
+           "ssm_conv")
+    if taps > 1 and write_state and not lib().atom_ssm_conv_updates_state(taps):
+        conv_state_update(state, xbc, cu_q, state_slots, num_seqs)
+
+
+def ssm_step(dt: torch.Tensor, la: torch.Tensor, raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor) -> None:
+    """dt = softplus(raw + dt_bias), la = -exp(a_log) * dt; dt, la float32 [T, H], raw a view of the projection."""
+    _cuda(dt, la, raw, dt_bias, a_log)
+    T, H = dt.shape
+    assert dt.dtype == la.dtype == torch.float32 and dt.is_contiguous() and la.is_contiguous() and la.shape == (T, H)
+    assert raw.shape == (T, H) and raw.stride(1) == 1 and dt_bias.numel() == a_log.numel() == H
+    assert dt_bias.dtype == a_log.dtype
+    _check(lib().atom_ssm_step(dt.data_ptr(), la.data_ptr(), raw.data_ptr(), dtype_code(raw.dtype), raw.stride(0),
+                               dt_bias.data_ptr(), a_log.data_ptr(), dtype_code(a_log.dtype), T, H, _stream()), "ssm_step")
+
+
+def ssm_scan(out: torch.Tensor, u: torch.Tensor, dt: torch.Tensor, la: torch.Tensor, D: torch.Tensor, state: torch.Tensor,
+             scratch_b: Optional[torch.Tensor], scratch_a: Optional[torch.Tensor], cu_q: torch.Tensor,
+             state_slots: torch.Tensor, num_seqs: int, H: int, G: int, N: int, P: int, write_state: bool = True) -> None:
+    """out[t] (float32 [T, H P]) = S_t^T C_t + D x_t with S_t = exp(la_t) S_(t-1) + dt_t B_t x_t^T per head, over every
+    request's rows; u rows are [x (H P) | B (G N) | C (G N)]; state [slots, H, N, P] float32."""
+    _cuda(out, u, dt, la, D, state, scratch_b, scratch_a, cu_q, state_slots)
+    T = u.shape[0]
+    run = ssm_run(T)
+    assert out.dtype == torch.float32 and out.is_contiguous() and out.shape == (T, H * P)
+    assert u.is_contiguous() and u.shape == (T, H * P + 2 * G * N) and D.numel() == H
+    assert dt.shape == la.shape == (T, H) and dt.is_contiguous() and la.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, P)
+    if run:
+        nb, na = ssm_scratch_elems(T, num_seqs, H, N, P)
+        assert scratch_b is not None and scratch_a is not None and scratch_b.dtype == scratch_a.dtype == torch.float32
+        assert scratch_b.numel() >= nb and scratch_a.numel() >= na
+    _check(lib().atom_ssm_scan(out.data_ptr(), u.data_ptr(), dtype_code(u.dtype), dt.data_ptr(), la.data_ptr(), D.data_ptr(),
+                               dtype_code(D.dtype), state.data_ptr(), _ptr(scratch_b) if run else None,
+                               _ptr(scratch_a) if run else None, cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, H,
+                               G, N, P, run, int(write_state), _stream()), "ssm_scan")
+    if run:
+        add_launches(2)      # (the runs' sums, the prefix over the runs, the outputs)
+
+
+def ssm_gate_norm(out: torch.Tensor, y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, parts: int, eps: float,
+                  out_scale: float, seq_of_token: torch.Tensor) -> None:
+    """out = (y * silu(z)) / rms over each of ``parts`` equal parts of a row * w * out_scale; y float32 [T, n] dense, z and
+    out views whose rows may lie further apart."""
+    _cuda(out, y, z, w, seq_of_token)
+    T, n = y.shape
+    assert y.dtype == torch.float32 and y.is_contiguous() and z.shape == out.shape == (T, n) and z.dtype == out.dtype
+    assert z.stride(1) == out.stride(1) == 1 and w.numel() == n and n % parts == 0
+    _check(lib().atom_ssm_gate_norm(out.data_ptr(), dtype_code(out.dtype), out.stride(0), y.data_ptr(), z.data_ptr(),
+                                    z.stride(0), w.data_ptr(), dtype_code(w.dtype), T, n, parts, float(eps),
+                                    float(out_scale), seq_of_token.data_ptr(), _stream()), "ssm_gate_norm")
 
 
 # ------------------------------------------------------------------ attention over a window and pooled blocks

@@ -211,3 +211,83 @@ ATOM_EXPORT int atom_head_gate(void* x, const void* g, int dtype, int64_t ldg, i
     return ATOM_ERR_ARG;
   return atom::check_launch();
 }
+
+// The clamped gated product: out = clamped_gate(gu[:, :I], gu[:, I:], limit) (gate_act.cuh), in 32-bit.
+#include "gate_act.cuh"
+namespace atom {
+template <typename T>
+__global__ void clamped_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, int64_t n, int I, float limit) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = idx / I;
+    const int i = (int)(idx - t * I);
+    out[idx] = from_float<T>(clamped_gate(to_float(gu[t * 2 * I + i]), to_float(gu[t * 2 * I + I + i]), limit));
+  }
+}
+
+// bf16, I a multiple of 8: 16 bytes of gate and of up per thread.
+__global__ void clamped_mul_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gu,
+                                            int64_t nvec, int I8, float limit) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < nvec; idx += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = idx / I8;
+    const int i = (int)(idx - t * I8);
+    const uint4 g4 = *reinterpret_cast<const uint4*>(gu + (t * 2 * I8 + i) * 8);
+    const uint4 u4 = *reinterpret_cast<const uint4*>(gu + (t * 2 * I8 + I8 + i) * 8);
+    const __nv_bfloat162* gh = reinterpret_cast<const __nv_bfloat162*>(&g4);
+    const __nv_bfloat162* uh = reinterpret_cast<const __nv_bfloat162*>(&u4);
+    uint4 o4;
+    __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 g = __bfloat1622float2(gh[e]), u = __bfloat1622float2(uh[e]);
+      oh[e] = __floats2bfloat162_rn(clamped_gate(g.x, u.x, limit), clamped_gate(g.y, u.y, limit));
+    }
+    *reinterpret_cast<uint4*>(out + idx * 8) = o4;
+  }
+}
+
+// x = cap * tanh(x * scale / cap) (cap <= 0: x * scale), in place on 32-bit numbers.
+__global__ void scale_softcap_kernel(float* __restrict__ x, int64_t n, float scale, float cap) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (int64_t)gridDim.x * blockDim.x) {
+    const float y = x[i] * scale;
+    x[i] = cap > 0.f ? cap * tanhf(y / cap) : y;
+  }
+}
+}  // namespace atom
+
+ATOM_EXPORT int atom_clamped_mul(void* out, const void* gu, int dtype, int T, int I, float limit, cudaStream_t stream) {
+  if (T <= 0) return ATOM_OK;
+  if (I <= 0) return ATOM_ERR_ARG;
+  const int64_t n = (int64_t)T * I;
+  if (dtype == ATOM_BF16 && I % 8 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)gu % 16 == 0) {
+    int64_t vb = (n / 8 + 255) / 256;
+    if (vb > 148 * 32) vb = 148 * 32;
+    atom::launch_pdl(atom::clamped_mul_bf16_vec_kernel, dim3((int)vb), dim3(256), 0, stream, (__nv_bfloat16*)out,
+                     (const __nv_bfloat16*)gu, n / 8, I / 8, limit);
+    return atom::check_launch();
+  }
+  int64_t blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  if (dtype == ATOM_F32)
+    atom::launch_pdl(atom::clamped_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, (float*)out,
+                     (const float*)gu, n, I, limit);
+  else if (dtype == ATOM_BF16)
+    atom::launch_pdl(atom::clamped_mul_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, stream,
+                     (__nv_bfloat16*)out, (const __nv_bfloat16*)gu, n, I, limit);
+  else
+    return ATOM_ERR_ARG;
+  return atom::check_launch();
+}
+
+ATOM_EXPORT int atom_scale_softcap(float* x, int64_t n, float scale, float cap, cudaStream_t stream) {
+  if (n <= 0) return ATOM_OK;
+  int64_t blocks = (n + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  atom::launch_pdl(atom::scale_softcap_kernel, dim3((int)blocks), dim3(256), 0, stream, x, n, scale, cap);
+  return atom::check_launch();
+}

@@ -1,7 +1,8 @@
 // Matrix product for many rows on the 5th-generation tensor cores, two CTAs to a tile (tcgen05 with
 // cta_group::2), bf16 in, 32-bit sums in tensor memory, bf16 out:
 //     plain:   C[M, N] = X[M, K] W[N, K]^T
-//     gated:   W = [gate ; up] of N rows each, C[M, N] = act(X gate^T) * (X up^T), act = silu or gelu_tanh
+//     gated:   W = [gate ; up] of N rows each, C[M, N] = act(X gate^T) * (X up^T), act = silu or gelu_tanh,
+//              or the clamped form of gate_act.cuh
 // It is the prefill feed-forward's first product with the activation in its epilogue: the sums never
 // leave the chip, and the activation kernel with its pass over [M, 2N] goes away.
 //
@@ -24,6 +25,7 @@
 // one tile, so the MMAs of a tile wait until the epilogue of the one before has read the sums (a gated
 // tile's outputs fit in registers as bf16, so its stores come after that); the loads do not wait.
 // All waits are bounded (tma.cuh); tensor memory is freed on every path.
+#include "gate_act.cuh"
 #include "tma.cuh"
 #include <cuda_bf16.h>
 
@@ -53,7 +55,8 @@ struct Params {
   int mt, nt;         // tiles of 256 rows, tiles of 512 columns of sums
   int full_items;     // work items [0, full_items) are whole tiles, the others halves of the tiles that follow
   int items;
-  int act;            // gated: 1 silu, 2 gelu_tanh
+  int act;            // gated: 1 silu, 2 gelu_tanh, 3 the clamped form
+  float limit;        // of the clamped form
   int* error;
 };
 
@@ -178,6 +181,15 @@ __device__ __forceinline__ float silu(float x) {
 __device__ __forceinline__ float gelu_tanh(float z) {
   const float a = 0.7978845608028654f * (z + 0.044715f * z * z * z);
   return __fdividef(z, 1.f + __expf(fminf(-2.f * a, 80.f)));
+}
+
+// g sigmoid(1.702 g) (u + 1) of the clamped g and u, the sigmoid as 0.5 + 0.5 tanh(0.851 g).
+__device__ __forceinline__ float clamped(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  float t;
+  asm("tanh.approx.f32 %0, %1;\n" : "=f"(t) : "f"(0.5f * kClampedSlope * g));
+  return g * fmaf(0.5f, t, 0.5f) * (u + 1.f);
 }
 
 struct Item {
@@ -348,7 +360,8 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
             tmem_ld32(tbase + h * 256 + 128 + b * 64 + ch * 32, u);
             tmem_wait_ld();
 #pragma unroll
-            for (int j = 0; j < 32; ++j) g[j] = (p.act == 2 ? gelu_tanh(g[j]) : silu(g[j])) * u[j];
+            for (int j = 0; j < 32; ++j)
+              g[j] = p.act == 3 ? clamped(g[j], u[j], p.limit) : (p.act == 2 ? gelu_tanh(g[j]) : silu(g[j])) * u[j];
             pack(g, o[h][b]);
           }
           tc_fence_before();
@@ -445,9 +458,9 @@ static int plan_items(int tiles, int pairs, int* full_items) {
 }
 
 ATOM_EXPORT int atom_gemm_pairs(const void* X, int64_t lda, const void* W, void* out, int64_t ldc, int M, int N, int K,
-                                int gated, int* error, cudaStream_t stream) {
+                                int gated, float limit, int* error, cudaStream_t stream) {
   using namespace atom::pairs;
-  if (X == nullptr || W == nullptr || out == nullptr || error == nullptr || gated < 0 || gated > 2 ||
+  if (X == nullptr || W == nullptr || out == nullptr || error == nullptr || gated < 0 || gated > 3 ||
       !atom_gemm_pairs_supports(M, N, K, lda, ldc) ||
       ((uintptr_t)X % 16) != 0 || ((uintptr_t)W % 16) != 0 || ((uintptr_t)out % 16) != 0)
     return ATOM_ERR_ARG;
@@ -464,6 +477,7 @@ ATOM_EXPORT int atom_gemm_pairs(const void* X, int64_t lda, const void* W, void*
   p.mt = (M + 255) / 256;
   p.nt = gated ? (N + 255) / 256 : (N + 511) / 512;
   p.act = gated;
+  p.limit = limit;
   p.error = error;
   const int tiles = p.mt * p.nt;
   if (pairs > tiles) pairs = tiles;

@@ -36,6 +36,7 @@
 #include "gemm_rows.h"
 
 #include "common.cuh"
+#include "gate_act.cuh"
 #include "tma.cuh"
 
 namespace atom {
@@ -99,6 +100,7 @@ struct Params {
   __nv_bfloat16* xout;
   float* ssq_out;
   float res_scale;
+  float limit;
 };
 
 __device__ __forceinline__ int row_begin(const Params& p, int c) { return (int)((long long)p.N * c / gridDim.x); }
@@ -379,7 +381,9 @@ gemm_rows_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
           sq[nt] += rr * rr;
         } else {
           if (gated)
-            sum = (p.gated == 2 ? gelu_tanh(sum) : sum / (1.f + __expf(-sum))) * (up * scale[nt]);
+            sum = p.gated == kGateClamped ? clamped_gate(sum, up * scale[nt], p.limit)
+                                          : (p.gated == kGateGelu ? gelu_tanh(sum) : sum / (1.f + __expf(-sum))) *
+                                                (up * scale[nt]);
           else
             sum += bias;
           if (p.out_dtype == ATOM_F32)
@@ -450,7 +454,7 @@ ATOM_EXPORT int atom_gemm_rows(const AtomRowsOp* op, int M, int* error, cudaStre
   if (op == nullptr || error == nullptr) return ATOM_ERR_ARG;
   const AtomRowsOp& a = *op;
   const bool res = a.residual != nullptr;
-  if (!atom_gemm_rows_supports(M, a.N, a.K, a.lda) || a.gated < 0 || a.gated > 2 || (a.gated && a.bias != nullptr) ||
+  if (!atom_gemm_rows_supports(M, a.N, a.K, a.lda) || a.gated < 0 || a.gated > 3 || (a.gated && a.bias != nullptr) ||
       ((uintptr_t)a.X % 16) != 0 || ((uintptr_t)a.W % 16) != 0)
     return ATOM_ERR_ARG;
   if (!res && (a.out == nullptr || a.ldc < a.N || (a.out_dtype != ATOM_F32 && a.out_dtype != ATOM_BF16)))
@@ -500,5 +504,6 @@ ATOM_EXPORT int atom_gemm_rows(const AtomRowsOp* op, int M, int* error, cudaStre
   p.xout = reinterpret_cast<__nv_bfloat16*>(a.xout);
   p.ssq_out = a.ssq_out;
   p.res_scale = a.res_scale;
+  p.limit = a.limit;
   return MT == 1 ? launch<1>(mw, mx, p, grid, stream) : launch<2>(mw, mx, p, grid, stream);
 }

@@ -2,42 +2,96 @@
 //
 //   moe_route_kernel    per row (a warp): score = sigmoid(logit) or softmax over the experts, the top experts by
 //                       score (ties: the lower index), their weights (optionally divided by their sum), and the
-//                       experts' row counts
+//                       experts' row counts.  Options: a correction per expert that counts in the choice but not in
+//                       the weights; groups of neighbouring experts, of which only the `keep` groups with the largest
+//                       choice score in them can be chosen from; a factor on the weights; the last outputs of the
+//                       router as identity experts, which have no rows (moe_combine adds their weight times the input)
 //   moe_place_kernel    one CTA: the experts' first rows (a running sum of the counts) and a place for every
 //                       (row, choice) pair among its expert's rows; the counts go back to zero
 //   moe_gemm_kernel     out[r] = A[r] W_e^T for the rows r of every expert e, tile by tile.  A[r] is either a dense
 //                       row or weight_r * x[token_r] (the weight on the expert's INPUT); with GATED, W_e is
-//                       [gate ; up] and the output is silu(gate) * up.  32-bit sums, each output summed over k in
+//                       [gate ; up] and the output is silu(gate) * up, or with clamped halves
+//                       g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(1.702 g) * (u + 1).  32-bit sums, each output summed over k in
 //                       order, so a row's result does not depend on the rows beside it; in bfloat16 on the tensor
 //                       cores (moe_gemm_tc_kernel), in 32-bit and for odd sizes with plain FMAs
 //   moe_combine_kernel  out[t] = sum over t's choices of (weight *) y[place] (+ sigmoid(gate logit_t) * shared[t])
+//                       (+ the weights of t's identity choices * x[t])
 #include "common.cuh"
+#include "gate_act.cuh"
 
 namespace atom {
 
+struct MoeRouteArgs {
+  int E;                          // router outputs that can be chosen, identity experts included
+  int rows_from;                  // experts below this number have rows (the rest are identity experts)
+  int top, softmax_scores, renormalize;
+  float sum_eps, factor;          // weights: score (/ (sum + sum_eps) if renormalize) * factor
+  const void* correction;         // [E] or null
+  int correction_dtype;
+  int groups, keep;               // groups of E / groups neighbours (<= 1: none)
+};
+
 // logits [T, ld] float32.  ids, wts [T, top]; counts [E] (zero on entry).
-__global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, int E, int top, int softmax_scores,
-                                 int renormalize, const int* __restrict__ seq_of_token, int T, int* __restrict__ ids,
+__global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, const MoeRouteArgs p,
+                                 const int* __restrict__ seq_of_token, int T, int* __restrict__ ids,
                                  float* __restrict__ wts, int* __restrict__ counts) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
+  const int E = p.E, top = p.top;
   if (seq_of_token[t] < 0) {
     for (int k = lane; k < top; k += 32) ids[(int64_t)t * top + k] = -1;
     return;
   }
   const float* z = logits + (int64_t)t * ld;
   float zmax = -INFINITY, denom = 1.f;
-  if (softmax_scores) {
+  if (p.softmax_scores) {
     for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, z[e]);
     zmax = warp_max(zmax);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
     denom = warp_sum(sum);
   }
-  uint32_t taken = 0;                       // bit m: expert lane + 32 m has been chosen (E <= 1024)
+  auto score = [&](int e) { return p.softmax_scores ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e])); };
+  // what the choice goes by: the logit itself where scores grow with it and nothing is added to them
+  auto choice = [&](int e) { return p.correction ? score(e) + load_as_float(p.correction, p.correction_dtype, e) : z[e]; };
+  uint32_t taken = 0;                       // bit m: expert lane + 32 m cannot be chosen (any more) (E <= 1024)
+  if (p.groups > 1) {
+    // a group's score is its largest choice score: the best `keep` groups one after another (ties: the lower group)
+    const int size = E / p.groups;
+    uint32_t kept = 0;                      // bit m: group lane + 32 m is kept
+    for (int k = 0; k < p.keep; ++k) {
+      float best = -INFINITY;
+      int best_g = 0x7fffffff;
+      for (int g = lane, m = 0; g < p.groups; g += 32, ++m) {
+        if ((kept >> m) & 1u) continue;
+        float v = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) v = fmaxf(v, choice(e));
+        if (v > best || best_g == 0x7fffffff) {
+          best = v;
+          best_g = g;
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+        if (ob > best || (ob == best && og < best_g)) {
+          best = ob;
+          best_g = og;
+        }
+      }
+      if (best_g < p.groups && (best_g & 31) == lane) kept |= 1u << (best_g >> 5);
+    }
+    for (int e0 = 0, m = 0; e0 < E; e0 += 32, ++m) {
+      const int e = e0 + lane;
+      const int g = e < E ? e / size : 0;
+      const uint32_t owner = __shfl_sync(0xffffffffu, kept, g & 31);
+      if (e < E && !((owner >> (g >> 5)) & 1u)) taken |= 1u << m;
+    }
+  }
   float wsum = 0.f, mine = 0.f;             // lane k keeps the weight of choice k (top <= 32)
   int mine_id = -1;
   for (int k = 0; k < top; ++k) {
@@ -45,7 +99,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, i
     int best_e = 0x7fffffff;
     for (int e = lane, m = 0; e < E; e += 32, ++m) {
       if ((taken >> m) & 1u) continue;
-      const float v = z[e];
+      const float v = choice(e);
       if (v > best) {               // ascending e: the lower index wins a tie
         best = v;
         best_e = e;
@@ -60,8 +114,9 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, i
         best_e = oe;
       }
     }
+    if (best_e >= E) break;         // (nothing left to choose: the host refuses such sizes)
     if ((best_e & 31) == lane) taken |= 1u << (best_e >> 5);
-    const float w = softmax_scores ? expf(best - zmax) / denom : 1.f / (1.f + expf(-best));
+    const float w = score(best_e);
     wsum += w;
     if (lane == k) {
       mine = w;
@@ -70,12 +125,12 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, i
   }
   if (lane < top) {
     ids[(int64_t)t * top + lane] = mine_id;
-    wts[(int64_t)t * top + lane] = renormalize ? mine / wsum : mine;
-    atomicAdd(&counts[mine_id], 1);
+    wts[(int64_t)t * top + lane] = (p.renormalize ? mine / (wsum + p.sum_eps) : mine) * p.factor;
+    if (mine_id >= 0 && mine_id < p.rows_from) atomicAdd(&counts[mine_id], 1);
   }
 }
 
-// offsets [E + 1]; row_token, row_w [pairs]; pair_pos [pairs] (-1: a padding row's pair).
+// offsets [E + 1]; row_token, row_w [pairs]; pair_pos [pairs] (-1: the pair has no row).
 __global__ void __launch_bounds__(1024)
 moe_place_kernel(const int* __restrict__ ids, const float* __restrict__ wts, int pairs, int top, int E,
                  int* __restrict__ counts, int* __restrict__ offsets, int* __restrict__ row_token,
@@ -98,7 +153,7 @@ moe_place_kernel(const int* __restrict__ ids, const float* __restrict__ wts, int
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     const int e = ids[i];
-    if (e < 0) {
+    if (e < 0 || e >= E) {          // a padding row's choice, or an identity expert
       pair_pos[i] = -1;
       continue;
     }
@@ -134,7 +189,7 @@ template <typename T, bool GATED, bool GATHER>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ A, int64_t lda, const T* __restrict__ W,
                 const int* __restrict__ offsets, const int* __restrict__ row_token, const float* __restrict__ row_w,
-                int E, int N, int K) {
+                int E, int N, int K, int act, float limit) {
   atom::pdl_trigger();
   atom::pdl_wait();
   __shared__ float As[kMoeBK][kMoeBM + 1];
@@ -150,7 +205,7 @@ moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ A, int64_t lda, const
     const int r = threadIdx.x;
     if (r < rows) {
       a_row[r] = (GATHER ? (int64_t)row_token[row0 + r] : (int64_t)(row0 + r)) * lda;
-      a_mul[r] = GATHER ? row_w[row0 + r] : 1.f;
+      a_mul[r] = (GATHER && row_w) ? row_w[row0 + r] : 1.f;
     } else {
       a_row[r] = -1;
       a_mul[r] = 0.f;
@@ -200,8 +255,7 @@ moe_gemm_kernel(T* __restrict__ out, const T* __restrict__ A, int64_t lda, const
       float v = g;
       if (GATED) {
         // gate and up are rounded to the activation type first, as the unfused product hands them on
-        const float gr = to_float(from_float<T>(g)), ur = to_float(from_float<T>(u));
-        v = gr / (1.f + expf(-gr)) * ur;
+        v = gated_act(act, to_float(from_float<T>(g)), to_float(from_float<T>(u)), limit);
       }
       out[(int64_t)(row0 + r) * N + n0 + n] = from_float<T>(v);
     }
@@ -217,14 +271,19 @@ template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y, const int* __restrict__ pair_pos,
                                    const float* __restrict__ pair_w, int top, const T* __restrict__ shared_out,
                                    const float* __restrict__ gate, int64_t gate_ld, int n,
-                                   const int* __restrict__ seq_of_token) {
+                                   const int* __restrict__ seq_of_token, const T* __restrict__ x, int64_t ldx,
+                                   const int* __restrict__ ids, int identity_from) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int t = blockIdx.x;
   if (seq_of_token[t] < 0) return;
   const float sg = (shared_out && gate) ? 1.f / (1.f + expf(-gate[(int64_t)t * gate_ld])) : 1.f;
+  float own = 0.f;                        // the weights of the row's identity choices
+  if (x)
+    for (int k = 0; k < top; ++k)
+      if (ids[(int64_t)t * top + k] >= identity_from) own += pair_w ? pair_w[(int64_t)t * top + k] : 1.f;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
-    float sum = 0.f;
+    float sum = own != 0.f ? own * to_float(x[(int64_t)t * ldx + i]) : 0.f;
     for (int k = 0; k < top; ++k) {
       const int pos = pair_pos[(int64_t)t * top + k];
       if (pos >= 0) sum += (pair_w ? pair_w[(int64_t)t * top + k] : 1.f) * to_float(y[(int64_t)pos * n + i]);
@@ -265,11 +324,13 @@ constexpr size_t moe_tc_smem(int bm, bool gated, int bk, int stages) {
   return sizeof(__nv_bfloat16) * stages * ((size_t)bm + (gated ? 2 : 1) * kTcBN) * (bk + 8);
 }
 
-template <bool GATED, bool GATHER, int BM, int MI, int kTcBK, int kTcStages>
+// GATHER: 0 dense rows of A; 1 rows picked by row_token and weighted; 2 picked only (they come in with cp.async too).
+template <bool GATED, int GATHER, int BM, int MI, int kTcBK, int kTcStages>
 __global__ void __launch_bounds__(kTcThreads)
 moe_gemm_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ A, int64_t lda,
                    const __nv_bfloat16* __restrict__ W, const int* __restrict__ offsets,
-                   const int* __restrict__ row_token, const float* __restrict__ row_w, int E, int N, int K) {
+                   const int* __restrict__ row_token, const float* __restrict__ row_w, int E, int N, int K, int act,
+                   float limit) {
   atom::pdl_trigger();
   atom::pdl_wait();
   constexpr int kTcLD = kTcBK + 8;                         // bf16 elements per row in shared memory
@@ -289,7 +350,7 @@ moe_gemm_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restr
     const int r = threadIdx.x;
     if (r < rows) {
       a_row[r] = (GATHER ? (int64_t)row_token[row0 + r] : (int64_t)(row0 + r)) * lda;
-      a_mul[r] = GATHER ? row_w[row0 + r] : 1.f;
+      a_mul[r] = GATHER == 1 ? row_w[row0 + r] : 1.f;
     } else {
       a_row[r] = -1;
       a_mul[r] = 0.f;
@@ -307,7 +368,7 @@ moe_gemm_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restr
       const int r = idx / KC, c = idx - r * KC;
       const bool valid = a_row[r] >= 0 && k0 + c * 8 < K;
       __nv_bfloat16* dst = As + r * kTcLD + c * 8;
-      if (GATHER) {
+      if (GATHER == 1) {
         uint4 raw = make_uint4(0u, 0u, 0u, 0u);
         if (valid) {
           raw = *reinterpret_cast<const uint4*>(A + a_row[r] + k0 + c * 8);
@@ -397,9 +458,8 @@ moe_gemm_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restr
           float v = g[mi][nt][i];
           if (GATED) {
             // gate and up are rounded to the activation type first, as the unfused product hands them on
-            const float gr = __bfloat162float(__float2bfloat16_rn(v));
-            const float ur = __bfloat162float(__float2bfloat16_rn(u[mi][GATED ? nt : 0][i]));
-            v = gr / (1.f + expf(-gr)) * ur;
+            v = gated_act(act, __bfloat162float(__float2bfloat16_rn(v)),
+                          __bfloat162float(__float2bfloat16_rn(u[mi][GATED ? nt : 0][i])), limit);
           }
           out[(int64_t)(row0 + r) * N + n] = __float2bfloat16_rn(v);
         }
@@ -408,10 +468,10 @@ moe_gemm_tc_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restr
   }
 }
 
-template <bool GATED, bool GATHER, int BM, int MI, int BK, int STAGES>
+template <bool GATED, int GATHER, int BM, int MI, int BK, int STAGES>
 static int moe_gemm_tc_launch_one(__nv_bfloat16* out, const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W,
                                    const int* offsets, const int* row_token, const float* row_w, int R, int E, int N,
-                                   int K, cudaStream_t stream) {
+                                   int K, int act, float limit, cudaStream_t stream) {
   dim3 grid((R + BM - 1) / BM + E, (N + kTcBN - 1) / kTcBN);
   constexpr size_t smem = moe_tc_smem(BM, GATED, BK, STAGES);
   if (smem > 48 * 1024) {
@@ -424,7 +484,7 @@ static int moe_gemm_tc_launch_one(__nv_bfloat16* out, const __nv_bfloat16* A, in
     }
   }
   launch_pdl(moe_gemm_tc_kernel<GATED, GATHER, BM, MI, BK, STAGES>, grid, dim3(kTcThreads), smem, stream, out, A, lda, W, offsets,
-             row_token, row_w, E, N, K);
+             row_token, row_w, E, N, K, act, limit);
   return ATOM_OK;
 }
 
@@ -433,18 +493,20 @@ static int moe_gemm_tc_launch_one(__nv_bfloat16* out, const __nv_bfloat16* A, in
 // registers a thread and 60 KB a CTA leave an SM too few warps.)
 static int moe_gemm_tc_launch(__nv_bfloat16* out, const __nv_bfloat16* A, int64_t lda, const __nv_bfloat16* W,
                               const int* offsets, const int* row_token, const float* row_w, int R, int E, int N, int K,
-                              int gated, int gather, cudaStream_t stream) {
+                              int gated, int gather, float limit, cudaStream_t stream) {
   const bool small = R <= 16 * E;
   int rc = ATOM_OK;
 #define ATOM_MOE_TC(G, H)                                                                                                 \
   do {                                                                                                                    \
-    if (small) rc = moe_gemm_tc_launch_one<G, H, 16, 1, 64, 4>(out, A, lda, W, offsets, row_token, row_w, R, E, N, K, stream); \
-    else rc = moe_gemm_tc_launch_one<G, H, 64, 1, 32, 3>(out, A, lda, W, offsets, row_token, row_w, R, E, N, K, stream);      \
+    if (small) rc = moe_gemm_tc_launch_one<G, H, 16, 1, 64, 4>(out, A, lda, W, offsets, row_token, row_w, R, E, N, K, gated, limit, stream); \
+    else rc = moe_gemm_tc_launch_one<G, H, 64, 1, 32, 3>(out, A, lda, W, offsets, row_token, row_w, R, E, N, K, gated, limit, stream);      \
   } while (0)
-  if (gated && gather) ATOM_MOE_TC(true, true);
-  else if (gated) ATOM_MOE_TC(true, false);
-  else if (gather) ATOM_MOE_TC(false, true);
-  else ATOM_MOE_TC(false, false);
+  if (gated && gather && row_w) ATOM_MOE_TC(true, 1);
+  else if (gated && gather) ATOM_MOE_TC(true, 2);
+  else if (gated) ATOM_MOE_TC(true, 0);
+  else if (gather && row_w) ATOM_MOE_TC(false, 1);
+  else if (gather) ATOM_MOE_TC(false, 2);
+  else ATOM_MOE_TC(false, 0);
 #undef ATOM_MOE_TC
   if (rc != ATOM_OK) return rc;
   return check_launch();
@@ -452,10 +514,11 @@ static int moe_gemm_tc_launch(__nv_bfloat16* out, const __nv_bfloat16* A, int64_
 
 template <typename T>
 static int moe_gemm_launch(T* out, const T* A, int64_t lda, const T* W, const int* offsets, const int* row_token,
-                           const float* row_w, int R, int E, int N, int K, int gated, int gather, cudaStream_t stream) {
+                           const float* row_w, int R, int E, int N, int K, int gated, int gather, float limit,
+                           cudaStream_t stream) {
   dim3 grid((R + kMoeBM - 1) / kMoeBM + E, (N + kMoeBN - 1) / kMoeBN);
 #define ATOM_MOE(G, H) \
-  launch_pdl(moe_gemm_kernel<T, G, H>, grid, dim3(256), 0, stream, out, A, lda, W, offsets, row_token, row_w, E, N, K)
+  launch_pdl(moe_gemm_kernel<T, G, H>, grid, dim3(256), 0, stream, out, A, lda, W, offsets, row_token, row_w, E, N, K, gated, limit)
   if (gated && gather) ATOM_MOE(true, true);
   else if (gated) ATOM_MOE(true, false);
   else if (gather) ATOM_MOE(false, true);
@@ -466,13 +529,18 @@ static int moe_gemm_launch(T* out, const T* A, int64_t lda, const T* W, const in
 
 }  // namespace atom
 
-ATOM_EXPORT int atom_moe_route(const float* logits, int64_t ld, int T, int E, int top, int softmax_scores,
-                               int renormalize, const int* seq_of_token, int* ids, float* wts, int* counts,
-                               cudaStream_t stream) {
+// E: the router's outputs, of which the last `identity` are identity experts.
+ATOM_EXPORT int atom_moe_route(const float* logits, int64_t ld, int T, int E, int identity, int top, int softmax_scores,
+                               int renormalize, float sum_eps, float factor, const void* correction,
+                               int correction_dtype, int groups, int keep, const int* seq_of_token, int* ids,
+                               float* wts, int* counts, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  if (E <= 0 || E > 1024 || top <= 0 || top > 32 || top > E) return ATOM_ERR_ARG;
-  atom::launch_pdl(atom::moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, E, top, softmax_scores,
-                   renormalize, seq_of_token, T, ids, wts, counts);
+  if (E <= 0 || E > 1024 || top <= 0 || top > 32 || top > E || identity < 0 || identity >= E) return ATOM_ERR_ARG;
+  if (groups > 1 && (E % groups || keep < 1 || keep > groups || top > keep * (E / groups))) return ATOM_ERR_ARG;
+  const atom::MoeRouteArgs p{E, E - identity, top, softmax_scores, renormalize, sum_eps, factor, correction,
+                             correction_dtype, groups, keep};
+  atom::launch_pdl(atom::moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, p, seq_of_token, T, ids,
+                   wts, counts);
   return atom::check_launch();
 }
 
@@ -485,39 +553,43 @@ ATOM_EXPORT int atom_moe_place(const int* ids, const float* wts, int pairs, int 
   return atom::check_launch();
 }
 
-// R: the most rows there can be (rows of the step x top); the kernel finds the real ones from `offsets`.
+// R: the most rows there can be (rows of the step x top); the kernel finds the real ones from `offsets`.  gated: 0, or
+// the activation (gate_act.cuh) of which `limit` is the clamp; row_w null: gathered rows come in as they are.
 ATOM_EXPORT int atom_moe_gemm(void* out, const void* A, int dtype, int64_t lda, const void* W, const int* offsets,
                               const int* row_token, const float* row_w, int R, int E, int N, int K, int gated,
-                              int gather, int tc, cudaStream_t stream) {
+                              int gather, int tc, float limit, cudaStream_t stream) {
   if (R <= 0) return ATOM_OK;
-  if (E <= 0 || N <= 0 || K <= 0 || (gather && (!row_token || !row_w))) return ATOM_ERR_ARG;
+  if (E <= 0 || N <= 0 || K <= 0 || (gather && !row_token)) return ATOM_ERR_ARG;
+  if (gated != 0 && gated != atom::kGateSilu && gated != atom::kGateClamped) return ATOM_ERR_ARG;
   if (dtype == ATOM_F32)
     return atom::moe_gemm_launch<float>((float*)out, (const float*)A, lda, (const float*)W, offsets, row_token, row_w,
-                                        R, E, N, K, gated, gather, stream);
+                                        R, E, N, K, gated, gather, limit, stream);
   if (dtype == ATOM_BF16 && tc && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0)
     return atom::moe_gemm_tc_launch((__nv_bfloat16*)out, (const __nv_bfloat16*)A, lda, (const __nv_bfloat16*)W, offsets,
-                                    row_token, row_w, R, E, N, K, gated, gather, stream);
+                                    row_token, row_w, R, E, N, K, gated, gather, limit, stream);
   if (dtype == ATOM_BF16)
     return atom::moe_gemm_launch<__nv_bfloat16>((__nv_bfloat16*)out, (const __nv_bfloat16*)A, lda,
                                                 (const __nv_bfloat16*)W, offsets, row_token, row_w, R, E, N, K, gated,
-                                                gather, stream);
+                                                gather, limit, stream);
   return ATOM_ERR_ARG;
 }
 
 ATOM_EXPORT int atom_moe_combine(void* out, const void* y, int dtype, const int* pair_pos, const float* pair_w, int top,
                                  const void* shared_out, const float* gate, int64_t gate_ld, int T, int n,
-                                 const int* seq_of_token, cudaStream_t stream) {
+                                 const int* seq_of_token, const void* x, int64_t ldx, const int* ids,
+                                 int identity_from, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  if (n <= 0 || top <= 0) return ATOM_ERR_ARG;
+  if (n <= 0 || top <= 0 || (x && !ids)) return ATOM_ERR_ARG;
   // few rows: the columns are shared out among CTAs too (a row's sums are chains of dependent loads)
   const dim3 grid(T, T >= 512 ? 1 : (unsigned)min(8, (n + 255) / 256));
   if (dtype == ATOM_F32)
     atom::launch_pdl(atom::moe_combine_kernel<float>, grid, dim3(256), 0, stream, (float*)out, (const float*)y,
-                     pair_pos, pair_w, top, (const float*)shared_out, gate, gate_ld, n, seq_of_token);
+                     pair_pos, pair_w, top, (const float*)shared_out, gate, gate_ld, n, seq_of_token, (const float*)x, ldx, ids,
+                     identity_from);
   else if (dtype == ATOM_BF16)
     atom::launch_pdl(atom::moe_combine_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (__nv_bfloat16*)out,
                      (const __nv_bfloat16*)y, pair_pos, pair_w, top, (const __nv_bfloat16*)shared_out, gate, gate_ld, n,
-                     seq_of_token);
+                     seq_of_token, (const __nv_bfloat16*)x, ldx, ids, identity_from);
   else
     return ATOM_ERR_ARG;
   return atom::check_launch();

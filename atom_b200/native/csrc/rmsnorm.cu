@@ -249,7 +249,7 @@ ATOM_EXPORT int atom_rmsnorm(void* out, const void* x, int act_dtype, const void
 
 // A sub-block whose output passes an RMSNorm of its own before it enters the residual stream, fused with the norm
 // that reads the stream next:
-//   r = residual[row] + rmsnorm(delta[row]; wd, eps_d);   residual[row] = r (unless rows are picked);
+//   r = residual[row] + dscale * rmsnorm(delta[row]; wd, eps_d);   residual[row] = r (unless rows are picked);
 //   out = rmsnorm(r; w, eps)
 // all in 32-bit; the row's numbers wait in shared memory between the passes.
 namespace atom {
@@ -258,7 +258,7 @@ template <typename TA>
 __global__ void normed_add_rmsnorm_kernel(TA* __restrict__ out, float* __restrict__ residual,
                                           const TA* __restrict__ delta, const void* __restrict__ wd, float eps_d,
                                           const void* __restrict__ w, int w_dtype, float eps,
-                                          const int* __restrict__ rows, int H) {
+                                          const int* __restrict__ rows, int H, float dscale) {
   atom::pdl_trigger();
   atom::pdl_wait();
   extern __shared__ float row_s[];
@@ -277,7 +277,7 @@ __global__ void normed_add_rmsnorm_kernel(TA* __restrict__ out, float* __restric
   const float rd = rsqrtf(sd / (float)H + eps_d);
   float ss = 0.f;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float v = res[i] + row_s[i] * rd * load_as_float(wd, w_dtype, i);
+    const float v = res[i] + row_s[i] * rd * load_as_float(wd, w_dtype, i) * dscale;
     row_s[i] = v;
     if (!rows) res[i] = v;
     ss = fmaf(v, v, ss);
@@ -312,7 +312,7 @@ template <int NV>
 __global__ void normed_add_rmsnorm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ residual,
                                                    const __nv_bfloat16* __restrict__ delta, const void* __restrict__ wd,
                                                    float eps_d, const void* __restrict__ w, int w_dtype, float eps,
-                                                   const int* __restrict__ rows, int H) {
+                                                   const int* __restrict__ rows, int H, float dscale) {
   atom::pdl_trigger();
   atom::pdl_wait();
   __shared__ float scratch[32];
@@ -342,7 +342,7 @@ __global__ void normed_add_rmsnorm_bf16_vec_kernel(__nv_bfloat16* __restrict__ o
       load8(res, ATOM_F32, i, rv);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        v[k][e] = rv[e] + v[k][e] * rd * wv[e];
+        v[k][e] = rv[e] + v[k][e] * rd * wv[e] * dscale;
         ss = fmaf(v[k][e], v[k][e], ss);
       }
       if (!rows) {
@@ -375,7 +375,7 @@ __global__ void normed_add_rmsnorm_bf16_vec_kernel(__nv_bfloat16* __restrict__ o
 // wd and w have one type (w_dtype).
 ATOM_EXPORT int atom_normed_add_rmsnorm(void* out, int act_dtype, float* residual, const void* delta, const void* wd,
                                         float eps_d, const void* w, int w_dtype, float eps, const int* rows, int n_rows,
-                                        int H, cudaStream_t stream) {
+                                        int H, float dscale, cudaStream_t stream) {
   if (n_rows <= 0) return ATOM_OK;
   if (H <= 0 || H > 48 * 256 || !delta || !wd || (w_dtype != ATOM_F32 && w_dtype != ATOM_BF16)) return ATOM_ERR_ARG;
   const int threads = atom::norm_threads(H);
@@ -392,18 +392,18 @@ ATOM_EXPORT int atom_normed_add_rmsnorm(void* out, int act_dtype, float* residua
     if (th < 64) th = 64;
     if (nv == 1)
       atom::launch_pdl(atom::normed_add_rmsnorm_bf16_vec_kernel<1>, dim3(n_rows), dim3(th), 0, stream, (__nv_bfloat16*)out,
-                       residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H);
+                       residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H, dscale);
     else
       atom::launch_pdl(atom::normed_add_rmsnorm_bf16_vec_kernel<2>, dim3(n_rows), dim3(th), 0, stream, (__nv_bfloat16*)out,
-                       residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H);
+                       residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H, dscale);
     return atom::check_launch();
   }
   if (act_dtype == ATOM_F32)
     atom::launch_pdl(atom::normed_add_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), smem, stream, (float*)out,
-                     residual, (const float*)delta, wd, eps_d, w, w_dtype, eps, rows, H);
+                     residual, (const float*)delta, wd, eps_d, w, w_dtype, eps, rows, H, dscale);
   else if (act_dtype == ATOM_BF16)
     atom::launch_pdl(atom::normed_add_rmsnorm_kernel<__nv_bfloat16>, dim3(n_rows), dim3(threads), smem, stream,
-                     (__nv_bfloat16*)out, residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H);
+                     (__nv_bfloat16*)out, residual, (const __nv_bfloat16*)delta, wd, eps_d, w, w_dtype, eps, rows, H, dscale);
   else
     return ATOM_ERR_ARG;
   return atom::check_launch();

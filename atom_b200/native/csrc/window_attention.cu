@@ -5,13 +5,17 @@
 //                               y_t[c] = sum_j w[c, j] * u_(t - taps + 1 + j)[c]        (zeros before the request's start)
 //                             with rows before the step's first token of a request taken from the request's
 //                             convolution state (its last taps - 1 projected rows); rotation of the first rot_dims
-//                             numbers of every query and key head by position * frequency (pairs (i, i + rot_dims/2));
-//                             q to a dense array, k and v to their pages (conv_rope_write_vec_kernel: the same
-//                             for bfloat16 sizes in steps of 8, 16 bytes at a time)
+//                             numbers of every query and key head by position * frequency (pairs (i, i + rot_dims/2),
+//                             or neighbours (2i, 2i + 1)), cos and sin times a constant; optionally a bias on every
+//                             channel (without a convolution), and values blended with another layer's values of
+//                             the same token, v <- (1 - mix) v + mix v_first; q to a dense array, k and v to their
+//                             pages (conv_rope_write_vec_kernel: the same for bfloat16 sizes in steps of 8, 16 bytes
+//                             at a time)
 //   conv_state_update_kernel  per request: the last taps - 1 projected rows after this step
 //   window_attention_kernel   one CTA per (token, query head): keys j <= p with p - j < window or j < keep_first,
 //                             s = scale * q.k, s <- cap * tanh(s / cap), online softmax in 32-bit; any sizes, both
-//                             precisions
+//                             precisions; optionally a sink per head (exp(sink_h) is added to the denominator), a
+//                             gate number per head (the output times sigmoid(gate)) and a constant on the output
 // Convolution sums, angles, scores, weights and sums are 32-bit in both precisions.
 #include "common.cuh"
 
@@ -36,6 +40,17 @@ __device__ __forceinline__ float conv_at(const T* __restrict__ qkv, int64_t ld, 
   return y;
 }
 
+// What the kernels below take beside the convolution and the plain rotation.
+struct RopeExtras {
+  const void* bias;      // [C] added to every projected channel (null: none; not together with a convolution)
+  int bias_dtype;
+  int neighbours;        // 1: rotated pairs are (2i, 2i + 1); 0: (i, i + rot_dims / 2)
+  float mag;             // factor on cos and sin
+  const void* v_first;   // [T, G dv] dense, activation type: values to blend in (null: none)
+  float v_mix;
+  void* v_keep;          // [T, G dv] dense: takes a copy of this layer's values (null: none)
+};
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t ld, int H, int G, int dk, int dv,
@@ -44,7 +59,7 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
                        const int* __restrict__ seq_of_token, const int* __restrict__ cu_q,
                        const int* __restrict__ state_slots, const int* __restrict__ block_table, int max_pages,
                        int page_size, T* __restrict__ k_pages, T* __restrict__ v_pages, int64_t num_pages,
-                       int* __restrict__ status) {
+                       int* __restrict__ status, const RopeExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int t = blockIdx.x;
@@ -64,10 +79,15 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
   const int slot = p % page_size;
   const int half = rot_dims / 2;
   const float pos = (float)p;
+  auto value_at = [&](int c) {
+    float y = conv_at(qkv, ld, state_row, C, taps, conv_w, w_dtype, first, t, c);
+    if (x.bias) y += load_as_float(x.bias, x.bias_dtype, c);
+    return y;
+  };
   // queries and keys: H + G vectors of dk numbers
   for (int idx = threadIdx.x; idx < (H + G) * dk; idx += blockDim.x) {
     const int n = idx / dk, i = idx - n * dk;
-    if (i >= half && i < rot_dims) continue;      // the second of a pair: written by the first
+    if (x.neighbours ? (i < rot_dims && (i & 1)) : (i >= half && i < rot_dims)) continue;   // written by the pair's first
     const int c = n * dk + i;                      // (keys follow the queries in the row)
     T* dst;
     if (n < H) {
@@ -76,23 +96,27 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
       if (!writes) continue;
       dst = k_pages + (((int64_t)page * G + (n - H)) * page_size + slot) * dk;
     }
-    const float a = conv_at(qkv, ld, state_row, C, taps, conv_w, w_dtype, first, t, c);
-    if (i < half) {
-      const float b = conv_at(qkv, ld, state_row, C, taps, conv_w, w_dtype, first, t, c + half);
+    const float a = value_at(c);
+    if (i < rot_dims) {
+      const int other = x.neighbours ? 1 : half;
+      const float b = value_at(c + other);
       float sn, cs;
-      sincosf(pos * freq[i], &sn, &cs);
+      sincosf(pos * freq[x.neighbours ? i >> 1 : i], &sn, &cs);
+      sn *= x.mag;
+      cs *= x.mag;
       dst[i] = from_float<T>(a * cs - b * sn);
-      dst[i + half] = from_float<T>(b * cs + a * sn);
+      dst[i + other] = from_float<T>(b * cs + a * sn);
     } else {
       dst[i] = from_float<T>(a);
     }
   }
-  if (!writes) return;
   const int v0 = (H + G) * dk;
   for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) {
     const int g = idx / dv, i = idx - g * dv;
-    v_pages[(((int64_t)page * G + g) * page_size + slot) * dv + i] =
-        from_float<T>(conv_at(qkv, ld, state_row, C, taps, conv_w, w_dtype, first, t, v0 + idx));
+    float v = value_at(v0 + idx);
+    if (x.v_first) v = (1.f - x.v_mix) * v + x.v_mix * to_float(((const T*)x.v_first)[(int64_t)t * G * dv + idx]);
+    if (x.v_keep) ((T*)x.v_keep)[(int64_t)t * G * dv + idx] = from_float<T>(v);
+    if (writes) v_pages[(((int64_t)page * G + g) * page_size + slot) * dv + i] = from_float<T>(v);
   }
 }
 
@@ -109,10 +133,10 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
                            const int* __restrict__ cu_q, const int* __restrict__ state_slots,
                            const int* __restrict__ block_table, int max_pages, int page_size,
                            __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages, int64_t num_pages,
-                           int* __restrict__ status) {
+                           int* __restrict__ status, const RopeExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
-  extern __shared__ __align__(16) float cv_y[];      // [C]
+  extern __shared__ __align__(16) float cv_y[];      // [C], then cos and sin of the rotated pairs
   const int t = blockIdx.x;
   const int s = seq_of_token[t];
   if (s < 0) return;
@@ -130,6 +154,15 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
   }
   const int slot = p % page_size;
   const int groups = C / 8;
+  const int half = rot_dims / 2;
+  float* ang_c = cv_y + C;
+  float* ang_s = ang_c + half;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {      // (all heads of the token share the angles)
+    float sn, cs;
+    sincosf((float)p * freq[i], &sn, &cs);
+    ang_c[i] = cs * x.mag;
+    ang_s[i] = sn * x.mag;
+  }
   for (int g = threadIdx.x; g < groups; g += blockDim.x) {
     const int c = g * 8;
     float y[8];
@@ -141,6 +174,21 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
         const float2 f = __bfloat1622float2(h2[e]);
         y[2 * e] = f.x;
         y[2 * e + 1] = f.y;
+      }
+      if (x.bias) {
+        if (x.bias_dtype == ATOM_F32) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[e] += ((const float*)x.bias)[c + e];
+        } else {
+          const uint4 braw = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)x.bias + c);
+          const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(&braw);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(b2[e]);
+            y[2 * e] += f.x;
+            y[2 * e + 1] += f.y;
+          }
+        }
       }
     } else {
       constexpr int NW = TAPS > 0 ? TAPS : 1;
@@ -167,14 +215,14 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
     *reinterpret_cast<float4*>(cv_y + c + 4) = make_float4(y[4], y[5], y[6], y[7]);
   }
   __syncthreads();
-  const int half = rot_dims / 2;
-  const float pos = (float)p;
   const int qk_end = (H + G) * dk;
   for (int g = threadIdx.x; g < groups; g += blockDim.x) {
     const int c = g * 8;
     __nv_bfloat16* dst;
     int i0 = 0;
     bool rotated = false;
+    int64_t keep_at = -1;
+    float o[8];
     if (c < qk_end) {
       const int n = c / dk;
       i0 = c - n * dk;
@@ -186,33 +234,47 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
         dst = k_pages + (((int64_t)page * G + (n - H)) * page_size + slot) * dk + i0;
       }
     } else {
-      if (!writes) continue;
+      if (!writes && !x.v_keep) continue;
       const int idx = c - qk_end;
       const int gg = idx / dv;
-      dst = v_pages + (((int64_t)page * G + gg) * page_size + slot) * dv + (idx - gg * dv);
+      keep_at = (int64_t)t * G * dv + idx;
+      dst = writes ? v_pages + (((int64_t)page * G + gg) * page_size + slot) * dv + (idx - gg * dv) : nullptr;
     }
-    float o[8];
-    if (rotated) {
+    if (rotated && x.neighbours) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float a = cv_y[c + 2 * e], b = cv_y[c + 2 * e + 1];
+        const float cs = ang_c[(i0 >> 1) + e], sn = ang_s[(i0 >> 1) + e];
+        o[2 * e] = a * cs - b * sn;
+        o[2 * e + 1] = b * cs + a * sn;
+      }
+    } else if (rotated) {
       const bool low = i0 < half;                      // the first of the pair: (a, b) = (own, + half); else (- half, own)
       const float* av = cv_y + (low ? c : c - half);
       const float* bv = cv_y + (low ? c + half : c);
-      const float* fr = freq + (low ? i0 : i0 - half);
+      const int f0 = low ? i0 : i0 - half;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        float sn, cs;
-        sincosf(pos * fr[e], &sn, &cs);
+        const float cs = ang_c[f0 + e], sn = ang_s[f0 + e];
         const float a = av[e], b = bv[e];
         o[e] = low ? a * cs - b * sn : b * cs + a * sn;
       }
     } else {
 #pragma unroll
       for (int e = 0; e < 8; ++e) o[e] = cv_y[c + e];
+      if (keep_at >= 0 && x.v_first) {
+        const uint4 raw = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)x.v_first + keep_at);
+        const __nv_bfloat16* fv = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = (1.f - x.v_mix) * o[e] + x.v_mix * __bfloat162float(fv[e]);
+      }
     }
     uint4 packed;
     __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
     for (int e = 0; e < 4; ++e) h2[e] = __floats2bfloat162_rn(o[2 * e], o[2 * e + 1]);
-    *reinterpret_cast<uint4*>(dst) = packed;
+    if (keep_at >= 0 && x.v_keep) *reinterpret_cast<uint4*>((__nv_bfloat16*)x.v_keep + keep_at) = packed;
+    if (dst) *reinterpret_cast<uint4*>(dst) = packed;
   }
 }
 
@@ -235,6 +297,23 @@ __global__ void conv_state_update_kernel(T* __restrict__ conv_state, const T* __
   }
 }
 
+// Beside the softmax over keys: a sink per head, a gate number per (token, head), a constant on the output, and the
+// output's row stride (a row may be part of a wider one).
+struct AttnExtras {
+  const float* sink;     // [nh] or null
+  const void* gate;      // [T, nh] rows at stride gate_ld, activation type, or null
+  int64_t gate_ld;
+  float out_mul;
+  int64_t out_ld;
+};
+
+template <typename T>
+__device__ __forceinline__ float attn_out_factor(const AttnExtras& x, int t, int h) {
+  float f = x.out_mul;
+  if (x.gate) f /= 1.f + expf(-to_float(((const T*)x.gate)[(int64_t)t * x.gate_ld + h]));
+  return f;
+}
+
 constexpr int kWinThreads = 128;
 constexpr int kWinChunk = 256;
 
@@ -243,7 +322,8 @@ __global__ void __launch_bounds__(kWinThreads)
 window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ k_pages,
                         const T* __restrict__ v_pages, const int* __restrict__ block_table, int max_pages,
                         int page_size, const int* __restrict__ positions, const int* __restrict__ seq_of_token, int nh,
-                        int nkv, int dk, int dv, float scale, float softcap, int window, int keep_first) {
+                        int nkv, int dk, int dv, float scale, float softcap, int window, int keep_first,
+                        const AttnExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -309,8 +389,9 @@ window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
     }
     __syncthreads();
   }
-  T* orow = out + ((int64_t)t * nh + h) * dv;
-  const float inv = 1.f / l;
+  T* orow = out + (int64_t)t * x.out_ld + (int64_t)h * dv;
+  if (x.sink) l += expf(x.sink[h] - m);
+  const float inv = attn_out_factor<T>(x, t, h) / l;
 #pragma unroll
   for (int a = 0; a < 4; ++a) {
     const int d = threadIdx.x + a * kWinThreads;
@@ -322,7 +403,8 @@ window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
 // a share's running maximum (natural logarithm), sum and unnormalised output.  One CTA per (token, head).
 template <typename T>
 __global__ void window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part,
-                                              const int* __restrict__ seq_of_token, int nh, int dv, int nsplit) {
+                                              const int* __restrict__ seq_of_token, int nh, int dv, int nsplit,
+                                              const AttnExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -331,6 +413,8 @@ __global__ void window_attention_merge_kernel(T* __restrict__ out, const float* 
   const float* pt = part + (int64_t)t * nsplit * stride;
   float M = -INFINITY;
   for (int s = 0; s < nsplit; ++s) M = fmaxf(M, pt[s * stride + h]);
+  const float sink = x.sink ? expf(x.sink[h] - M) : 0.f;
+  const float f = attn_out_factor<T>(x, t, h);
   for (int i = threadIdx.x; i < dv; i += blockDim.x) {
     float L = 0.f, o = 0.f;
     for (int s = 0; s < nsplit; ++s) {
@@ -339,7 +423,7 @@ __global__ void window_attention_merge_kernel(T* __restrict__ out, const float* 
       L = fmaf(pt[s * stride + nh + h], w, L);
       o = fmaf(pt[s * stride + 2 * nh + (int64_t)h * dv + i], w, o);
     }
-    out[((int64_t)t * nh + h) * dv + i] = from_float<T>(o / L);
+    out[(int64_t)t * x.out_ld + (int64_t)h * dv + i] = from_float<T>(o * (f / (L + sink)));
   }
 }
 
@@ -352,8 +436,11 @@ ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, in
                                      const float* freq, int rot_dims, const int* positions, const int* seq_of_token,
                                      const int* cu_q, const int* state_slots, const int* block_table, int max_pages,
                                      int page_size, void* k_pages, void* v_pages, int64_t num_pages, int* status,
-                                     cudaStream_t stream) {
+                                     const void* bias, int bias_dtype, int neighbours, float mag, const void* v_first,
+                                     float v_mix, void* v_keep, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
+  if (bias && taps > 0) return ATOM_ERR_ARG;
+  const atom::RopeExtras x{bias, bias_dtype, neighbours, mag, v_first, v_mix, v_keep};
   if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dk || taps < 0 ||
       page_size <= 0 || (rot_dims > 0 && !freq) || (taps > 0 && !conv_w))
     return ATOM_ERR_ARG;
@@ -361,19 +448,20 @@ ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, in
     atom::launch_pdl(atom::conv_rope_write_kernel<float>, dim3(T), dim3(256), 0, stream, (float*)q_out,
                      (const float*)qkv, ld, H, G, dk, dv, conv_w, w_dtype, taps, (const float*)conv_state, freq,
                      rot_dims, positions, seq_of_token, cu_q, state_slots, block_table, max_pages, page_size,
-                     (float*)k_pages, (float*)v_pages, num_pages, status);
-  else if (dtype == ATOM_BF16 && dk % 8 == 0 && dv % 8 == 0 && rot_dims % 16 == 0 && ld % 8 == 0 && taps <= 8 &&
+                     (float*)k_pages, (float*)v_pages, num_pages, status, x);
+  else if (dtype == ATOM_BF16 && dk % 8 == 0 && dv % 8 == 0 && rot_dims % (neighbours ? 8 : 16) == 0 && ld % 8 == 0 && taps <= 8 &&
            (taps == 0 || w_dtype == ATOM_BF16) && ((H + 2 * G) * dk + G * dv) * sizeof(float) <= 48 * 1024 &&
            ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)conv_w % 16) == 0 && ((uintptr_t)conv_state % 16) == 0 &&
+           ((uintptr_t)bias % 16) == 0 && ((uintptr_t)v_first % 16) == 0 && ((uintptr_t)v_keep % 16) == 0 &&
            ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0) {
     const int C = (H + G) * dk + G * dv;
     const int threads = C / 8 >= 256 ? 256 : ((C / 8 + 31) / 32) * 32;
 #define ATOM_CV(TAPS)                                                                                               \
-  atom::launch_pdl(atom::conv_rope_write_vec_kernel<TAPS>, dim3(T), dim3(threads), C * sizeof(float), stream,       \
+  atom::launch_pdl(atom::conv_rope_write_vec_kernel<TAPS>, dim3(T), dim3(threads), (C + rot_dims) * sizeof(float), stream, \
                    (__nv_bfloat16*)q_out, (const __nv_bfloat16*)qkv, ld, H, G, dk, dv, (const __nv_bfloat16*)conv_w, \
                    (const __nv_bfloat16*)conv_state, freq, rot_dims, positions, seq_of_token, cu_q, state_slots,    \
                    block_table, max_pages, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages,  \
-                   status)
+                   status, x)
     switch (taps) {
       case 0: ATOM_CV(0); break;
       case 1: ATOM_CV(1); break;
@@ -391,7 +479,7 @@ ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, in
                      (__nv_bfloat16*)q_out, (const __nv_bfloat16*)qkv, ld, H, G, dk, dv, conv_w, w_dtype, taps,
                      (const __nv_bfloat16*)conv_state, freq, rot_dims, positions, seq_of_token, cu_q, state_slots,
                      block_table, max_pages, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages,
-                     status);
+                     status, x);
   else
     return ATOM_ERR_ARG;
   return atom::check_launch();
@@ -413,12 +501,15 @@ ATOM_EXPORT int atom_conv_state_update(void* conv_state, const void* qkv, int dt
   return atom::check_launch();
 }
 
-// out [T, nh dv]; q [T, nh dk] dense.  window <= 0: every earlier key; softcap <= 0: none.
+// out: row t at out + t * out_ld, heads packed [nh, dv]; q [T, nh dk] dense.  window <= 0: every earlier key;
+// softcap <= 0: none; sink, gate null: none.
 ATOM_EXPORT int atom_window_attention(void* out, const void* q, int dtype, const void* k_pages, const void* v_pages,
                                       const int* block_table, int max_pages, int page_size, const int* positions,
                                       const int* seq_of_token, int T, int nh, int nkv, int dk, int dv, float scale,
-                                      float softcap, int window, int keep_first, cudaStream_t stream) {
+                                      float softcap, int window, int keep_first, const float* sink, const void* gate,
+                                      int64_t gate_ld, float out_mul, int64_t out_ld, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
+  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld};
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || dk <= 0 || dv <= 0 || dv > 4 * atom::kWinThreads || dk > 4096 ||
       page_size <= 0 || nh > 65535 || keep_first < 0)
     return ATOM_ERR_ARG;
@@ -427,28 +518,30 @@ ATOM_EXPORT int atom_window_attention(void* out, const void* q, int dtype, const
   if (dtype == ATOM_F32)
     atom::launch_pdl(atom::window_attention_kernel<float>, grid, dim3(atom::kWinThreads), smem, stream, (float*)out,
                      (const float*)q, (const float*)k_pages, (const float*)v_pages, block_table, max_pages, page_size,
-                     positions, seq_of_token, nh, nkv, dk, dv, scale, softcap, window, keep_first);
+                     positions, seq_of_token, nh, nkv, dk, dv, scale, softcap, window, keep_first, x);
   else if (dtype == ATOM_BF16)
     atom::launch_pdl(atom::window_attention_kernel<__nv_bfloat16>, grid, dim3(atom::kWinThreads), smem, stream,
                      (__nv_bfloat16*)out, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
                      (const __nv_bfloat16*)v_pages, block_table, max_pages, page_size, positions, seq_of_token, nh,
-                     nkv, dk, dv, scale, softcap, window, keep_first);
+                     nkv, dk, dv, scale, softcap, window, keep_first, x);
   else
     return ATOM_ERR_ARG;
   return atom::check_launch();
 }
 
 ATOM_EXPORT int atom_window_attention_merge(void* out, int dtype, const float* part, const int* seq_of_token, int T, int nh,
-                                            int dv, int nsplit, cudaStream_t stream) {
+                                            int dv, int nsplit, const float* sink, const void* gate, int64_t gate_ld,
+                                            float out_mul, int64_t out_ld, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
+  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld};
   if (nsplit < 1 || part == nullptr || nh <= 0 || nh > 65535 || dv <= 0) return ATOM_ERR_ARG;
   const int threads = dv >= 128 ? 128 : (dv >= 64 ? 64 : 32);
   if (dtype == ATOM_F32)
     atom::launch_pdl(atom::window_attention_merge_kernel<float>, dim3(T, nh), dim3(threads), 0, stream, (float*)out, part,
-                     seq_of_token, nh, dv, nsplit);
+                     seq_of_token, nh, dv, nsplit, x);
   else if (dtype == ATOM_BF16)
     atom::launch_pdl(atom::window_attention_merge_kernel<__nv_bfloat16>, dim3(T, nh), dim3(threads), 0, stream,
-                     (__nv_bfloat16*)out, part, seq_of_token, nh, dv, nsplit);
+                     (__nv_bfloat16*)out, part, seq_of_token, nh, dv, nsplit, x);
   else
     return ATOM_ERR_ARG;
   return atom::check_launch();

@@ -13,6 +13,8 @@
 // and unnormalised output per (token, head) in a scratch array that window_attention.cu's merge kernel puts together.
 // In a step of single tokens a CTA's rows are the query heads that share one key head, so a request's keys and values
 // are read once per key head.
+// A sink per head adds exp(sink_h) to the denominator; a gate number per (token, head) and a constant multiply the
+// output, whose rows may lie further apart (with shares the merge kernel does all of this).
 #include "common.cuh"
 
 #if !defined(ATOM_WA_DK) || !defined(ATOM_WA_DV)
@@ -99,6 +101,10 @@ struct Params {
   int window, keep;
   int nsplit;
   float* part;
+  const float* sink;               // [nh] or null
+  const __nv_bfloat16* gate;       // [T, nh] rows at stride gate_ld, or null
+  int64_t gate_ld, out_ld;
+  float out_mul;
 };
 
 // Two threads per key row: the page is looked up once per row and tile, the row's 16-byte pieces alternate between them.
@@ -310,8 +316,12 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
     for (int k = 0; k < 2; ++k) {
       const int row = k ? row_b : row_a;
       if (row >= rows) continue;
-      const float inv = l_run[k] > 0.f ? 1.f / l_run[k] : 0.f;
-      __nv_bfloat16* dst = p.out + (int64_t)(HEADS ? t0 : t0 + row) * p.nh * DV + (int64_t)(HEADS ? h + row : h) * DV;
+      const int tt = HEADS ? t0 : t0 + row, hh = HEADS ? h + row : h;
+      float l = l_run[k];
+      if (p.sink) l += ex2(p.sink[hh] * kLog2e - m_run[k]);
+      float inv = l > 0.f ? p.out_mul / l : 0.f;
+      if (p.gate) inv = __fdividef(inv, 1.f + ex2(-kLog2e * __bfloat162float(p.gate[(int64_t)tt * p.gate_ld + hh])));
+      __nv_bfloat16* dst = p.out + (int64_t)tt * p.out_ld + (int64_t)hh * DV;
 #pragma unroll
       for (int nt = 0; nt < DV / 8; ++nt)
         *reinterpret_cast<__nv_bfloat162*>(dst + nt * 8 + col) =
@@ -345,7 +355,7 @@ ATOM_EXPORT void atom_watc_sizes(int* dk, int* dv) {
   *dv = atom::watc::DV;
 }
 
-// out [T, nh * DV]; q: row t at q + t * q_stride, heads packed [nh, DK]; k_pages [pages, nkv, page, DK]; v_pages
+// out: row t at out + t * out_ld, heads packed [nh, DV]; q: row t at q + t * q_stride, heads packed [nh, DK]; k_pages [pages, nkv, page, DK]; v_pages
 // [pages, nkv, page, DV]; units: an upper bound of the step's tiles (ceil(T / 64) + num_seqs), or with heads_rows (a
 // step of single tokens: a CTA's rows are the query heads of one key head) the step's tokens.  nsplit > 1: part holds
 // T * nsplit * nh * (DV + 2) floats, which attention_mixed.cu's merge kernel puts together.
@@ -353,11 +363,13 @@ ATOM_EXPORT int atom_window_attention_tc(void* out, const void* q, int64_t q_str
                                          const void* v_pages, int64_t num_pages, const int* block_table, int max_pages,
                                          int page_size, const int* positions, const int* seq_of_token, const int* cu_q,
                                          int num_seqs, int units, int nh, int nkv, float scale, float cap, int window,
-                                         int keep, int nsplit, float* part, int heads_rows, cudaStream_t stream) {
+                                         int keep, int nsplit, float* part, int heads_rows, const float* sink,
+                                         const void* gate, int64_t gate_ld, float out_mul, int64_t out_ld,
+                                         cudaStream_t stream) {
   using namespace atom::watc;
   if (units <= 0) return ATOM_OK;
   if (nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || nsplit < 1 || nsplit > 65535 || nh > 65535 ||
-      (nsplit > 1 && part == nullptr) || (q_stride % 8) != 0 || (heads_rows && nh / nkv > BM))
+      (nsplit > 1 && part == nullptr) || (q_stride % 8) != 0 || (out_ld % 2) != 0 || (heads_rows && nh / nkv > BM))
     return ATOM_ERR_ARG;
   Params p;
   p.out = (__nv_bfloat16*)out;
@@ -381,6 +393,11 @@ ATOM_EXPORT int atom_window_attention_tc(void* out, const void* q, int64_t q_str
   p.keep = window > 0 ? keep : 0;
   p.nsplit = nsplit;
   p.part = part;
+  p.sink = sink;
+  p.gate = (const __nv_bfloat16*)gate;
+  p.gate_ld = gate_ld;
+  p.out_ld = out_ld;
+  p.out_mul = out_mul;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(window_attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,

@@ -113,6 +113,8 @@ class Part:
 # arrangement asks before it uses either, so a part that says nothing gets and gives plain tensors):
 #   takes_scaled_rows  x may come as parts.linear.ScaledRows (rows whose RMSNorm the part's first product
 #                      finishes; ``linear`` and ``gated_linear`` take them as they take a tensor);
+#   leaves_bias        an arrangement whose norms add a bias may set ``leave_bias`` on the part; ``forward`` then leaves
+#                      the bias of its last product out and ``late_bias`` is that bias (or None);
 #   defers_output      ``forward`` takes the keyword ``defer``; with defer=True it may return its last
 #                      product unrun, as a parts.linear.PendingProduct.
 # A norm that says ``fuses_products`` takes a PendingProduct as delta and the keyword ``scaled_ok``
@@ -170,6 +172,74 @@ class Mixer(Part):
         """x: [T, hidden] normalised input.  ``step`` is the StepContext of this batch,
         ``cache`` the view of this run entry's cache slot.  Returns [T, hidden]."""
         raise NotImplementedError
+
+
+class ProjectedMixer(Mixer):
+    """A mixer of the form  out = W_o f(W_in x) (+ b_o)  whose f works on the rows of one stacked projection and writes
+    its own rows, so that several such mixers that read the same x can share both products (``summed_mixers``).
+
+    A kind gives ``hidden_size``, ``segments()`` (name -> extents of the checkpoint tensors stacked in it), ``inner_cols``
+    (columns of f's rows), ``inner_params()`` and ``inner``; ``out_bias`` says whether b_o exists.  Segments whose size is
+    a multiple of 8 come first in the stacked projection and its width is rounded up to such a multiple, so that rows
+    can be read 16 bytes at a time."""
+
+    graph_safe = True
+    leaves_bias = True
+    leave_bias = False
+    out_bias = False
+    inner_cols = 0
+    hidden_size = 0
+
+    def segments(self) -> Dict[str, Tuple[int, ...]]:
+        raise NotImplementedError
+
+    def inner_params(self) -> Dict[str, ParamSpec]:
+        return {}
+
+    def inner(self, x, proj: Dict[str, torch.Tensor], step, cache, writes_cache: bool, y: torch.Tensor, y_scale: float) -> None:
+        """y [T, inner_cols] (rows may lie further apart) = y_scale * f(the segments' columns of the projection)."""
+        raise NotImplementedError
+
+    # ---- what follows is the same for every kind
+
+    @staticmethod
+    def layout(segments: Dict[str, Tuple[int, ...]]):
+        """(segment names in their order in the projection, name -> (first column, columns), width with padding)."""
+        names = sorted(segments, key=lambda n: sum(segments[n]) % 8 != 0)     # (a stable sort)
+        at, where = 0, {}
+        for n in names:
+            where[n] = (at, sum(segments[n]))
+            at += sum(segments[n])
+        return names, where, -(-at // 8) * 8
+
+    def _in_spec(self) -> ParamSpec:
+        segs = self.segments()
+        names, where, width = self.layout(segs)
+        rows = tuple(r for n in names for r in segs[n])
+        return ParamSpec((width, self.hidden_size), rows=rows, pad=width - sum(rows))
+
+    def params(self) -> Dict[str, ParamSpec]:
+        p = {"in.weight": self._in_spec(), "o.weight": ParamSpec((self.hidden_size, self.inner_cols))}
+        if self.out_bias:
+            p["o.bias"] = ParamSpec((self.hidden_size,), role="vector", init="normal")
+        p.update(self.inner_params())
+        return p
+
+    @property
+    def late_bias(self) -> Optional[torch.Tensor]:
+        return self.w_o_bias if self.out_bias and self.leave_bias else None
+
+    def forward(self, x, step, cache, writes_cache):
+        from .linear import linear
+
+        T = x.shape[0]
+        ws, dt = self.rt.workspace, self.rt.dtype
+        _, where, width = self.layout(self.segments())
+        proj = linear(x, self.w_in_weight, None, ws.get("pm.in", (T, width), dt))
+        y = ws.get("pm.y", (T, self.inner_cols), dt)
+        self.inner(x, {n: proj[:, a:a + k] for n, (a, k) in where.items()}, step, cache, writes_cache, y, 1.0)
+        bias = self.w_o_bias if self.out_bias and not self.leave_bias else None
+        return linear(y, self.w_o_weight, bias, ws.get("pm.out", (T, self.hidden_size), dt))
 
 
 class FeedForward(Part):

@@ -19,9 +19,10 @@ by whoever comes next (``delta_scale`` tells the model the factor of what ``run`
    r += delta;  h = norm(r);  r += mixer(h) + ffn(h)        (a layer may have no feed-forward).
 
 "sandwich" puts a norm before and after each sub-block (the feed-forward and its two norms optional):
-   r += delta;  a = norm1(r);  r += norm1b(mixer(a));  [b = norm2(r);  r += norm2b(ffn(b))]
-A sub-block's output travels to the next norm as a ``NormedDelta``, so that the norm after a sub-block, the add and
-the norm before the next sub-block are one kernel.
+   r += delta;  a = norm1(r);  r += m * norm1b(mixer(a));  [b = norm2(r);  r += m * norm2b(ffn(b))]
+(m: a constant, 1 unless given).  A sub-block's output travels to the next norm as a ``NormedDelta``, so that the norm
+after a sub-block, the add and the norm before the next sub-block are one kernel; a part that says ``leaves_bias`` leaves
+the bias of its last product to that kernel too.
 
 Between parts that say they can, an output travels as a product still to run and normalised rows
 as ``ScaledRows`` (parts/linear.py), so that in a step of few rows the norms need no kernel of their
@@ -95,7 +96,8 @@ class SandwichBlock:
     optional = ("ffn_norm", "ffn", "ffn_post_norm")
     takes_pending = True      # delta may be a NormedDelta (or a PendingProduct), and run() returns a NormedDelta
 
-    def __init__(self, mixer_norm, mixer, mixer_post_norm, ffn_norm=None, ffn=None, ffn_post_norm=None):
+    def __init__(self, mixer_norm, mixer, mixer_post_norm, ffn_norm=None, ffn=None, ffn_post_norm=None,
+                 residual_mult: float = 1.0):
         if len({ffn is None, ffn_norm is None, ffn_post_norm is None}) != 1:
             raise ValueError("sandwich: a feed-forward and its two norms come together")
         for n in (mixer_post_norm, ffn_post_norm):
@@ -103,21 +105,27 @@ class SandwichBlock:
                 raise ValueError("sandwich: the norms after a sub-block take plain weights")
         self.mixer_norm, self.mixer, self.mixer_post_norm = mixer_norm, mixer, mixer_post_norm
         self.ffn_norm, self.ffn, self.ffn_post_norm = ffn_norm, ffn, ffn_post_norm
+        self.delta_scale = float(residual_mult)     # the factor of the output that run() hands on
+        for part in (mixer, ffn):
+            if getattr(part, "leaves_bias", False):
+                part.leave_bias = True
 
     @staticmethod
-    def _normed(x, norm, tag):
+    def _normed(x, part, norm, tag):
         out = norm.rt.workspace.get(tag, tuple(x.shape), x.dtype)
-        return NormedDelta(x, norm.w_weight, norm.eps, out)
+        return NormedDelta(x, norm, out, getattr(part, "late_bias", None))
 
-    def run(self, residual, delta, step, cache, writes_cache):
-        a = self.mixer_norm.add_norm(residual, delta, "norm.mixer")
+    def run(self, residual, delta, step, cache, writes_cache, delta_scale=None):
+        """delta_scale: the factor of the incoming delta (the block's own constant unless the model says otherwise)."""
+        scale = self.delta_scale
+        a = self.mixer_norm.add_norm(residual, delta, "norm.mixer", delta_scale=scale if delta_scale is None else delta_scale)
         m = self.mixer.forward(a, step, cache, writes_cache)
-        m = self._normed(m, self.mixer_post_norm, "norm.mixer.post")
+        m = self._normed(m, self.mixer, self.mixer_post_norm, "norm.mixer.post")
         if self.ffn is None:
             return m
-        b = self.ffn_norm.add_norm(residual, m, "norm.ffn")
+        b = self.ffn_norm.add_norm(residual, m, "norm.ffn", delta_scale=scale)
         f = self.ffn.forward(b, step)
-        return self._normed(f, self.ffn_post_norm, "norm.ffn.post")
+        return self._normed(f, self.ffn, self.ffn_post_norm, "norm.ffn.post")
 
 
 @register("arrangement", "parallel")

@@ -28,6 +28,56 @@ from .registry import register
 from .spec import CacheEntry, CacheNeed, ParamSpec, PartSpec
 
 
+def rotation_options(position) -> dict:
+    """What ``native.conv_rope_write`` has to know of a position part that gives frequencies."""
+    if position is None:
+        return {}
+    return {"neighbours": getattr(position, "neighbours", False), "magnitude": getattr(position, "magnitude", 1.0)}
+
+
+def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int], keep_first: int, dtype):
+    """(into how many shares the tensor-core kernel cuts the key tiles of every unit, or 0 for the plain kernel;
+    whether a unit is a token with the query heads of one key head as rows, which steps of single tokens use, or
+    a tile of 64 tokens with one head), for attention over a window that keeps first tokens (or over all keys)."""
+    key = ("window_attention", nh, nkv, dk, dv, window or 0, keep_first)
+    plan = step.plans.get(key)
+    if plan is None:
+        if native.WINDOW_TC and native.window_attention_tc_supports(dk, dv, dtype):
+            longest = min(step.max_ctx_len, window + keep_first) if window else step.max_ctx_len
+            heads_rows = step.max_q_len <= 1 and nh // nkv <= native.WINDOW_TC_ROWS
+            if heads_rows:
+                units = step.num_tokens * nkv
+            elif step.max_q_len <= 1:
+                units = step.num_tokens * nh
+            else:
+                units = (-(-step.num_tokens // native.WINDOW_TC_ROWS) + step.num_seqs - 1) * nh
+            # (two CTAs fit an SM; steps with prompt portions fill it once before their keys are shared out: the
+            # shares cost a pass over 32-bit partial outputs of every row)
+            plan = (native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 else 1,
+                                                  min_share=128), heads_rows)
+        else:
+            plan = (0, False)
+        step.plans[key] = plan
+    return plan
+
+
+def attend(plan, ws, o, q, cache, step, nh: int, nkv: int, dk: int, dv: int, scale: float, softcap: float,
+           window: Optional[int], keep_first: int, **extras) -> None:
+    """Runs the attention of ``plan`` (``window_plan``) over the cache's pages; extras: sink, gate, out_scale."""
+    bt = step.block_tables[cache.group]
+    nsplit, heads_rows = plan
+    if nsplit:
+        scratch = None
+        if nsplit > 1:
+            scratch = ws.get("cwa.splits", (native.attention_mixed_scratch_elems(q.shape[0], nh, dv, nsplit),), torch.float32)
+        native.window_attention_tc(o, q, cache.k_pages, cache.v_pages, bt, step.positions, step.seq_of_token,
+                                   step.cu_q, step.num_seqs, nh, nkv, dk, dv, scale, softcap, window or 0, keep_first,
+                                   nsplit, scratch, heads_rows, **extras)
+    else:
+        native.window_attention(o, q, cache.k_pages, cache.v_pages, bt, step.positions, step.seq_of_token, nh, nkv,
+                                dk, dv, scale, softcap, window or 0, keep_first, **extras)
+
+
 @register("mixer", "conv_window_attention")
 class ConvWindowAttention(Mixer):
     graph_safe = True
@@ -76,26 +126,7 @@ class ConvWindowAttention(Mixer):
         whether a unit is a token with the query heads of one key head as rows, which steps of single tokens use, or
         a tile of 64 tokens with one head).  Where the units do not fill the device (decoding, short portions) their
         keys are shared out, in shares of at least 128."""
-        key = ("conv_window_attention", self.nh, self.nkv, self.dk, self.dv, self.window or 0, self.keep_first)
-        plan = step.plans.get(key)
-        if plan is None:
-            if native.WINDOW_TC and native.window_attention_tc_supports(self.dk, self.dv, self.rt.dtype):
-                longest = min(step.max_ctx_len, self.window + self.keep_first) if self.window else step.max_ctx_len
-                heads_rows = step.max_q_len <= 1 and self.nh // self.nkv <= native.WINDOW_TC_ROWS
-                if heads_rows:
-                    units = step.num_tokens * self.nkv
-                elif step.max_q_len <= 1:
-                    units = step.num_tokens * self.nh
-                else:
-                    units = (-(-step.num_tokens // native.WINDOW_TC_ROWS) + step.num_seqs - 1) * self.nh
-                # (two CTAs fit an SM; steps with prompt portions fill it once before their keys are shared out: the
-                # shares cost a pass over 32-bit partial outputs of every row)
-                plan = (native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 else 1,
-                                                      min_share=128), heads_rows)
-            else:
-                plan = (0, False)
-            step.plans[key] = plan
-        return plan
+        return window_plan(step, self.nh, self.nkv, self.dk, self.dv, self.window, self.keep_first, self.rt.dtype)
 
     def forward(self, x, step, cache, writes_cache, defer=False):
         T = x.shape[0]
@@ -111,21 +142,12 @@ class ConvWindowAttention(Mixer):
                                self.position.rotary_dim if self.position is not None else 0, step.positions,
                                step.seq_of_token, step.cu_q, step.state_slots, bt, cache.page_size,
                                cache.k_pages if writes_cache else None, cache.v_pages if writes_cache else None,
-                               step.status)
+                               step.status, **rotation_options(self.position))
         if conv_state is not None and writes_cache:
             native.conv_state_update(conv_state, qkv, step.cu_q, step.state_slots, step.num_seqs)
         o = ws.get("cwa.o", (T, nh * dv), dt)
-        nsplit, heads_rows = self.launch_plan(step)
-        if nsplit:
-            scratch = None
-            if nsplit > 1:
-                scratch = ws.get("cwa.splits", (native.attention_mixed_scratch_elems(T, nh, dv, nsplit),), torch.float32)
-            native.window_attention_tc(o, q, cache.k_pages, cache.v_pages, bt, step.positions, step.seq_of_token,
-                                       step.cu_q, step.num_seqs, nh, nkv, dk, dv, self.scale, self.softcap,
-                                       self.window or 0, self.keep_first, nsplit, scratch, heads_rows)
-        else:
-            native.window_attention(o, q, cache.k_pages, cache.v_pages, bt, step.positions, step.seq_of_token, nh, nkv,
-                                    dk, dv, self.scale, self.softcap, self.window or 0, self.keep_first)
+        attend(self.launch_plan(step), ws, o, q, cache, step, nh, nkv, dk, dv, self.scale, self.softcap, self.window,
+               self.keep_first)
         out = ws.get("cwa.out", (T, self.hidden_size), dt)
         if defer and may_defer(o, self.w_o_weight):
             return PendingProduct(o, self.w_o_weight, None, out)

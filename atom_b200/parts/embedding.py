@@ -81,8 +81,10 @@ class StepVectors(Part):
 class LMHead(Part):
     graph_safe = True
 
-    def __init__(self, vocab_size: int, hidden_size: int, tied: bool):
+    def __init__(self, vocab_size: int, hidden_size: int, tied: bool, scale: float = 1.0, softcap: float = 0.0):
+        """scale: factor on the logits; softcap: then cap * tanh(logits / cap) (0: none), both in 32-bit."""
         self.vocab_size, self.hidden_size, self.tied = vocab_size, hidden_size, tied
+        self.scale, self.softcap = float(scale), float(softcap or 0.0)
 
     def params(self) -> Dict[str, ParamSpec]:
         if self.tied:
@@ -97,4 +99,7 @@ class LMHead(Part):
         tensor the caller may keep."""
         if out is None:
             out = torch.empty((x.shape[0], self.vocab_size), dtype=torch.float32, device=x.device)
-        return linear(x, self.w_weight, None, out[: x.shape[0]])
+        out = linear(x, self.w_weight, None, out[: x.shape[0]])
+        if self.scale != 1.0 or self.softcap:
+            native.scale_softcap_(out, self.scale, self.softcap)
+        return out

@@ -56,6 +56,8 @@ class LatentAttention(Mixer):
         self.window, self.cache_window = window, cache_window
         self.sink, self.gate, self.borrows = sink, gate, reads_cache_of_other
         self.position = registry.build("position", position)
+        if getattr(self.position, "neighbours", False):
+            raise ValueError("latent_attention rotates half-split pairs")
         if self.position.rotary_dim > rot_dim:
             raise ValueError(f"latent_attention: {self.position.rotary_dim} rotated numbers in a part of {rot_dim}")
         if window is not None and (cache_window is not None and cache_window < window):

@@ -49,17 +49,16 @@ class ScaledRows:
 
 
 class NormedDelta:
-    """A sub-block's output x that enters the residual stream through an RMSNorm of its own, rmsnorm(x; weight),
-    described but not yet normalised: the norm that reads the stream next does both in one kernel; whoever cannot
-    calls ``run()`` and has the normalised rows."""
-    __slots__ = ("x", "weight", "eps", "out")
+    """A sub-block's output x (+ x_bias) that enters the residual stream through a norm of its own, described but not
+    yet normalised: a norm of the same kind that reads the stream next does both in one kernel; whoever cannot calls
+    ``run()`` and has the normalised rows."""
+    __slots__ = ("x", "norm", "out", "x_bias")
 
-    def __init__(self, x, weight, eps, out):
-        self.x, self.weight, self.eps, self.out = x, weight, eps, out
+    def __init__(self, x, norm, out, x_bias=None):
+        self.x, self.norm, self.out, self.x_bias = x, norm, out, x_bias
 
     def run(self) -> torch.Tensor:
-        native.rmsnorm(self.out, self.x, self.weight, self.eps)
-        return self.out
+        return self.norm.normalise(self.x, self.out, self.x_bias)
 
 
 def resolve(delta):
@@ -124,21 +123,27 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], 
     return out
 
 
-def gated_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, scratch, act: str = "silu") -> torch.Tensor:
-    """out[M, I] = act(x W_gate^T) * (x W_up^T) for weight [2I, K] = [gate ; up], act "silu" or "gelu_tanh".  Few
+def gated_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, scratch, act: str = "silu",
+                 limit: float = 0.0) -> torch.Tensor:
+    """out[M, I] = act(x W_gate^T) * (x W_up^T) for weight [2I, K] = [gate ; up], act "silu", "gelu_tanh" or "clamped"
+    (g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1)).  Few
     rows, and long portions in bf16 (``pairs_pay``): one kernel, the activation fused into the product.  Else
     the product into ``scratch(M, 2I)`` and the activation kernel."""
     M, K = x.shape
     I = weight.shape[0] // 2
     if isinstance(x, ScaledRows):
-        native.gemm_rows(x.x, weight, out, gated=True, ssq_in=x.ssq, norm_size=x.size, norm_eps=x.eps, act=act)
+        native.gemm_rows(x.x, weight, out, gated=True, ssq_in=x.ssq, norm_size=x.size, norm_eps=x.eps, act=act,
+                         limit=limit)
         return out
     if x.dtype == torch.bfloat16 and streams(M, I, K, x.stride(0), gated=True):
-        native.gemm_rows(x, weight, out, gated=True, act=act)
+        native.gemm_rows(x, weight, out, gated=True, act=act, limit=limit)
         return out
     if x.dtype == torch.bfloat16 and pairs_pay(M, I, K, x.stride(0), out.stride(0)):
-        native.gemm_pairs(x, weight, out, gated=True, act=act)
+        native.gemm_pairs(x, weight, out, gated=True, act=act, limit=limit)
         return out
     gu = linear(x, weight, None, scratch(M, 2 * I))
-    (native.gelu_mul if act == "gelu_tanh" else native.silu_mul)(out, gu)
+    if act == "clamped":
+        native.clamped_mul(out, gu, limit)
+    else:
+        (native.gelu_mul if act == "gelu_tanh" else native.silu_mul)(out, gu)
     return out

@@ -1,4 +1,4 @@
-"""RMSNorm fused with the residual add (atom/model_ops/layernorm.py:57-75):
+"""Norms, fused with the residual add.  RMSNorm (atom/model_ops/layernorm.py:57-75):
    r = x + r;  y = r * rsqrt(mean(r^2) + eps) * w,  computed in 32-bit on a 32-bit residual.
 
 In a step of few rows the norm can do without a kernel of its own.  If what is to be added comes as
@@ -44,13 +44,14 @@ class RMSNorm(Norm):
         """delta_scale: what is added to the residual is delta_scale * delta (a design whose sub-blocks enter the
         residual stream times a constant); the product's residual epilogue takes the factor too."""
         if isinstance(delta, NormedDelta):
-            # what is added passes a norm of its own first: both norms and the add in one kernel
-            if delta_scale != 1.0:
-                raise ValueError("a normalised delta enters the residual stream as it is")
-            n = residual.shape[0] if rows is None else (rows.numel() if n_rows is None else n_rows)
-            out = self.rt.workspace.get(tag, (n, self.size), self.rt.dtype)
-            native.normed_add_rmsnorm(out, residual, delta.x, delta.weight, delta.eps, self.w_weight, self.eps, rows, n)
-            return out
+            if isinstance(delta.norm, RMSNorm) and delta.x_bias is None:
+                # what is added passes a norm of its own first: both norms and the add in one kernel
+                n = residual.shape[0] if rows is None else (rows.numel() if n_rows is None else n_rows)
+                out = self.rt.workspace.get(tag, (n, self.size), self.rt.dtype)
+                native.normed_add_rmsnorm(out, residual, delta.x, delta.norm.w_weight, delta.norm.eps, self.w_weight,
+                                          self.eps, rows, n, delta_scale)
+                return out
+            delta = delta.run()
         if isinstance(delta, PendingProduct):
             if scaled_ok and rows is None and self._folds(residual, delta):
                 M, ws = residual.shape[0], self.rt.workspace
@@ -65,6 +66,13 @@ class RMSNorm(Norm):
         native.add_rmsnorm(out, residual, delta, self.w_weight, self.eps, rows, n, delta_scale)
         return out
 
+    def normalise(self, x, out, x_bias=None):
+        """out = norm(x (+ x_bias)) of rows that are no part of the stream."""
+        if x_bias is not None:
+            native.add_bias(x, x_bias)
+        native.rmsnorm(out, x, self.w_weight, self.eps)
+        return out
+
     def _folds(self, residual, p: PendingProduct) -> bool:
         """The pending product can run with the residual epilogue, and a product over this norm's
         ``size`` columns can take the rows' factors."""
@@ -73,3 +81,35 @@ class RMSNorm(Norm):
                 and residual.dtype == torch.float32 and residual.is_contiguous()
                 and p.weight.shape[0] == self.size and _linear.may_defer(p.x, p.weight)
                 and M <= native.ROWS_M and native.gemm_rows_supports(M, 1, self.size, self.size))
+
+
+@register("norm", "layernorm")
+class LayerNorm(Norm):
+    """(x - mean) / sqrt(variance + eps) * w + b, with the variance as the mean of squared deviations; the add in front
+    of it, and the norm that what is added passes first (a ``NormedDelta`` with a LayerNorm), are the same kernel."""
+    graph_safe = True
+    fuses_products = True
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = size, eps
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.size,), role="vector", init="norm"),
+                "bias": ParamSpec((self.size,), role="vector", init="normal")}
+
+    def add_norm(self, residual, delta, tag, rows=None, n_rows=None, scaled_ok=False, delta_scale=1.0):
+        """delta_scale: what is added to the residual is delta_scale * delta (after the delta's own norm)."""
+        own, x_bias = None, None
+        if isinstance(delta, NormedDelta) and isinstance(delta.norm, LayerNorm):
+            own, x_bias = (delta.norm.w_weight, delta.norm.w_bias, delta.norm.eps), delta.x_bias
+            delta = delta.x
+        delta = _linear.resolve(delta)
+        n = residual.shape[0] if rows is None else (rows.numel() if n_rows is None else n_rows)
+        out = self.rt.workspace.get(tag, (n, self.size), self.rt.dtype)
+        native.add_layernorm(out, residual, delta, self.w_weight, self.w_bias, self.eps, rows, n, delta_scale, x_bias, own)
+        return out
+
+    def normalise(self, x, out, x_bias=None):
+        """out = norm(x (+ x_bias)) of rows that are no part of the stream."""
+        native.layernorm(out, x, self.w_weight, self.w_bias, self.eps, x_bias)
+        return out

@@ -26,6 +26,7 @@ import torch
 from .. import native
 from . import registry
 from .base import Mixer
+from .conv_attention import rotation_options
 from .linear import PendingProduct, linear, may_defer
 from .registry import register
 from .spec import CacheEntry, CacheNeed, ParamSpec, PartSpec
@@ -125,7 +126,7 @@ class PooledWindowAttention(Mixer):
         native.conv_rope_write(q, proj, nh, nkv, dk, dv, None, None, freq, pos.rotary_dim if freq is not None else 0,
                                step.positions, step.seq_of_token, step.cu_q, step.state_slots, bt, cache.page_size,
                                cache.k_pages if writes_cache else None, cache.v_pages if writes_cache else None,
-                               step.status)
+                               step.status, **rotation_options(pos))
         pk = pv = pool_bt = None
         if self.pool is not None:
             pk, pv = cache.block_pages["pk"], cache.block_pages["pv"]

@@ -60,16 +60,16 @@ def yarn_frequencies(rotary_dim: int, theta: float, factor: float, original: flo
 
 @register("position", "rope_yarn")
 class RotaryYarn(PositionEncoding):
-    """Half-split rotary pairs whose angle is computed in the kernel, position * frequency in 32-bit, from a vector
+    """Rotary pairs, half-split (i, i + dims/2) or with ``neighbours`` interleaved (2i, 2i + 1), whose angle is computed in the kernel, position * frequency in 32-bit, from a vector
     of frequencies (so no table bounds the positions), with YaRN's stretch when ``scaling`` is given as
     {factor, original, fast, slow}.  A mixer asks for ``frequencies(rt)`` and ``magnitude`` and hands them to its
     kernel; ``table`` gives None."""
     graph_safe = True
 
-    def __init__(self, rotary_dim: int, theta: float, scaling: Optional[dict] = None):
+    def __init__(self, rotary_dim: int, theta: float, scaling: Optional[dict] = None, neighbours: bool = False):
         if rotary_dim % 2:
             raise ValueError("rotary_dim must be even")
-        self.rotary_dim, self.theta = rotary_dim, float(theta)
+        self.rotary_dim, self.theta, self.neighbours = rotary_dim, float(theta), bool(neighbours)
         if scaling:
             self._f, self.magnitude = yarn_frequencies(rotary_dim, self.theta, float(scaling["factor"]),
                                                        float(scaling["original"]), float(scaling["fast"]),

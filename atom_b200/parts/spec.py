@@ -24,6 +24,7 @@ class ParamSpec:
     rows   when the parameter is several checkpoint tensors stacked along one axis, their extents
            along it.
     stack_dim   that axis (0: rows under one another, as q/k/v; 1: side by side).
+    pad    rows of zeros behind the stacked tensors along that axis (a product's width rounded up); in no checkpoint.
     members_lack_axis   the stacked checkpoint tensors have no such axis of their own (each is one
            slice: vectors [n] stacked into [m, n]); every extent in ``rows`` is then 1.
     """
@@ -34,6 +35,7 @@ class ParamSpec:
     rows: Optional[Tuple[int, ...]] = None
     stack_dim: int = 0
     members_lack_axis: bool = False
+    pad: int = 0
 
 
 @dataclass(frozen=True)

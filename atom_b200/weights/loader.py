@@ -56,8 +56,8 @@ def expected_tensors(model: Model) -> Dict[str, Tuple[str, str, int, Tuple[int, 
             d = ps.stack_dim
             if not 0 <= d < len(ps.shape):
                 raise ValueError(f"{path}.{name}: stack_dim {d} for a tensor of shape {ps.shape}")
-            rows = ps.rows if ps.rows is not None else (ps.shape[d],)
-            if len(rows) != len(srcs) or sum(rows) != ps.shape[d]:
+            rows = ps.rows if ps.rows is not None else (ps.shape[d] - ps.pad,)
+            if len(rows) != len(srcs) or sum(rows) + ps.pad != ps.shape[d]:
                 raise ValueError(f"{path}.{name}: {len(srcs)} source tensors for the split {rows} of axis {d}")
             if ps.members_lack_axis and any(r != 1 for r in rows):
                 raise ValueError(f"{path}.{name}: members without the stacked axis are one slice each, not {rows}")
@@ -139,6 +139,8 @@ def load_weights(model: Model, model_dir: str, compute: torch.dtype, device) -> 
     for key, ps in specs.items():
         dt = _target_dtype(ps, stored_dtypes[key], compute)
         out[key] = torch.empty(ps.shape, dtype=dt, device=device)
+        if ps.pad:
+            out[key].narrow(ps.stack_dim, ps.shape[ps.stack_dim] - ps.pad, ps.pad).zero_()
     for n, (key, _, off, shape, ps) in want.items():
         t = where[n].get_tensor(n)
         dst = out[key]
