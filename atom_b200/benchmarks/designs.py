@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of the Nurinex, Mugulorn, Simivik and Kibotar designs beside Qwen3 dense at equal sizes.
+"""Prefill and decode throughput of the Nurinex, Mugulorn, Simivik, Kibotar and Vudezen designs beside Qwen3 dense at equal
+sizes.
 
     python -m atom_b200.benchmarks.designs [--sizes 1024x8,2048x16] [--layers 4] [--prefill 2048]
-                                           [--batch 8] [--context 2048] [--kernels] [--only qwen3,kibotar]
+                                           [--batch 8] [--context 2048] [--kernels] [--only qwen3,vudezen]
 
 For each size (width x attention heads; head size 128, four query heads to a kv head, feed-forward three
 times the width, vocabulary 32768) two engines are built with random bfloat16 weights and the same number
@@ -18,7 +19,12 @@ layers (norms before and after every sub-block, a token shift before every mixer
 attention through a latent of width / 4 (the same heads, 128 numbers per key and value, a gate per head), attention
 over a window of 1024 and pooled blocks of 64 (the same heads, all 128 numbers rotated with stretched frequencies, a
 sink, mixed weights, an output gate, biases), which runs twice in a row, and gated linear attention (the same heads,
-128 numbers per key and value, a decay of rank 64), so that as many layers run as the other designs have.  Measured on the device with CUDA events: one prompt of ``--prefill`` tokens through
+128 numbers per key and value, a decay of rank 64), so that as many layers run as the other designs have; and Vudezen,
+whose layers (layer norms before and after every sub-block) are in turn attention over a window of 1024 (the same heads,
+all 128 numbers rotated in neighbouring pairs, a sink and a gate per head, biases) beside a state-space recurrence
+(width / 64 heads of 64 numbers, a state of 128, 4 groups, a convolution of 4 taps), and attention over all earlier
+tokens (the same heads, YaRN, blended values), all with 16 experts of the width's size and 4 identity experts in 4
+groups, of which 2 groups are kept and 2 experts used, beside a shared one.  Measured on the device with CUDA events: one prompt of ``--prefill`` tokens through
 one step, and decode steps of ``--batch`` requests whose caches hold ``--context`` tokens (captured graphs,
 as the engine runs them).  With ``--kernels`` the kernels of one prefill step and of one decode step are
 listed with their summed device time (the engine's profiler hook), which is what the per-kernel rooflines
@@ -106,6 +112,21 @@ def kibotar_config(width: int, heads: int, layers: int) -> dict:
     return {"architecture": "Kibotar", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5},
             "embedding": {"scale": 1.0, "bigram": {"buckets": 4093, "mul_prev": 257, "mul_cur": 11}},
             "loop": {"start": 1, "stop": 2, "times": 2}, "layers": [kinds[i % 3] for i in range(unique)]}
+
+
+def vudezen_config(width: int, heads: int, layers: int) -> dict:
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    left = dict(att, rot={"base": 250000.0, "dims": 128}, mask={"size": 1024})
+    right = {"heads": width // 64, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}
+    pair = {"left": left, "left_scale": 0.8, "right": right, "right_scale": 0.6}
+    full = dict(att, v_mix=True, rot={"base": 1000000.0, "dims": 128,
+                                      "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    moe = {"kind": "moe", "router": {"experts": 16, "identity": 4, "top": 2, "scale": 1.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": width, "limit": 7.0}, "shared": {"ff": width, "limit": 7.0}}
+    kinds = [("parallel", pair), ("attention", full)]
+    return {"architecture": "Vudezen", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "logit_scale": 0.5, "logit_softcap": 50.0,
+            "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in (kinds[i % 2] for i in range(layers))]}
 
 
 def _runner(cfg: dict, pages: int, max_len: int, batch: int):
@@ -225,10 +246,10 @@ def main(argv=None) -> int:
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=2048)
     ap.add_argument("--kernels", action="store_true", help="list the kernels of one prefill and one decode step")
-    ap.add_argument("--only", default="qwen3,nurinex,mugulorn,simivik,kibotar", help="the designs to measure, comma-separated")
+    ap.add_argument("--only", default="qwen3,nurinex,mugulorn,simivik,kibotar,vudezen", help="the designs to measure, comma-separated")
     args = ap.parse_args(argv)
     configs = {"qwen3": qwen3_config, "nurinex": nurinex_config, "mugulorn": mugulorn_config, "simivik": simivik_config,
-               "kibotar": kibotar_config}
+               "kibotar": kibotar_config, "vudezen": vudezen_config}
     chosen = [d for d in args.only.split(",") if d]
     if any(d not in configs for d in chosen):
         ap.error(f"--only takes {sorted(configs)}")
