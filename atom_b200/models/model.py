@@ -130,10 +130,10 @@ class Model:
                 self.stream_steps.add(residual, e.add_step)     # (sums commute: the pending delta is added by the next norm)
             if not getattr(block, "takes_pending", False):
                 delta = resolve(delta)      # (a block may hand its last product on unrun)
-            if hasattr(block, "delta_scale"):
+            if delta is not None and (scale != 1.0 or getattr(block, "delta_scale", 1.0) != 1.0):
+                if not hasattr(block, "delta_scale"):
+                    raise ValueError("a block that scales its output is followed by one that cannot take the factor")
                 delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache, delta_scale=scale)
-            elif scale != 1.0 and delta is not None:
-                raise ValueError("a block that scales its output is followed by one that cannot take the factor")
             else:
                 delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache)
             scale = getattr(block, "delta_scale", 1.0)
