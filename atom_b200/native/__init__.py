@@ -70,6 +70,10 @@ _SIGNATURES = {
     "atom_ssm_conv": [_vp, _vp, _i, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "atom_ssm_step": [_vp, _vp, _vp, _i, _i64, _vp, _vp, _i, _i, _i, _vp],
     "atom_ssm_scan": [_vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "atom_ssm_tc_supports": [_i, _i],
+    "atom_ssm_tc_chunk": [],
+    "atom_ssm_tc": [_i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "atom_ssm_prefix": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "atom_ssm_gate_norm": [_vp, _i, _i64, _vp, _vp, _i64, _vp, _i, _i, _i, _i, _f, _f, _vp, _vp],
     "atom_head_gate": [_vp, _vp, _i, _i64, _i, _i, _i, _vp],
     "atom_gla_supports": [_i, _i],
@@ -1618,19 +1622,22 @@ def ssm_supports(N: int, P: int) -> bool:
     return bool(lib().atom_ssm_supports(N, P))
 
 
-SSM_RUN = 64        # rows per run of the scan in steps of more rows than this
+SSM_RUN = 64        # rows per run of the scan in steps that bring more rows of a request than this
+SSM_TC = True       # False: the plain scan also where the tensor-core kernels take the sizes (measurements, tests)
 
 
-def ssm_run(T: int) -> int:
-    """Rows per run for a step of T rows (0: every request is walked once)."""
+def ssm_run(T: int, N: int, P: int, dtype: torch.dtype):
+    """(rows per run for a step whose longest portion may be T rows, 0: every request is walked once; whether the runs'
+    sums and outputs run on the tensor cores)."""
     if T <= SSM_RUN:
-        return 0
-    return SSM_RUN if T <= 64 * SSM_RUN else -(-T // 64)
+        return 0, False
+    if SSM_TC and dtype == torch.bfloat16 and lib().atom_ssm_tc_supports(N, P):
+        return int(lib().atom_ssm_tc_chunk()), True
+    return (SSM_RUN if T <= 64 * SSM_RUN else -(-T // 64)), False
 
 
-def ssm_scratch_elems(T: int, num_seqs: int, H: int, N: int, P: int):
-    """(floats of the runs' sums, floats of the runs' decays)."""
-    run = ssm_run(T)
+def ssm_scratch_elems(T: int, num_seqs: int, H: int, N: int, P: int, run: int):
+    """(floats of the runs' sums, floats of the runs' decays) of a step of T rows in runs of ``run``."""
     if run == 0:
         return 0, 0
     slots = -(-T // run) + num_seqs
@@ -1669,20 +1676,31 @@ def ssm_step(dt: torch.Tensor, la: torch.Tensor, raw: torch.Tensor, dt_bias: tor
 
 def ssm_scan(out: torch.Tensor, u: torch.Tensor, dt: torch.Tensor, la: torch.Tensor, D: torch.Tensor, state: torch.Tensor,
              scratch_b: Optional[torch.Tensor], scratch_a: Optional[torch.Tensor], cu_q: torch.Tensor,
-             state_slots: torch.Tensor, num_seqs: int, H: int, G: int, N: int, P: int, write_state: bool = True) -> None:
+             state_slots: torch.Tensor, num_seqs: int, H: int, G: int, N: int, P: int, write_state: bool = True,
+             longest: Optional[int] = None) -> None:
     """out[t] (float32 [T, H P]) = S_t^T C_t + D x_t with S_t = exp(la_t) S_(t-1) + dt_t B_t x_t^T per head, over every
-    request's rows; u rows are [x (H P) | B (G N) | C (G N)]; state [slots, H, N, P] float32."""
+    request's rows; u rows are [x (H P) | B (G N) | C (G N)]; state [slots, H, N, P] float32.  longest: the most rows that
+    one request can have in the step (all of them, unless given); it decides the form (``ssm_run``)."""
     _cuda(out, u, dt, la, D, state, scratch_b, scratch_a, cu_q, state_slots)
     T = u.shape[0]
-    run = ssm_run(T)
+    run, tc = ssm_run(T if longest is None else min(T, longest), N, P, u.dtype)
     assert out.dtype == torch.float32 and out.is_contiguous() and out.shape == (T, H * P)
     assert u.is_contiguous() and u.shape == (T, H * P + 2 * G * N) and D.numel() == H
     assert dt.shape == la.shape == (T, H) and dt.is_contiguous() and la.is_contiguous()
     assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, P)
     if run:
-        nb, na = ssm_scratch_elems(T, num_seqs, H, N, P)
+        nb, na = ssm_scratch_elems(T, num_seqs, H, N, P, run)
         assert scratch_b is not None and scratch_a is not None and scratch_b.dtype == scratch_a.dtype == torch.float32
         assert scratch_b.numel() >= nb and scratch_a.numel() >= na
+    if tc:
+        assert D.dtype == torch.float32
+        args = (out.data_ptr(), u.data_ptr(), dt.data_ptr(), la.data_ptr(), D.data_ptr(), scratch_b.data_ptr(),
+                scratch_a.data_ptr(), cu_q.data_ptr(), num_seqs, T, H, G, N, P, _stream())
+        _check(lib().atom_ssm_tc(0, *args), "ssm_tc sums")
+        _check(lib().atom_ssm_prefix(state.data_ptr(), scratch_b.data_ptr(), scratch_a.data_ptr(), cu_q.data_ptr(),
+                                     state_slots.data_ptr(), num_seqs, H, N, P, run, int(write_state), _stream()), "ssm_prefix")
+        _check(lib().atom_ssm_tc(1, *args), "ssm_tc outputs")
+        return
     _check(lib().atom_ssm_scan(out.data_ptr(), u.data_ptr(), dtype_code(u.dtype), dt.data_ptr(), la.data_ptr(), D.data_ptr(),
                                dtype_code(D.dtype), state.data_ptr(), _ptr(scratch_b) if run else None,
                                _ptr(scratch_a) if run else None, cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, H,

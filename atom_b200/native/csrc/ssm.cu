@@ -19,6 +19,7 @@
 //           slot the state after the step
 //   mode 2  every run from its beginning: the outputs
 // and a step of few rows walks each request once (mode 0: slot in, outputs, slot out).
+// (ssm_tc.cu: the runs' sums and outputs on the tensor cores, for bfloat16.)
 #include "common.cuh"
 
 namespace atom {
@@ -449,6 +450,17 @@ ATOM_EXPORT int atom_ssm_scan(float* out, const void* u, int dtype, const float*
     return atom::ssm_scan_dispatch<__nv_bfloat16>(out, (const __nv_bfloat16*)u, dt, la, D, d_dtype, state, sB, sA, cu_q,
                                                   state_slots, num_seqs, T, H, G, N, P, run, write_state, stream);
   return ATOM_ERR_ARG;
+}
+
+// The middle of the three launches over runs: ssm_prefix_kernel alone (ssm_tc.cu has the other two).
+ATOM_EXPORT int atom_ssm_prefix(float* state, float* sB, const float* sA, const int* cu_q, const int* state_slots,
+                                int num_seqs, int H, int N, int P, int run, int write_state, cudaStream_t stream) {
+  if (num_seqs <= 0) return ATOM_OK;
+  if (H <= 0 || H > 65535 || N <= 0 || P <= 0 || run <= 0 || num_seqs > 65535) return ATOM_ERR_ARG;
+  const int eb = (N * P + 255) / 256;
+  atom::launch_pdl(atom::ssm_prefix_kernel, dim3(num_seqs, H, eb > 64 ? 64 : eb), dim3(256), 0, stream, state, sB, sA, cu_q,
+                   state_slots, H, N * P, run, write_state);
+  return atom::check_launch();
 }
 
 ATOM_EXPORT int atom_ssm_gate_norm(void* out, int dtype, int64_t ldo, const float* y, const void* z, int64_t ldz,

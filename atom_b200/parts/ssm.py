@@ -56,6 +56,9 @@ class StateSpace(ProjectedMixer):
             states += (CacheEntry("conv", (self.taps - 1, self.channels), "compute"),)
         return CacheNeed("state", states=states)
 
+    def after_load(self) -> None:
+        self._D = self.w_D.float().contiguous()
+
     def inner(self, x, proj, step, cache, writes_cache, y, y_scale):
         T = y.shape[0]
         ws, dt_ = self.rt.workspace, self.rt.dtype
@@ -68,9 +71,10 @@ class StateSpace(ProjectedMixer):
         la = ws.get("ssm.la", (T, H), torch.float32)
         native.ssm_step(dt, la, rows[:, I + C:], self.w_dt_bias, self.w_A_log)
         o = ws.get("ssm.o", (T, I), torch.float32)
-        nb, na = native.ssm_scratch_elems(T, step.num_seqs, H, N, P)
+        run, _ = native.ssm_run(min(T, step.max_q_len), N, P, dt_)
+        nb, na = native.ssm_scratch_elems(T, step.num_seqs, H, N, P, run)
         sb = ws.get("ssm.runs", (nb,), torch.float32) if nb else None
         sa = ws.get("ssm.run_decays", (na,), torch.float32) if na else None
-        native.ssm_scan(o, u, dt, la, self.w_D, cache.states["S"], sb, sa, step.cu_q, step.state_slots, step.num_seqs,
-                        H, G, N, P, writes_cache)
+        native.ssm_scan(o, u, dt, la, self._D, cache.states["S"], sb, sa, step.cu_q, step.state_slots, step.num_seqs,
+                        H, G, N, P, writes_cache, step.max_q_len)
         native.ssm_gate_norm(y, o, rows[:, :I], self.w_norm, self.norm_groups, self.norm_eps, y_scale, step.seq_of_token)
