@@ -141,6 +141,9 @@ _SIGNATURES = {
     "atom_gemm_rows_grid": [],
     "atom_gemm_rows_supports": [_i, _i, _i, _i64],
     "atom_gemm_pairs": [_vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _f, _vp, _vp],
+    "atom_gemm_pairs_grouped": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp],
+    "atom_gemm_pairs_grouped_supports": [_i, _i, _i, _i],
+    "atom_moe_gather": [_vp, _vp, _i64, _vp, _i, _vp, _vp, _i, _i, _vp],
     "atom_gemm_pairs_resident": [],
     "atom_gemm_pairs_supports": [_i, _i, _i, _i64, _i64],
     "atom_set_option": [_i, _i],
@@ -1258,6 +1261,41 @@ def gemm_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gated: bool 
     _check(lib().atom_gemm_pairs(x.data_ptr(), x.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), M, N, K,
                                  GATE_ACTS[act] if gated else 0, float(limit), error_flag(x.device).data_ptr(), _stream()),
            "gemm_pairs")
+
+
+MOE_PAIRS_ROWS = 64     # rows per expert (on average, if all were used) from which the experts' products run on tcgen05 (0: never)
+
+
+def moe_pairs_pay(R: int, E: int, N: int, K: int, dtype: torch.dtype) -> bool:
+    """Whether the products of E experts over up to R sorted rows, N outputs, run on ``gemm_pairs_grouped``."""
+    return (MOE_PAIRS_ROWS > 0 and MOE_TC and dtype == torch.bfloat16 and R >= MOE_PAIRS_ROWS * E
+            and bool(lib().atom_gemm_pairs_grouped_supports(R, E, N, K)) and gemm_pairs_resident() > 0)
+
+
+def gemm_pairs_grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offsets: torch.Tensor, gated: bool = False,
+                       act: str = "silu", limit: float = 0.0) -> None:
+    """out[r] = x[r] w[e]^T for the rows offsets[e] <= r < offsets[e + 1] of every expert e on tcgen05; x [R, K], out
+    [R, N] dense, w [E, N or 2 N, K]; ``gated``: w[e] = [gate ; up], out = act (csrc/gemm_pairs.cu).  The host need not
+    know the offsets; rows behind the last expert's stay as they are."""
+    R, N = out.shape
+    E, K = w.shape[0], w.shape[2]
+    _cuda(x, w, out, offsets)
+    assert x.dtype == w.dtype == out.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
+    assert x.shape == (R, K) and w.shape[1] == (2 * N if gated else N) and offsets.dtype == torch.int32 and offsets.numel() >= E + 1
+    _check(lib().atom_gemm_pairs_grouped(x.data_ptr(), w.data_ptr(), out.data_ptr(), offsets.data_ptr(), R, E, N, K,
+                                         GATE_ACTS[act] if gated else 0, float(limit), error_flag(x.device).data_ptr(),
+                                         _stream()), "gemm_pairs_grouped")
+
+
+def moe_gather(out: torch.Tensor, x: torch.Tensor, offsets: torch.Tensor, E: int, row_token: torch.Tensor,
+               row_w: Optional[torch.Tensor] = None) -> None:
+    """out[r] = (row_w[r] *) x[row_token[r]] for the rows r < offsets[E]; bfloat16, rows of a multiple of 8 numbers."""
+    _cuda(out, x, offsets, row_token, row_w)
+    R, n = out.shape
+    assert out.dtype == x.dtype == torch.bfloat16 and out.is_contiguous() and x.stride(1) == 1 and x.shape[1] == n
+    assert row_token.numel() >= R and (row_w is None or (row_w.dtype == torch.float32 and row_w.numel() >= R))
+    _check(lib().atom_moe_gather(out.data_ptr(), x.data_ptr(), x.stride(0), offsets.data_ptr(), E, row_token.data_ptr(),
+                                 _ptr(row_w), R, n, _stream()), "moe_gather")
 
 
 def add_bias(out: torch.Tensor, bias: torch.Tensor) -> None:

@@ -25,6 +25,12 @@
 // one tile, so the MMAs of a tile wait until the epilogue of the one before has read the sums (a gated
 // tile's outputs fit in registers as bf16, so its stores come after that); the loads do not wait.
 // All waits are bounded (tma.cuh); tensor memory is freed on every path.
+//
+// Grouped form (routed experts): the rows of X are sorted by expert, rows offsets[e] .. offsets[e + 1] - 1 belong to expert
+// e, and W holds one matrix per expert.  A tile's rows are one expert's; the tiles are laid out from `offsets` on the
+// device (the host knows only the most rows there can be), an expert's row tiles next to one another so that they
+// share its W from L2.  A block of output rows that reaches beyond its expert's last row is written by the epilogue's
+// threads row by row, since a TMA store could not stop there.
 #include "gate_act.cuh"
 #include "tma.cuh"
 #include <cuda_bf16.h>
@@ -49,6 +55,9 @@ struct Bars {
   int aborted;
 };
 constexpr size_t SMEM = 1024 + BARS_OFF + 256;
+constexpr int MAX_EXPERTS = 512;                // grouped: the experts' first row tiles, 16-bit numbers in shared memory
+constexpr size_t SMEM_GROUPED = SMEM + 2 * (MAX_EXPERTS + 8);
+static_assert(SMEM_GROUPED <= 227 * 1024, "shared memory");
 
 struct Params {
   int M, N, K;        // N: columns of C (gated: W has 2 N rows)
@@ -58,6 +67,11 @@ struct Params {
   int act;            // gated: 1 silu, 2 gelu_tanh, 3 the clamped form
   float limit;        // of the clamped form
   int* error;
+  // grouped
+  const int* offsets; // [E + 1] on the device
+  int E;
+  void* out;          // C, for rows that no TMA store takes
+  int64_t ldc;
 };
 
 // ---- the cluster
@@ -196,18 +210,59 @@ struct Item {
   int tile;
   bool h0, h1;   // which halves of the tile
 };
-__device__ __forceinline__ Item item_of(const Params& p, int i) {
+__device__ __forceinline__ Item item_of(int full_items, int i) {
   Item w;
-  if (i < p.full_items) {
+  if (i < full_items) {
     w.tile = i; w.h0 = w.h1 = true;
   } else {
-    const int j = i - p.full_items;
-    w.tile = p.full_items + (j >> 1); w.h0 = (j & 1) == 0; w.h1 = !w.h0;
+    const int j = i - full_items;
+    w.tile = full_items + (j >> 1); w.h0 = (j & 1) == 0; w.h1 = !w.h0;
   }
   return w;
 }
 
-template <bool GATED>
+// Where a tile lies: its first row in X and C, the row behind its last, its column tile, the expert's first row in W.
+struct Place {
+  int m0, end, nti;
+  int64_t w0;
+};
+template <bool GATED, bool GROUPED>
+__device__ __forceinline__ Place place_of(const Params& p, const uint16_t* first, int tile) {
+  Place t;
+  if (!GROUPED) {
+    t.m0 = (tile % p.mt) * 256;
+    t.end = p.M;
+    t.nti = tile / p.mt;
+    t.w0 = 0;
+    return t;
+  }
+  int lo = 0, hi = p.E;                       // the expert e with first[e] * nt <= tile < first[e + 1] * nt
+  while (hi - lo > 1) {
+    const int mid = (lo + hi) >> 1;
+    if ((int)first[mid] * p.nt <= tile) lo = mid;
+    else hi = mid;
+  }
+  const int row_tiles = (int)first[lo + 1] - (int)first[lo], rem = tile - (int)first[lo] * p.nt;
+  t.nti = rem / row_tiles;
+  t.m0 = p.offsets[lo] + (rem - t.nti * row_tiles) * 256;
+  t.end = p.offsets[lo + 1];
+  t.w0 = (int64_t)lo * (GATED ? 2 : 1) * p.N;
+  return t;
+}
+
+// The work items of `tiles` tiles on `pairs` pairs: whole tiles, and the last, ragged wave in halves where that shortens it.
+// Returns the number of items; *full_items of them are whole tiles.
+__host__ __device__ __forceinline__ int plan_items(int tiles, int pairs, int* full_items) {
+  const int full = tiles / pairs, rem = tiles % pairs;
+  if (full > 0 && rem > 0 && 2 * rem <= pairs) {
+    *full_items = tiles - rem;
+    return tiles + rem;
+  }
+  *full_items = tiles;
+  return tiles;
+}
+
+template <bool GATED, bool GROUPED>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(NTHREADS, 1)
 gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constant__ CUtensorMap mapW,
                   const __grid_constant__ CUtensorMap mapC, const Params p) {
@@ -220,6 +275,27 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
   const uint32_t rank = cluster_rank();
   const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
   const int KT = (p.K + 63) / 64;
+  uint16_t* first = reinterpret_cast<uint16_t*>(smem_raw + (sbase - smem_u32(smem_raw)) + BARS_OFF + 256);   // grouped: [E + 1]
+  int items = p.items, full_items = p.full_items;
+  if (GROUPED) {
+    atom::pdl_wait();          // the offsets come from a kernel of this step
+    if (warp == 0) {           // running sums of the experts' row tiles
+      int acc = 0;
+      for (int e0 = 0; e0 < p.E; e0 += 32) {
+        const int e = e0 + lane;
+        const int n = e < p.E ? (p.offsets[e + 1] - p.offsets[e] + 255) / 256 : 0;
+        int sum = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const int up = __shfl_up_sync(0xffffffffu, sum, o);
+          if (lane >= o) sum += up;
+        }
+        if (e < p.E) first[e] = (uint16_t)(acc + sum - n);
+        acc += __shfl_sync(0xffffffffu, sum, 31);
+      }
+      if (lane == 0) first[p.E] = (uint16_t)acc;
+    }
+  }
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) {
@@ -239,6 +315,7 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
   cluster_sync_all();          // both CTAs' barriers exist before anything arrives at them
   tc_fence_after();
   const uint32_t tmem = bars->tmem_base;
+  if (GROUPED) items = plan_items((int)first[p.E] * p.nt, n_pairs, &full_items);
 
   if (warp == 0 || warp >= W_WARP0) {
     // ------------------------------------------------------------------ loaders: one block of every stage each
@@ -246,17 +323,19 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
       const int which = warp == 0 ? 0 : warp - W_WARP0 + 1;       // 0: X, 1: W of half 0, 2: W of half 1
       const CUtensorMap* map = which == 0 ? &mapX : &mapW;
       prefetch_map(map);
-      if (which == 0) atom::pdl_wait();      // X is written by the kernel before this one; W is not
+      if (which == 0 && !GROUPED) atom::pdl_wait();      // X is written by the kernel before this one; W is not
       int it = 0;
-      for (int i = pair; i < p.items; i += n_pairs) {
-        const Item w = item_of(p, i);
-        const int m0 = (w.tile % p.mt) * 256, nti = w.tile / p.mt;
+      for (int i = pair; i < items; i += n_pairs) {
+        const Item w = item_of(full_items, i);
+        const Place at = place_of<GATED, GROUPED>(p, first, w.tile);
+        const int m0 = at.m0, nti = at.nti;
         const bool mine = which == 0 || (which == 1 ? w.h0 : w.h1);
         const uint32_t bytes = 2 * BLK * (1 + (int)w.h0 + (int)w.h1);
         int row;
         if (which == 0) row = m0 + 128 * (int)rank;
         else if (GATED) row = (int)rank * p.N + nti * 256 + (which - 1) * 128;
         else row = nti * 512 + (which - 1) * 256 + 128 * (int)rank;
+        if (which != 0) row += (int)at.w0;
         for (int kt = 0; kt < KT; ++kt, ++it) {
           if (!mine) continue;
           const int s = it % STAGES;
@@ -272,8 +351,8 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
       const uint32_t idesc = instr_desc(256, 256);
       int it = 0;
       int used0 = 0, used1 = 0;       // how often a half of the tensor memory has been filled
-      for (int i = pair; i < p.items; i += n_pairs) {
-        const Item w = item_of(p, i);
+      for (int i = pair; i < items; i += n_pairs) {
+        const Item w = item_of(full_items, i);
         if (w.h0 && used0 > 0) wait_cluster(&bars->acc_empty[0], (used0 - 1) & 1, aborted, p.error);
         if (w.h1 && used1 > 0) wait_cluster(&bars->acc_empty[1], (used1 - 1) & 1, aborted, p.error);
         tc_fence_after();
@@ -313,7 +392,18 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
     int used[2] = {0, 0};
     int blocks = 0;                               // output blocks written so far (they alternate between two buffers)
     // 32 values of this thread's row (16 registers of bf16 pairs) into the block buffer, and the block on its way.
-    auto put_block = [&](const uint32_t* v, int x, int y) {
+    auto put_block = [&](const uint32_t* v, int x, int y, int end) {
+      if (GROUPED && y + 128 > end) {
+        // the block reaches beyond its expert's rows: every thread writes its own row's 32 columns
+        if (y + r < end) {
+          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (int64_t)(y + r) * p.ldc + x + ch * 32;
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            if (x + ch * 32 + c * 8 < p.N)
+              *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(v[4 * c], v[4 * c + 1], v[4 * c + 2], v[4 * c + 3]);
+        }
+        return;
+      }
       if (issuer && blocks >= 2) stores_read_but_one();   // the store that read this buffer two blocks ago is through with it
       epi_sync();
       const uint32_t buf = sbase + OUT_OFF + (blocks & 1) * BLK;
@@ -339,10 +429,10 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
         o[j] = *reinterpret_cast<uint32_t*>(&h2);
       }
     };
-    for (int i = pair; i < p.items; i += n_pairs) {
-      const Item w = item_of(p, i);
-      const int m0 = (w.tile % p.mt) * 256, nti = w.tile / p.mt;
-      const int y = m0 + 128 * (int)rank;
+    for (int i = pair; i < items; i += n_pairs) {
+      const Item w = item_of(full_items, i);
+      const Place at = place_of<GATED, GROUPED>(p, first, w.tile);
+      const int nti = at.nti, y = at.m0 + 128 * (int)rank;
       if (GATED) {
         // First everything out of the tensor memory (a tile's 256 outputs of this thread's row and column half
         // fit in 64 registers as bf16), so that the next tile's MMAs wait for the reads only; then the stores.
@@ -372,7 +462,7 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
         for (int h = 0; h < 2; ++h) {
           if (!(h == 0 ? w.h0 : w.h1)) continue;
 #pragma unroll
-          for (int b = 0; b < 2; ++b) put_block(o[h][b], nti * 256 + h * 128 + b * 64, y);
+          for (int b = 0; b < 2; ++b) put_block(o[h][b], nti * 256 + h * 128 + b * 64, y, at.end);
         }
       } else {
 #pragma unroll
@@ -392,7 +482,7 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
               if (lane == 0) arrive_at(empty0[h]);
             }
             pack(v, o);
-            put_block(o, nti * 512 + h * 256 + b * 64, y);
+            put_block(o, nti * 512 + h * 256 + b * 64, y, at.end);
           }
         }
       }
@@ -409,13 +499,17 @@ gemm_pairs_kernel(const __grid_constant__ CUtensorMap mapX, const __grid_constan
 static int resident_pairs() {
   static int pairs = 0;
   if (pairs == 0) {
-    if (cudaFuncSetAttribute(gemm_pairs_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess ||
-        cudaFuncSetAttribute(gemm_pairs_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM) != cudaSuccess)
+    auto allow = [](const void* f, size_t bytes) {
+      return cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
+    };
+    if (!allow((const void*)gemm_pairs_kernel<false, false>, SMEM) || !allow((const void*)gemm_pairs_kernel<true, false>, SMEM) ||
+        !allow((const void*)gemm_pairs_kernel<false, true>, SMEM_GROUPED) ||
+        !allow((const void*)gemm_pairs_kernel<true, true>, SMEM_GROUPED))
       return 0;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(2, 1, 1);
     cfg.blockDim = dim3(NTHREADS, 1, 1);
-    cfg.dynamicSmemBytes = SMEM;
+    cfg.dynamicSmemBytes = SMEM_GROUPED;
     cudaLaunchAttribute at[1];
     at[0].id = cudaLaunchAttributeClusterDimension;
     at[0].val.clusterDim.x = 2;
@@ -424,7 +518,7 @@ static int resident_pairs() {
     cfg.attrs = at;
     cfg.numAttrs = 1;
     int n = 0;
-    if (cudaOccupancyMaxActiveClusters(&n, gemm_pairs_kernel<true>, &cfg) != cudaSuccess || n < 1) {
+    if (cudaOccupancyMaxActiveClusters(&n, gemm_pairs_kernel<true, true>, &cfg) != cudaSuccess || n < 1) {
       (void)cudaGetLastError();
       return 0;
     }
@@ -445,18 +539,6 @@ ATOM_EXPORT int atom_gemm_pairs_supports(int M, int N, int K, int64_t lda, int64
          atom::tma::encode_fn() != nullptr;
 }
 
-// The work items of a product on `pairs` pairs: whole tiles, and the last, ragged wave in halves where that
-// shortens it.  Returns the number of items; *full_items of them are whole tiles.
-static int plan_items(int tiles, int pairs, int* full_items) {
-  const int rem = tiles % pairs;
-  if (tiles > pairs && rem > 0 && 2 * rem <= pairs) {
-    *full_items = tiles - rem;
-    return tiles + rem;
-  }
-  *full_items = tiles;
-  return tiles;
-}
-
 ATOM_EXPORT int atom_gemm_pairs(const void* X, int64_t lda, const void* W, void* out, int64_t ldc, int M, int N, int K,
                                 int gated, float limit, int* error, cudaStream_t stream) {
   using namespace atom::pairs;
@@ -470,7 +552,7 @@ ATOM_EXPORT int atom_gemm_pairs(const void* X, int64_t lda, const void* W, void*
   if (!atom::tma::cached_map(&mx, X, M, K, lda, 128) || !atom::tma::cached_map(&mw, W, gated ? 2 * (int64_t)N : N, K, K, 128) ||
       !atom::tma::cached_map(&mc, out, M, N, ldc, 128))
     return ATOM_ERR_LIB;
-  Params p;
+  Params p{};
   p.M = M;
   p.N = N;
   p.K = K;
@@ -482,7 +564,46 @@ ATOM_EXPORT int atom_gemm_pairs(const void* X, int64_t lda, const void* W, void*
   const int tiles = p.mt * p.nt;
   if (pairs > tiles) pairs = tiles;
   p.items = plan_items(tiles, pairs, &p.full_items);
-  if (gated) atom::launch_pdl(gemm_pairs_kernel<true>, dim3(2 * pairs), dim3(NTHREADS), SMEM, stream, mx, mw, mc, p);
-  else atom::launch_pdl(gemm_pairs_kernel<false>, dim3(2 * pairs), dim3(NTHREADS), SMEM, stream, mx, mw, mc, p);
+  if (gated) atom::launch_pdl(gemm_pairs_kernel<true, false>, dim3(2 * pairs), dim3(NTHREADS), SMEM, stream, mx, mw, mc, p);
+  else atom::launch_pdl(gemm_pairs_kernel<false, false>, dim3(2 * pairs), dim3(NTHREADS), SMEM, stream, mx, mw, mc, p);
+  return atom::check_launch();
+}
+
+// 1 if the grouped form takes products of E experts of these sizes over at most R rows.
+ATOM_EXPORT int atom_gemm_pairs_grouped_supports(int R, int E, int N, int K) {
+  return E >= 1 && E <= atom::pairs::MAX_EXPERTS && (R + 255) / 256 + E < 65536 && atom_gemm_pairs_supports(R, N, K, K, N);
+}
+
+// C[r] = X[r] W_e^T for the rows r of every expert e; X [R, K] and C [R, N] dense, W [E, N (2 N if gated), K].
+ATOM_EXPORT int atom_gemm_pairs_grouped(const void* X, const void* W, void* out, const int* offsets, int R, int E, int N,
+                                        int K, int gated, float limit, int* error, cudaStream_t stream) {
+  using namespace atom::pairs;
+  if (X == nullptr || W == nullptr || out == nullptr || offsets == nullptr || error == nullptr || gated < 0 || gated > 3 ||
+      !atom_gemm_pairs_grouped_supports(R, E, N, K) ||
+      ((uintptr_t)X % 16) != 0 || ((uintptr_t)W % 16) != 0 || ((uintptr_t)out % 16) != 0)
+    return ATOM_ERR_ARG;
+  int pairs = resident_pairs();
+  if (pairs < 1) return ATOM_ERR_LIB;
+  CUtensorMap mx, mw, mc;
+  if (!atom::tma::cached_map(&mx, X, R, K, K, 128) ||
+      !atom::tma::cached_map(&mw, W, (uint64_t)E * (gated ? 2 : 1) * N, K, K, 128) ||
+      !atom::tma::cached_map(&mc, out, R, N, N, 128))
+    return ATOM_ERR_LIB;
+  Params p{};
+  p.M = R;
+  p.N = N;
+  p.K = K;
+  p.nt = gated ? (N + 255) / 256 : (N + 511) / 512;
+  p.act = gated;
+  p.limit = limit;
+  p.error = error;
+  p.offsets = offsets;
+  p.E = E;
+  p.out = out;
+  p.ldc = N;
+  const int most = ((R + 255) / 256 + E) * p.nt;      // the most tiles there can be
+  if (pairs > most) pairs = most;
+  if (gated) atom::launch_pdl(gemm_pairs_kernel<true, true>, dim3(2 * pairs), dim3(NTHREADS), SMEM_GROUPED, stream, mx, mw, mc, p);
+  else atom::launch_pdl(gemm_pairs_kernel<false, true>, dim3(2 * pairs), dim3(NTHREADS), SMEM_GROUPED, stream, mx, mw, mc, p);
   return atom::check_launch();
 }

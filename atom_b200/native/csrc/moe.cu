@@ -164,6 +164,30 @@ moe_place_kernel(const int* __restrict__ ids, const float* __restrict__ wts, int
   }
 }
 
+// out[r] = (row_w[r] *) x[row_token[r]] for the rows r < offsets[E]; n a multiple of 8, 16 bytes at a time.
+__global__ void moe_gather_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, int64_t ldx,
+                                  const int* __restrict__ offsets, int E, const int* __restrict__ row_token,
+                                  const float* __restrict__ row_w, int n) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  const int r = blockIdx.x;
+  if (r >= offsets[E]) return;
+  const __nv_bfloat16* src = x + (int64_t)row_token[r] * ldx;
+  for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+    uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+    if (row_w) {
+      __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&raw);
+      const float m = row_w[r];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 f = __bfloat1622float2(h2[e]);
+        h2[e] = __floats2bfloat162_rn(f.x * m, f.y * m);
+      }
+    }
+    *reinterpret_cast<uint4*>(out + (int64_t)r * n + i) = raw;
+  }
+}
+
 constexpr int kMoeBM = 32, kMoeBN = 32, kMoeBK = 32;
 
 // Finds the expert and the first row of row tile x: expert e takes ceil(rows_e / BM) tiles, one after another.
@@ -550,6 +574,17 @@ ATOM_EXPORT int atom_moe_place(const int* ids, const float* wts, int pairs, int 
   if (E <= 0 || E > 1024 || top <= 0) return ATOM_ERR_ARG;
   atom::launch_pdl(atom::moe_place_kernel, dim3(1), dim3(1024), 0, stream, ids, wts, pairs, top, E, counts, offsets,
                    row_token, row_w, pair_pos);
+  return atom::check_launch();
+}
+
+// out [R, n] dense; bfloat16 only.
+ATOM_EXPORT int atom_moe_gather(void* out, const void* x, int64_t ldx, const int* offsets, int E, const int* row_token,
+                                const float* row_w, int R, int n, cudaStream_t stream) {
+  if (R <= 0) return ATOM_OK;
+  if (n <= 0 || n % 8 || ldx % 8 || ((uintptr_t)x % 16) != 0 || ((uintptr_t)out % 16) != 0) return ATOM_ERR_ARG;
+  const int threads = n / 8 >= 256 ? 256 : ((n / 8 + 31) / 32) * 32;
+  atom::launch_pdl(atom::moe_gather_kernel, dim3(R), dim3(threads), 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)x,
+                   ldx, offsets, E, row_token, row_w, n);
   return atom::check_launch();
 }
 

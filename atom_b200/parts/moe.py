@@ -92,10 +92,17 @@ class RoutedExperts(FeedForward):
         native.moe_place(ids, wts, E, counts, offsets, row_token, row_w, pair_pos)
         on_input = self.weight_on == "input"
         act = ws.get("moe.act", (R, F), dt)
-        native.moe_gemm(act, x, self.w_gate_up_weight.view(E, 2 * F, H), offsets, gated=True, row_token=row_token,
-                        row_w=row_w if on_input else None, act=self.act, limit=self.limit)
         y = ws.get("moe.y", (R, H), dt)
-        native.moe_gemm(y, act, self.w_down_weight.view(E, H, F), offsets)
+        w_in, w_out, weight = self.w_gate_up_weight.view(E, 2 * F, H), self.w_down_weight.view(E, H, F), row_w if on_input else None
+        if native.moe_pairs_pay(R, E, F, H, dt) and native.moe_pairs_pay(R, E, H, F, dt) and x.stride(0) % 8 == 0:
+            rows = ws.get("moe.rows", (R, H), dt)          # long portions: every expert's rows gathered, then tcgen05
+            native.moe_gather(rows, x, offsets, E, row_token, weight)
+            native.gemm_pairs_grouped(rows, w_in, act, offsets, gated=True, act=self.act, limit=self.limit)
+            native.gemm_pairs_grouped(act, w_out, y, offsets)
+        else:
+            native.moe_gemm(act, x, w_in, offsets, gated=True, row_token=row_token, row_w=weight, act=self.act,
+                            limit=self.limit)
+            native.moe_gemm(y, act, w_out, offsets)
         shared = None
         if self.shared_size is not None:
             S = self.shared_size

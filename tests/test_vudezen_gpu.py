@@ -627,6 +627,47 @@ def test_clamped_experts_with_groups_and_identities(case, dtype, monkeypatch):
         _close(got.cpu()[clear], want[clear], dtype, "experts", f32=3e-5, bf16=3e-2)
 
 
+@pytest.mark.parametrize("counts,N,K", [
+    ([300, 0, 1, 128, 129, 0, 255, 256, 257], 192, 136), ([0, 0, 700], 520, 64), ([64] * 40, 64, 320), ([1], 8, 8),
+    ([513, 2, 127, 90], 1032, 200), ([5, 4, 0, 3, 2, 1], 256, 512), ([0, 0], 128, 128), ([2600, 1500], 768, 256)])
+def test_grouped_products_on_tcgen05(counts, N, K):
+    """Every expert's rows against its own matrix: experts without rows, rows that end anywhere in a tile, sizes that end
+    anywhere in a tile; rows behind the last expert's are left alone, gathered rows are the right ones."""
+    from atom_b200 import native
+
+    g = torch.Generator().manual_seed(sum(counts) + N)
+    E, n = len(counts), sum(counts)
+    R = n + 37
+    off = torch.tensor([0] + counts).cumsum(0).to(torch.int32)
+    src = torch.randn(50, K, generator=g).to(torch.bfloat16)
+    tok = torch.randint(0, 50, (R,), generator=g).to(torch.int32)
+    wts = torch.rand(R, generator=g)
+    for weighted in (False, True):
+        x = torch.full((R, K), float("nan"), dtype=torch.bfloat16, device=DEV)
+        native.moe_gather(x, src.to(DEV), off.to(DEV), E, tok.to(DEV), wts.to(DEV) if weighted else None)
+        rows = src[tok.long()][:n]
+        rows = (rows.float() * wts[:n, None]).to(torch.bfloat16) if weighted else rows
+        assert torch.equal(x.cpu()[:n], rows) and bool(x[n:].isnan().all())
+    for gated, act in ((False, "silu"), (True, "silu"), (True, "clamped")):
+        w = (torch.randn(E, (2 if gated else 1) * N, K, generator=g) * 2 / K ** 0.5).to(torch.bfloat16)
+        out = torch.full((R, N), 7.0, dtype=torch.bfloat16, device=DEV)
+        native.gemm_pairs_grouped(x, w.to(DEV), out, off.to(DEV), gated, act, 1.25)
+        torch.cuda.synchronize()
+        native.check_error_flags()
+        assert bool((out[n:] == 7).all())
+        for e in range(E):
+            r = rows[off[e]:off[e + 1]].double()
+            we = w[e].double()
+            if not gated:
+                want = r @ we.T
+            elif act == "silu":
+                want = torch.nn.functional.silu(r @ we[:N].T) * (r @ we[N:].T)
+            else:
+                want = plain.clamped_expert(r, {"gate": we[:N], "up": we[N:], "down": torch.eye(N, dtype=F64)}, "", 1.25)
+            if counts[e]:
+                _close(out[off[e]:off[e + 1]], want, "bfloat16", f"expert {e}, {act if gated else 'plain'}", bf16=1.5e-2)
+
+
 def test_router_choice_kernel_with_groups_corrections_and_identities():
     from atom_b200 import native
 
