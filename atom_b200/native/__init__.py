@@ -67,8 +67,8 @@ _SIGNATURES = {
     "atom_scale_softcap": [_vp, _i64, _f, _f, _vp],
     "atom_ssm_supports": [_i, _i],
     "atom_ssm_conv_updates_state": [_i],
-    "atom_ssm_conv": [_vp, _vp, _i, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
-    "atom_ssm_step": [_vp, _vp, _vp, _i, _i64, _vp, _vp, _i, _i, _i, _vp],
+    "atom_ssm_conv": [_vp, _vp, _i, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp,
+                      _i, _vp],
     "atom_ssm_scan": [_vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "atom_ssm_tc_supports": [_i, _i],
     "atom_ssm_tc_chunk": [],
@@ -1683,33 +1683,30 @@ def ssm_scratch_elems(T: int, num_seqs: int, H: int, N: int, P: int, run: int):
 
 
 def ssm_conv(u: torch.Tensor, xbc: torch.Tensor, w: torch.Tensor, b: torch.Tensor, state: Optional[torch.Tensor],
+             dt: torch.Tensor, la: torch.Tensor, raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
              seq_of_token: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, num_seqs: int,
              write_state: bool = True) -> None:
-    """u [T, C] = silu(causal convolution of xbc's C channels with w [C, taps], + b) within each request; rows before the
-    step come from state [slots, taps - 1, C] (None for one tap), which takes the request's last taps - 1 rows."""
-    _cuda(u, xbc, w, b, state, seq_of_token, cu_q, state_slots)
+    """What the scan reads.  u [T, C] = silu(causal convolution of xbc's C channels with w [C, taps], + b) within each
+    request; rows before the step come from state [slots, taps - 1, C] (None for one tap), which takes the request's last
+    taps - 1 rows.  dt = softplus(raw + dt_bias), la = -exp(a_log) * dt, float32 [T, H].  xbc and raw are columns of the
+    same rows."""
+    _cuda(u, xbc, w, b, state, dt, la, raw, dt_bias, a_log, seq_of_token, cu_q, state_slots)
     T, C = u.shape
-    taps = w.shape[1]
-    assert xbc.shape == (T, C) and xbc.stride(1) == 1 and u.is_contiguous() and u.dtype == xbc.dtype
+    taps, H = w.shape[1], dt.shape[1]
+    assert xbc.shape == (T, C) and xbc.stride(1) == 1 and u.is_contiguous() and u.dtype == xbc.dtype == raw.dtype
     assert w.shape == (C, taps) and w.is_contiguous() and b.numel() == C and b.dtype == w.dtype
     assert taps == 1 or (state.is_contiguous() and state.dtype == u.dtype and tuple(state.shape[1:]) == (taps - 1, C))
+    assert dt.dtype == la.dtype == torch.float32 and dt.is_contiguous() and la.is_contiguous() and dt.shape == la.shape == (T, H)
+    assert raw.shape == (T, H) and raw.stride(1) == 1 and raw.stride(0) == xbc.stride(0)
+    assert dt_bias.numel() == a_log.numel() == H and dt_bias.dtype == a_log.dtype == w.dtype
     _check(lib().atom_ssm_conv(u.data_ptr(), xbc.data_ptr(), dtype_code(u.dtype), xbc.stride(0), w.data_ptr(), b.data_ptr(),
                                dtype_code(w.dtype), _ptr(state) if taps > 1 else None, taps, seq_of_token.data_ptr(),
-                               cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, C, int(write_state), _stream()),
-           "ssm_conv")
-    if taps > 1 and write_state and not lib().atom_ssm_conv_updates_state(taps):
-        conv_state_update(state, xbc, cu_q, state_slots, num_seqs)
-
-
-def ssm_step(dt: torch.Tensor, la: torch.Tensor, raw: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor) -> None:
-    """dt = softplus(raw + dt_bias), la = -exp(a_log) * dt; dt, la float32 [T, H], raw a view of the projection."""
-    _cuda(dt, la, raw, dt_bias, a_log)
-    T, H = dt.shape
-    assert dt.dtype == la.dtype == torch.float32 and dt.is_contiguous() and la.is_contiguous() and la.shape == (T, H)
-    assert raw.shape == (T, H) and raw.stride(1) == 1 and dt_bias.numel() == a_log.numel() == H
-    assert dt_bias.dtype == a_log.dtype
-    _check(lib().atom_ssm_step(dt.data_ptr(), la.data_ptr(), raw.data_ptr(), dtype_code(raw.dtype), raw.stride(0),
-                               dt_bias.data_ptr(), a_log.data_ptr(), dtype_code(a_log.dtype), T, H, _stream()), "ssm_step")
+                               cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, C, int(write_state), dt.data_ptr(),
+                               la.data_ptr(), raw.data_ptr(), dt_bias.data_ptr(), a_log.data_ptr(), H, _stream()), "ssm_conv")
+    if not lib().atom_ssm_conv_updates_state(taps):
+        add_launches(1)
+        if write_state:
+            conv_state_update(state, xbc, cu_q, state_slots, num_seqs)
 
 
 def ssm_scan(out: torch.Tensor, u: torch.Tensor, dt: torch.Tensor, la: torch.Tensor, D: torch.Tensor, state: torch.Tensor,

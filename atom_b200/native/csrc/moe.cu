@@ -37,10 +37,12 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
                                  float* __restrict__ wts, int* __restrict__ counts) {
   atom::pdl_trigger();
   atom::pdl_wait();
+  extern __shared__ float route_s[];        // a row of E choice scores per warp
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (t >= T) return;
   const int E = p.E, top = p.top;
+  float* cs = route_s + (threadIdx.x >> 5) * E;
   if (seq_of_token[t] < 0) {
     for (int k = lane; k < top; k += 32) ids[(int64_t)t * top + k] = -1;
     return;
@@ -56,7 +58,10 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ld, c
   }
   auto score = [&](int e) { return p.softmax_scores ? expf(z[e] - zmax) / denom : 1.f / (1.f + expf(-z[e])); };
   // what the choice goes by: the logit itself where scores grow with it and nothing is added to them
-  auto choice = [&](int e) { return p.correction ? score(e) + load_as_float(p.correction, p.correction_dtype, e) : z[e]; };
+  for (int e = lane; e < E; e += 32)
+    cs[e] = p.correction ? score(e) + load_as_float(p.correction, p.correction_dtype, e) : z[e];
+  __syncwarp();
+  auto choice = [&](int e) { return cs[e]; };
   uint32_t taken = 0;                       // bit m: expert lane + 32 m cannot be chosen (any more) (E <= 1024)
   if (p.groups > 1) {
     // a group's score is its largest choice score: the best `keep` groups one after another (ties: the lower group)
@@ -317,6 +322,57 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const T* __restrict__ y,
   }
 }
 
+// The same for bfloat16 rows of a multiple of 8 numbers, 16 bytes at a time; the row's places and weights are read once,
+// the sums run over the choices in the same order.
+constexpr int kCombineTop = 8;
+__global__ void moe_combine_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ y,
+                                            const int* __restrict__ pair_pos, const float* __restrict__ pair_w, int top,
+                                            const __nv_bfloat16* __restrict__ shared_out, const float* __restrict__ gate,
+                                            int64_t gate_ld, int n, const int* __restrict__ seq_of_token,
+                                            const __nv_bfloat16* __restrict__ x, int64_t ldx, const int* __restrict__ ids,
+                                            int identity_from) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  const int t = blockIdx.x;
+  if (seq_of_token[t] < 0) return;
+  const float sg = (shared_out && gate) ? 1.f / (1.f + expf(-gate[(int64_t)t * gate_ld])) : 1.f;
+  int pos[kCombineTop];
+  float w[kCombineTop], own = 0.f;
+#pragma unroll
+  for (int k = 0; k < kCombineTop; ++k) {
+    pos[k] = -1;
+    w[k] = 0.f;
+    if (k < top) {
+      pos[k] = pair_pos[(int64_t)t * top + k];
+      w[k] = pair_w ? pair_w[(int64_t)t * top + k] : 1.f;
+      if (x && ids[(int64_t)t * top + k] >= identity_from) own += w[k];
+    }
+  }
+  auto add8 = [](float (&s)[8], float f, const __nv_bfloat16* p) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 v = __bfloat1622float2(h2[e]);
+      s[2 * e] += f * v.x;
+      s[2 * e + 1] += f * v.y;
+    }
+  };
+  for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 8; i < n; i += gridDim.y * blockDim.x * 8) {
+    float s[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (own != 0.f) add8(s, own, x + (int64_t)t * ldx + i);
+#pragma unroll
+    for (int k = 0; k < kCombineTop; ++k)
+      if (pos[k] >= 0) add8(s, w[k], y + (int64_t)pos[k] * n + i);
+    if (shared_out) add8(s, sg, shared_out + (int64_t)t * n + i);
+    uint4 q;
+    __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&q);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h2[e] = __floats2bfloat162_rn(s[2 * e], s[2 * e + 1]);
+    *reinterpret_cast<uint4*>(out + (int64_t)t * n + i) = q;
+  }
+}
+
 // ---- the same product in bfloat16 on the tensor cores -----------------------------------------------------------
 // A CTA of 4 warps takes BM rows of one expert (64, or 16 in steps of few rows, where the warps share out the
 // columns instead of the rows) and 64 output columns (with GATED the 64 gate rows and the 64 up rows of W_e), and
@@ -563,7 +619,7 @@ ATOM_EXPORT int atom_moe_route(const float* logits, int64_t ld, int T, int E, in
   if (groups > 1 && (E % groups || keep < 1 || keep > groups || top > keep * (E / groups))) return ATOM_ERR_ARG;
   const atom::MoeRouteArgs p{E, E - identity, top, softmax_scores, renormalize, sum_eps, factor, correction,
                              correction_dtype, groups, keep};
-  atom::launch_pdl(atom::moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, p, seq_of_token, T, ids,
+  atom::launch_pdl(atom::moe_route_kernel, dim3((T + 3) / 4), dim3(128), sizeof(float) * 4 * (size_t)E, stream, logits, ld, p, seq_of_token, T, ids,
                    wts, counts);
   return atom::check_launch();
 }
@@ -621,7 +677,14 @@ ATOM_EXPORT int atom_moe_combine(void* out, const void* y, int dtype, const int*
     atom::launch_pdl(atom::moe_combine_kernel<float>, grid, dim3(256), 0, stream, (float*)out, (const float*)y,
                      pair_pos, pair_w, top, (const float*)shared_out, gate, gate_ld, n, seq_of_token, (const float*)x, ldx, ids,
                      identity_from);
-  else if (dtype == ATOM_BF16)
+  else if (dtype == ATOM_BF16 && n % 8 == 0 && top <= atom::kCombineTop && ldx % 8 == 0 && ((uintptr_t)out % 16) == 0 &&
+           ((uintptr_t)y % 16) == 0 && ((uintptr_t)shared_out % 16) == 0 && ((uintptr_t)x % 16) == 0) {
+    const int vecs = n / 8, threads = vecs >= 256 ? 256 : ((vecs + 31) / 32) * 32;
+    atom::launch_pdl(atom::moe_combine_bf16_vec_kernel, dim3(T, T >= 512 ? 1 : (unsigned)((vecs + threads - 1) / threads)),
+                     dim3(threads), 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)y, pair_pos, pair_w, top,
+                     (const __nv_bfloat16*)shared_out, gate, gate_ld, n, seq_of_token, (const __nv_bfloat16*)x, ldx, ids,
+                     identity_from);
+  } else if (dtype == ATOM_BF16)
     atom::launch_pdl(atom::moe_combine_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (__nv_bfloat16*)out,
                      (const __nv_bfloat16*)y, pair_pos, pair_w, top, (const __nv_bfloat16*)shared_out, gate, gate_ld, n,
                      seq_of_token, (const __nv_bfloat16*)x, ldx, ids, identity_from);

@@ -6,6 +6,7 @@
 //                         updated by conv_state_update_kernel afterwards).  A thread owns two channels over a strip of
 //                         16 rows of one request; the strip of a request's first rows holds all rows that read the
 //                         state, so the thread that read it may write it.
+//                         The blocks of the last grid row do the work of ssm_step_kernel for the strip's rows.
 //   ssm_step_kernel       dt = softplus(raw + dt_bias), la = -exp(A_log) * dt   per (token, head), 32-bit
 //   ssm_scan_kernel       S_t = exp(la_t) S_(t-1) + dt_t B_t x_t^T;   y_t = S_t^T C_t + D x_t
 //   ssm_gate_norm_kernel  y <- (y * silu(z)) / rms over each of `parts` equal parts * w (* a constant)
@@ -70,16 +71,39 @@ __device__ __forceinline__ void store_pair<__nv_bfloat16>(__nv_bfloat16* p, floa
   }
 }
 
+// dt = softplus(raw + dt_bias), la = -exp(A_log) dt of one (token, head).
+struct StepArgs {
+  float* dt;                   // [T, H]
+  float* la;
+  const void* raw;             // rows of the projection (their own stride), activation type
+  const void* dt_bias;
+  const void* a_log;
+  int H;
+};
+template <typename T>
+__device__ __forceinline__ void ssm_step_at(const StepArgs& p, int64_t ld, int w_dtype, int64_t t, int h) {
+  const float v = to_float(((const T*)p.raw)[t * ld + h]) + load_as_float(p.dt_bias, w_dtype, h);
+  const float d = fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
+  p.dt[t * p.H + h] = d;
+  p.la[t * p.H + h] = -expf(load_as_float(p.a_log, w_dtype, h)) * d;
+}
+
 // u [T, C] dense; xbc: rows of the projection (stride ld); state [slots, TAPS - 1, C].
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 ssm_conv_kernel(T* __restrict__ u, const T* __restrict__ xbc, int64_t ld, const void* __restrict__ w,
                 const void* __restrict__ b, int w_dtype, T* __restrict__ state, const int* __restrict__ cu_q,
-                const int* __restrict__ state_slots, int num_seqs, int C, int write_state) {
+                const int* __restrict__ state_slots, int num_seqs, int C, int write_state, const StepArgs steps) {
   atom::pdl_trigger();
   atom::pdl_wait();
   int s, r;
   if (!ssm_find_run(blockIdx.x, cu_q, num_seqs, kSsmStrip, s, r)) return;
+  if (blockIdx.y == gridDim.y - 1) {
+    const int ta = cu_q[s] + r * kSsmStrip, n = min(cu_q[s + 1] - ta, kSsmStrip);
+    for (int e = threadIdx.x; e < n * steps.H; e += blockDim.x)
+      ssm_step_at<T>(steps, ld, w_dtype, ta + e / steps.H, e % steps.H);
+    return;
+  }
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 2;
   if (c >= C) return;
   const bool two = c + 1 < C;
@@ -155,19 +179,12 @@ __global__ void ssm_conv_any_kernel(T* __restrict__ u, const T* __restrict__ xbc
 }
 
 template <typename T>
-__global__ void ssm_step_kernel(float* __restrict__ dt, float* __restrict__ la, const T* __restrict__ raw, int64_t ld,
-                                const void* __restrict__ dt_bias, const void* __restrict__ a_log, int w_dtype, int H,
-                                int64_t total) {
+__global__ void ssm_step_kernel(const StepArgs steps, int64_t ld, int w_dtype, int64_t total) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int64_t e = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (e >= total) return;
-  const int64_t t = e / H;
-  const int h = (int)(e - t * H);
-  const float v = to_float(raw[t * ld + h]) + load_as_float(dt_bias, w_dtype, h);
-  const float d = fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
-  dt[e] = d;
-  la[e] = -expf(load_as_float(a_log, w_dtype, h)) * d;
+  ssm_step_at<T>(steps, ld, w_dtype, e / steps.H, (int)(e % steps.H));
 }
 
 // Row n of register m of a thread of slice 0..3: runs of four in a row (one 16-byte load each).
@@ -336,21 +353,73 @@ __global__ void ssm_gate_norm_kernel(T* __restrict__ out, int64_t ldo, const flo
     out[(int64_t)t * ldo + i0 + i] = from_float<T>(gated[i] * f * load_as_float(w, w_dtype, i0 + i) * mul);
 }
 
+// The same for bfloat16 parts of a multiple of 8 numbers, 16 bytes at a time; at most 8 * NV * blockDim numbers a part,
+// which wait in registers.
+template <int NV>
+__global__ void ssm_gate_norm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, int64_t ldo, const float* __restrict__ y,
+                                              const __nv_bfloat16* __restrict__ z, int64_t ldz,
+                                              const __nv_bfloat16* __restrict__ w, int n, int parts, float eps, float mul,
+                                              const int* __restrict__ seq_of_token) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  __shared__ float scratch[32];
+  const int t = blockIdx.x;
+  if (seq_of_token[t] < 0) return;
+  const int len = n / parts, i0 = blockIdx.y * len;
+  float v[NV][8], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 8;
+    if (i < len) {
+      const float4 a = *reinterpret_cast<const float4*>(y + (int64_t)t * n + i0 + i);
+      const float4 b = *reinterpret_cast<const float4*>(y + (int64_t)t * n + i0 + i + 4);
+      const uint4 raw = *reinterpret_cast<const uint4*>(z + (int64_t)t * ldz + i0 + i);
+      const __nv_bfloat16* zv = reinterpret_cast<const __nv_bfloat16*>(&raw);
+      v[k][0] = a.x; v[k][1] = a.y; v[k][2] = a.z; v[k][3] = a.w;
+      v[k][4] = b.x; v[k][5] = b.y; v[k][6] = b.z; v[k][7] = b.w;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        v[k][e] *= ssm_silu(__bfloat162float(zv[e]));
+        ss = fmaf(v[k][e], v[k][e], ss);
+      }
+    }
+  }
+  ss = block_sum(ss, scratch);
+  const float f = rsqrtf(ss / (float)len + eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 8;
+    if (i < len) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(w + i0 + i);
+      const __nv_bfloat16* wv = reinterpret_cast<const __nv_bfloat16*>(&raw);
+      uint4 q;
+      __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&q);
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        h2[e] = __floats2bfloat162_rn(v[k][2 * e] * f * __bfloat162float(wv[2 * e]) * mul,
+                                      v[k][2 * e + 1] * f * __bfloat162float(wv[2 * e + 1]) * mul);
+      *reinterpret_cast<uint4*>(out + (int64_t)t * ldo + i0 + i) = q;
+    }
+  }
+}
+
 template <typename T>
 static int ssm_conv_launch(T* u, const T* xbc, int64_t ld, const void* w, const void* b, int w_dtype, T* state, int taps,
                            const int* seq_of_token, const int* cu_q, const int* state_slots, int num_seqs, int rows, int C,
-                           int write_state, cudaStream_t stream) {
-  const dim3 grid((rows + kSsmStrip - 1) / kSsmStrip + num_seqs, (C + 255) / 256);
+                           int write_state, const StepArgs& steps, cudaStream_t stream) {
+  const dim3 grid((rows + kSsmStrip - 1) / kSsmStrip + num_seqs, (C + 255) / 256 + 1);
 #define ATOM_SC(N)                                                                                                  \
   case N:                                                                                                           \
     launch_pdl(ssm_conv_kernel<T, N>, grid, dim3(128), 0, stream, u, xbc, ld, w, b, w_dtype, state, cu_q, state_slots, \
-               num_seqs, C, write_state);                                                                           \
+               num_seqs, C, write_state, steps);                                                                    \
     break;
   switch (taps) {
     ATOM_SC(1) ATOM_SC(2) ATOM_SC(3) ATOM_SC(4) ATOM_SC(5) ATOM_SC(6) ATOM_SC(7) ATOM_SC(8)
     default:
       launch_pdl(ssm_conv_any_kernel<T>, dim3(rows, (C + 255) / 256), dim3(256), 0, stream, u, xbc, ld, w, b, w_dtype,
                  (const T*)state, taps, seq_of_token, cu_q, state_slots, C);
+      const int64_t total = (int64_t)rows * steps.H;
+      launch_pdl(ssm_step_kernel<T>, dim3((unsigned)((total + 127) / 128)), dim3(128), 0, stream, steps, ld, w_dtype, total);
   }
 #undef ATOM_SC
   return check_launch();
@@ -399,39 +468,26 @@ static int ssm_scan_dispatch(float* out, const T* u, const float* dt, const floa
 
 ATOM_EXPORT int atom_ssm_supports(int N, int P) { return N > 0 && N <= 256 && P > 0 ? 1 : 0; }
 
-// Whether the convolution with so many taps also brings its state up to date.
+// Whether the convolution with so many taps also brings its state up to date (and is one launch).
 ATOM_EXPORT int atom_ssm_conv_updates_state(int taps) { return taps <= 8 ? 1 : 0; }
 
+// The convolution, and dt and la [T, H] of the same rows: raw lies in rows of the same stride ld; dt_bias, a_log [H] have
+// w's type.
 ATOM_EXPORT int atom_ssm_conv(void* u, const void* xbc, int dtype, int64_t ld, const void* w, const void* b, int w_dtype,
                               void* state, int taps, const int* seq_of_token, const int* cu_q, const int* state_slots,
-                              int num_seqs, int T, int C, int write_state, cudaStream_t stream) {
+                              int num_seqs, int T, int C, int write_state, float* dt, float* la, const void* raw,
+                              const void* dt_bias, const void* a_log, int H, cudaStream_t stream) {
   if (T <= 0 || num_seqs <= 0) return ATOM_OK;
-  if (C <= 0 || taps < 1 || taps > 64 || (taps > 1 && !state)) return ATOM_ERR_ARG;
+  const atom::StepArgs steps{dt, la, raw, dt_bias, a_log, H};
+  if (C <= 0 || H <= 0 || !dt || !la || !raw || taps < 1 || taps > 64 || (taps > 1 && !state)) return ATOM_ERR_ARG;
   if (dtype == ATOM_F32)
     return atom::ssm_conv_launch<float>((float*)u, (const float*)xbc, ld, w, b, w_dtype, (float*)state, taps, seq_of_token,
-                                        cu_q, state_slots, num_seqs, T, C, write_state, stream);
+                                        cu_q, state_slots, num_seqs, T, C, write_state, steps, stream);
   if (dtype == ATOM_BF16)
     return atom::ssm_conv_launch<__nv_bfloat16>((__nv_bfloat16*)u, (const __nv_bfloat16*)xbc, ld, w, b, w_dtype,
                                                 (__nv_bfloat16*)state, taps, seq_of_token, cu_q, state_slots, num_seqs, T,
-                                                C, write_state, stream);
+                                                C, write_state, steps, stream);
   return ATOM_ERR_ARG;
-}
-
-ATOM_EXPORT int atom_ssm_step(float* dt, float* la, const void* raw, int dtype, int64_t ld, const void* dt_bias,
-                              const void* a_log, int w_dtype, int T, int H, cudaStream_t stream) {
-  if (T <= 0) return ATOM_OK;
-  if (H <= 0) return ATOM_ERR_ARG;
-  const int64_t total = (int64_t)T * H;
-  const int blocks = (int)((total + 127) / 128);
-  if (dtype == ATOM_F32)
-    atom::launch_pdl(atom::ssm_step_kernel<float>, dim3(blocks), dim3(128), 0, stream, dt, la, (const float*)raw, ld,
-                     dt_bias, a_log, w_dtype, H, total);
-  else if (dtype == ATOM_BF16)
-    atom::launch_pdl(atom::ssm_step_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), 0, stream, dt, la,
-                     (const __nv_bfloat16*)raw, ld, dt_bias, a_log, w_dtype, H, total);
-  else
-    return ATOM_ERR_ARG;
-  return atom::check_launch();
 }
 
 // run 0: every request is walked once.  Otherwise sB holds (ceil(T / run) + num_seqs) * H * N * P floats and sA
@@ -470,6 +526,18 @@ ATOM_EXPORT int atom_ssm_gate_norm(void* out, int dtype, int64_t ldo, const floa
   if (n <= 0 || parts <= 0 || n % parts || parts > 65535 || n / parts > 11 * 1024) return ATOM_ERR_ARG;
   const int len = n / parts;
   const int threads = len >= 1024 ? 256 : (len >= 256 ? 128 : (len > 32 ? 64 : 32));
+  auto al = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
+  if (dtype == ATOM_BF16 && w_dtype == ATOM_BF16 && len % 8 == 0 && len <= 8 * 1024 && ldo % 8 == 0 && ldz % 8 == 0 && al(out) &&
+      al(y) && al(z) && al(w)) {
+    const int vecs = len / 8, th = vecs <= 512 ? ((vecs + 31) / 32) * 32 : ((vecs / 2 + 32) / 32) * 32;
+    if (vecs <= 512)
+      atom::launch_pdl(atom::ssm_gate_norm_bf16_vec_kernel<1>, dim3(T, parts), dim3(th), 0, stream, (__nv_bfloat16*)out, ldo, y,
+                       (const __nv_bfloat16*)z, ldz, (const __nv_bfloat16*)w, n, parts, eps, mul, seq_of_token);
+    else
+      atom::launch_pdl(atom::ssm_gate_norm_bf16_vec_kernel<2>, dim3(T, parts), dim3(th), 0, stream, (__nv_bfloat16*)out, ldo, y,
+                       (const __nv_bfloat16*)z, ldz, (const __nv_bfloat16*)w, n, parts, eps, mul, seq_of_token);
+    return atom::check_launch();
+  }
   const size_t smem = sizeof(float) * (size_t)len;
   if (dtype == ATOM_F32)
     atom::launch_pdl(atom::ssm_gate_norm_kernel<float>, dim3(T, parts), dim3(threads), smem, stream, (float*)out, ldo, y,

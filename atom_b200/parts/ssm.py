@@ -65,11 +65,11 @@ class StateSpace(ProjectedMixer):
         H, P, N, G, I, C = self.nh, self.dv, self.n, self.g, self.inner_cols, self.channels
         rows = proj["in"]
         u = ws.get("ssm.u", (T, C), dt_)
-        native.ssm_conv(u, rows[:, I:I + C], self.w_conv_weight, self.w_conv_bias, cache.states.get("conv"),
-                        step.seq_of_token, step.cu_q, step.state_slots, step.num_seqs, writes_cache)
         dt = ws.get("ssm.dt", (T, H), torch.float32)
         la = ws.get("ssm.la", (T, H), torch.float32)
-        native.ssm_step(dt, la, rows[:, I + C:], self.w_dt_bias, self.w_A_log)
+        native.ssm_conv(u, rows[:, I:I + C], self.w_conv_weight, self.w_conv_bias, cache.states.get("conv"), dt, la,
+                        rows[:, I + C:], self.w_dt_bias, self.w_A_log, step.seq_of_token, step.cu_q, step.state_slots,
+                        step.num_seqs, writes_cache)
         o = ws.get("ssm.o", (T, I), torch.float32)
         run, _ = native.ssm_run(min(T, step.max_q_len), N, P, dt_)
         nb, na = native.ssm_scratch_elems(T, step.num_seqs, H, N, P, run)

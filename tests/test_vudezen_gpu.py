@@ -476,10 +476,17 @@ def test_step_sizes_have_no_clamp():
     from atom_b200 import native
 
     raw = torch.tensor([[-200.0, -20.0, -1.0, 0.0, 3.0, 25.0, 300.0]], device=DEV)
-    H = raw.shape[1]
-    dt, la = torch.empty(1, H, device=DEV), torch.empty(1, H, device=DEV)
+    H, z = raw.shape[1], lambda *n: torch.zeros(*n, device=DEV)
     b, a_log = torch.full((H,), 0.25, device=DEV), torch.linspace(-3, 2, H, device=DEV)
-    native.ssm_step(dt, la, raw, b, a_log)
+    for taps in (1, 4, 9):
+        dt, la = torch.full((1, H), -1.0, device=DEV), torch.full((1, H), 1.0, device=DEV)
+        rows = torch.cat([z(1, 5), raw], dim=1)
+        native.ssm_conv(z(1, 5), rows[:, :5], z(5, taps), z(5), z(2, taps - 1, 5) if taps > 1 else None, dt, la, rows[:, 5:], b,
+                        a_log, _i32([0]), _i32([0, 1]), _i32([1]), 1)
+        _check_steps(dt, la, raw, a_log)
+
+
+def _check_steps(dt, la, raw, a_log):
     v = raw.double().cpu() + 0.25
     want = torch.log1p(torch.exp(-v.abs())) + v.clamp(min=0)
     assert torch.allclose(dt.double().cpu(), want, rtol=1e-6, atol=1e-40)
