@@ -7,8 +7,7 @@
 //   residual[row] = r  (unless rows are picked);   out = LN(r; w, b, eps)
 // With `rows` given only those rows are normalised and written densely (the gather of the rows whose logits are
 // wanted).  All arithmetic is 32-bit; the variance is the mean of squared deviations, formed in a pass of its own
-// over numbers that stay on chip (the 16-byte kernel merges every thread's count, mean and sum of squared deviations
-// instead: one reduction per norm).  delta and out have the activation type.
+// over numbers that stay on chip.  delta and out have the activation type.
 #include "common.cuh"
 
 namespace atom {
@@ -99,63 +98,47 @@ __device__ __forceinline__ void ln_load8(const void* w, int dtype, int64_t i, fl
   }
 }
 
-// Count, mean and sum of squared deviations of a set of numbers; merge takes two disjoint sets together (the parallel
-// form of Chan, Golub and LeVeque).
-struct Moments {
-  float n, mean, m2;
-};
-__device__ __forceinline__ Moments merge(const Moments& a, const Moments& b) {
-  const float n = a.n + b.n;
-  const float share = n > 0.f ? __fdividef(b.n, n) : 0.f;
-  const float d = b.mean - a.mean;
-  return {n, fmaf(d, share, a.mean), a.m2 + b.m2 + d * d * a.n * share};
-}
-// scratch: 32 Moments in shared memory.  Every thread gets the whole block's.
-__device__ __forceinline__ Moments block_moments(Moments v, Moments* scratch) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
-  auto lanes = [](Moments a) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const Moments b{__shfl_xor_sync(0xffffffffu, a.n, o), __shfl_xor_sync(0xffffffffu, a.mean, o),
-                      __shfl_xor_sync(0xffffffffu, a.m2, o)};
-      a = (threadIdx.x & o) ? merge(b, a) : merge(a, b);      // (the same order in both lanes: the same result)
-    }
-    return a;
-  };
-  v = lanes(v);
-  __syncthreads();           // scratch may still be read from an earlier reduction
-  if (lane == 0) scratch[warp] = v;
+// A block's sum with a scratch row of its own for every sum of the kernel, so that one barrier is enough.
+__device__ __forceinline__ float block_sum_once(float v, float* scratch) {
+  const int lane = threadIdx.x & 31, warps = (blockDim.x + 31) >> 5;
+  v = warp_sum(v);
+  if (lane == 0) scratch[threadIdx.x >> 5] = v;
   __syncthreads();
-  return lanes(lane < warps ? scratch[lane] : Moments{0.f, 0.f, 0.f});
+  return warp_sum(lane < warps ? scratch[lane] : 0.f);
 }
+// Mean of the row and sum of squared deviations from it.
 template <int NV>
-__device__ __forceinline__ Moments thread_moments(const float (&v)[NV][8], int H) {
-  Moments m{0.f, 0.f, 0.f};
+__device__ __forceinline__ void row_moments(const float (&v)[NV][8], int H, float* sums, float& mean, float& m2) {
+  float s = 0.f;
 #pragma unroll
-  for (int k = 0; k < NV; ++k) {
-    if ((int)(threadIdx.x + k * blockDim.x) * 8 >= H) continue;
-    float s = 0.f, q = 0.f;
+  for (int k = 0; k < NV; ++k)
+    if ((int)(threadIdx.x + k * blockDim.x) * 8 < H) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) s += v[k][e];
-    s *= 0.125f;
+      for (int e = 0; e < 8; ++e) s += v[k][e];
+    }
+  mean = block_sum_once(s, sums) / (float)H;
+  s = 0.f;
 #pragma unroll
-    for (int e = 0; e < 8; ++e) q = fmaf(v[k][e] - s, v[k][e] - s, q);
-    m = merge(m, Moments{8.f, s, q});
-  }
-  return m;
+  for (int k = 0; k < NV; ++k)
+    if ((int)(threadIdx.x + k * blockDim.x) * 8 < H) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s = fmaf(v[k][e] - mean, v[k][e] - mean, s);
+    }
+  m2 = block_sum_once(s, sums + 32);
 }
 
 // bfloat16 rows of a multiple of 8 numbers, at most 8 * NV * blockDim: a thread keeps its 8 * NV numbers in registers,
-// so that every array is read once and written once, 16 bytes at a time.  AHEAD (steps of few rows, NV == 1): the weights,
-// which do not depend on the kernel in front of this one, are on their way before the wait.
-template <int NV, bool AHEAD>
+// so that every array is read once and written once, 16 bytes at a time.  A CTA takes row after row; with NV == 1 it keeps
+// the weights in registers over its rows, and they are on their way before the wait, since they do not depend on the
+// kernel in front of this one.
+template <int NV>
 __global__ void __launch_bounds__(1024)
 add_layernorm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, float* __restrict__ residual,
-                              const __nv_bfloat16* __restrict__ delta, const LayerNormArgs p) {
+                              const __nv_bfloat16* __restrict__ delta, const LayerNormArgs p, int n_rows) {
   atom::pdl_trigger();
-  __shared__ Moments scratch[32];
-  const int r = blockIdx.x, H = p.H;
-  const int64_t src = p.rows ? p.rows[r] : r;
+  __shared__ float scratch[2][4][32];      // (two rows in turn: a row's sums may still be read when the next begins)
+  constexpr bool AHEAD = NV == 1;
+  const int H = p.H;
   const bool normed = delta && p.wd;
   float w1[8], b1[8], w2[8], b2[8];
   if (AHEAD && threadIdx.x * 8 < H) {
@@ -167,70 +150,76 @@ add_layernorm_bf16_vec_kernel(__nv_bfloat16* __restrict__ out, float* __restrict
     ln_load8(p.b, p.w_dtype, threadIdx.x * 8, b2);
   }
   atom::pdl_wait();
-  float* res = residual + src * H;
-  float v[NV][8], rv[NV][8];
+  for (int r = blockIdx.x, odd = 0; r < n_rows; r += gridDim.x, odd ^= 1) {
+    float(*sums)[32] = scratch[odd];
+    const int64_t src = p.rows ? p.rows[r] : r;
+    float* res = residual + src * H;
+    float v[NV][8], rv[NV][8];
 #pragma unroll
-  for (int k = 0; k < NV; ++k) {
-    const int i = (threadIdx.x + k * blockDim.x) * 8;
-    if (i < H) {
-      ln_load8(res, ATOM_F32, i, rv[k]);
-      if (delta) {
-        ln_load8(delta, ATOM_BF16, src * H + i, v[k]);
-        if (p.dbias) {
-          float bv[8];
-          ln_load8(p.dbias, p.w_dtype, i, bv);
+    for (int k = 0; k < NV; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i < H) {
+        ln_load8(res, ATOM_F32, i, rv[k]);
+        if (delta) {
+          ln_load8(delta, ATOM_BF16, src * H + i, v[k]);
+          if (p.dbias) {
+            float bv[8];
+            ln_load8(p.dbias, p.w_dtype, i, bv);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) v[k][e] += bv[e];
+            for (int e = 0; e < 8; ++e) v[k][e] += bv[e];
+          }
         }
       }
     }
-  }
-  if (normed) {
-    const Moments m = block_moments(thread_moments<NV>(v, H), scratch);
-    const float rstd = ln_rstd(m.m2, H, p.eps_d);
+    if (normed) {
+      float mean, m2;
+      row_moments<NV>(v, H, sums[0], mean, m2);
+      const float rstd = ln_rstd(m2, H, p.eps_d);
+#pragma unroll
+      for (int k = 0; k < NV; ++k) {
+        const int i = (threadIdx.x + k * blockDim.x) * 8;
+        if (i < H) {
+          if (!AHEAD) {
+            ln_load8(p.wd, p.w_dtype, i, w1);
+            ln_load8(p.bd, p.w_dtype, i, b1);
+          }
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[k][e] = (v[k][e] - mean) * rstd * w1[e] + b1[e];
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i < H && delta) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) rv[k][e] += p.dscale * v[k][e];
+        if (!p.rows) {
+          *reinterpret_cast<float4*>(res + i) = make_float4(rv[k][0], rv[k][1], rv[k][2], rv[k][3]);
+          *reinterpret_cast<float4*>(res + i + 4) = make_float4(rv[k][4], rv[k][5], rv[k][6], rv[k][7]);
+        }
+      }
+    }
+    float mean, m2;
+    row_moments<NV>(rv, H, sums[2], mean, m2);
+    const float rstd = ln_rstd(m2, H, p.eps);
+    __nv_bfloat16* o = out + (int64_t)r * H;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
       const int i = (threadIdx.x + k * blockDim.x) * 8;
       if (i < H) {
         if (!AHEAD) {
-          ln_load8(p.wd, p.w_dtype, i, w1);
-          ln_load8(p.bd, p.w_dtype, i, b1);
+          ln_load8(p.w, p.w_dtype, i, w2);
+          ln_load8(p.b, p.w_dtype, i, b2);
         }
+        uint4 q;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&q);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[k][e] = (v[k][e] - m.mean) * rstd * w1[e] + b1[e];
+        for (int e = 0; e < 4; ++e)
+          h[e] = __floats2bfloat162_rn((rv[k][2 * e] - mean) * rstd * w2[2 * e] + b2[2 * e],
+                                       (rv[k][2 * e + 1] - mean) * rstd * w2[2 * e + 1] + b2[2 * e + 1]);
+        *reinterpret_cast<uint4*>(o + i) = q;
       }
-    }
-  }
-#pragma unroll
-  for (int k = 0; k < NV; ++k) {
-    const int i = (threadIdx.x + k * blockDim.x) * 8;
-    if (i < H && delta) {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) rv[k][e] += p.dscale * v[k][e];
-      if (!p.rows) {
-        *reinterpret_cast<float4*>(res + i) = make_float4(rv[k][0], rv[k][1], rv[k][2], rv[k][3]);
-        *reinterpret_cast<float4*>(res + i + 4) = make_float4(rv[k][4], rv[k][5], rv[k][6], rv[k][7]);
-      }
-    }
-  }
-  const Moments m = block_moments(thread_moments<NV>(rv, H), scratch);
-  const float rstd = ln_rstd(m.m2, H, p.eps);
-  __nv_bfloat16* o = out + (int64_t)r * H;
-#pragma unroll
-  for (int k = 0; k < NV; ++k) {
-    const int i = (threadIdx.x + k * blockDim.x) * 8;
-    if (i < H) {
-      if (!AHEAD) {
-        ln_load8(p.w, p.w_dtype, i, w2);
-        ln_load8(p.b, p.w_dtype, i, b2);
-      }
-      uint4 q;
-      __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&q);
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        h[e] = __floats2bfloat162_rn((rv[k][2 * e] - m.mean) * rstd * w2[2 * e] + b2[2 * e],
-                                     (rv[k][2 * e + 1] - m.mean) * rstd * w2[2 * e + 1] + b2[2 * e + 1]);
-      *reinterpret_cast<uint4*>(o + i) = q;
     }
   }
 }
@@ -280,21 +269,15 @@ ATOM_EXPORT int atom_add_layernorm(void* out, int act_dtype, float* residual, co
   if (act_dtype == ATOM_BF16 && H % 8 == 0 && H <= 8 * 2 * 1024 && al(out) && al(residual) && al(delta) && al(w) && al(b) && al(wd) && al(bd) &&
       al(dbias)) {
     const int vecs = H / 8;
-    int nv = 1, th = ((vecs + 31) / 32) * 32;
-    if (th > 1024) {
-      nv = 2;
-      th = (((vecs + 1) / 2 + 31) / 32) * 32;
-    }
-    if (th < 64) th = 64;
-    if (nv == 1 && n_rows <= 2 * 148)
-      launch_pdl(add_layernorm_bf16_vec_kernel<1, true>, dim3(n_rows), dim3(th), 0, stream, (__nv_bfloat16*)out, residual,
-                 (const __nv_bfloat16*)delta, p);
-    else if (nv == 1)
-      launch_pdl(add_layernorm_bf16_vec_kernel<1, false>, dim3(n_rows), dim3(th), 0, stream, (__nv_bfloat16*)out, residual,
-                 (const __nv_bfloat16*)delta, p);
+    auto threads = [&](int nv) { return (((vecs + nv - 1) / nv + 31) / 32) * 32; };
+    const int nv = vecs <= 1024 ? 1 : 2, th = threads(nv);
+    const int grid = min(n_rows, 148 * max(1, 1024 / th));      // (64 registers a thread)
+    if (nv == 1)
+      launch_pdl(add_layernorm_bf16_vec_kernel<1>, dim3(grid), dim3(th), 0, stream, (__nv_bfloat16*)out, residual,
+                 (const __nv_bfloat16*)delta, p, n_rows);
     else
-      launch_pdl(add_layernorm_bf16_vec_kernel<2, false>, dim3(n_rows), dim3(th), 0, stream, (__nv_bfloat16*)out, residual,
-                 (const __nv_bfloat16*)delta, p);
+      launch_pdl(add_layernorm_bf16_vec_kernel<2>, dim3(grid), dim3(th), 0, stream, (__nv_bfloat16*)out, residual,
+                 (const __nv_bfloat16*)delta, p, n_rows);
     return check_launch();
   }
   if (H > kLnMaxRow) return ATOM_ERR_ARG;
