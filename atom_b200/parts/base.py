@@ -189,6 +189,7 @@ class ProjectedMixer(Mixer):
     out_bias = False
     inner_cols = 0
     hidden_size = 0
+    _where = None             # (where the segments lie in the projection, its width), formed at the first step
 
     def segments(self) -> Dict[str, Tuple[int, ...]]:
         raise NotImplementedError
@@ -234,7 +235,9 @@ class ProjectedMixer(Mixer):
 
         T = x.shape[0]
         ws, dt = self.rt.workspace, self.rt.dtype
-        _, where, width = self.layout(self.segments())
+        if self._where is None:
+            self._where = self.layout(self.segments())[1:]
+        where, width = self._where
         proj = linear(x, self.w_in_weight, None, ws.get("pm.in", (T, width), dt))
         y = ws.get("pm.y", (T, self.inner_cols), dt)
         self.inner(x, {n: proj[:, a:a + k] for n, (a, k) in where.items()}, step, cache, writes_cache, y, 1.0)

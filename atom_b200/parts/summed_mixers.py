@@ -84,7 +84,11 @@ class SummedMixers(ProjectedMixer):
 
     def inner(self, x, proj, step, cache, writes_cache, y, y_scale):
         at = 0
+        own_of = {n: {} for n in self.members}
+        for k, v in proj.items():
+            n, _, segment = k.partition(".")
+            own_of[n][segment] = v
         for n, m in self.members.items():
-            own = {k[len(n) + 1:]: v for k, v in proj.items() if k.startswith(n + ".")}
+            own = own_of[n]
             m.inner(x, own, step, cache.member(n), writes_cache, y[:, at:at + m.inner_cols], y_scale * self.scales[n])
             at += m.inner_cols
