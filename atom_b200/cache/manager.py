@@ -5,7 +5,7 @@ Cache slots (one per run-order entry that writes a cache) are grouped by what th
 keeps: (the arrays it holds per token, window).  A group has its own pool and its own block table
 per request; all slots of a group share the table (page id p means page p of every slot's
 storage in that group).  A group with a window gives pages back as soon as every position
-on them is further back than any later query can look; the pages of the first ``keep_first``
+on them is further back than any later query can look (with chunks: lies in a chunk that is over); the pages of the first ``keep_first``
 positions, which every later query still sees, stay.  A need that also keeps one row per whole block of
 positions (``CacheNeed.block_entries``) gets a second group for those rows: its pages hold ``page_size`` rows, a
 request of n positions has n // block of them, and no window gives them back.
@@ -47,6 +47,7 @@ class CacheGroup:
     entries: Tuple                   # the CacheEntry arrays every slot of the group holds per token
     slots: List[int]                 # cache slots (run-order cache ids) stored in this group
     pool: PagePool = None            # type: ignore
+    chunked: bool = False            # the window is a chunk: keys of the query's own chunk of positions are seen
     block: int = 0                   # > 0: the group holds one row per whole block of this many positions
 
 
@@ -91,7 +92,8 @@ class CacheManager:
             k = need.group_key()
             g = by_key.get(k)
             if g is None:
-                g = CacheGroup(len(self.groups), k, need.window, need.keep_first if need.window else 0, need.entries, [])
+                g = CacheGroup(len(self.groups), k, need.window, need.keep_first if need.window else 0, need.entries, [],
+                               chunked=bool(need.window) and need.chunked)
                 n = num_pages[k] if isinstance(num_pages, dict) else num_pages
                 g.pool = PagePool(n)
                 by_key[k] = g
@@ -124,7 +126,8 @@ class CacheManager:
         """Logical page below which no later query of the request can look."""
         if g.window is None:
             return 0
-        first_pos = committed - g.window + 1   # oldest key the next query (at `committed`) sees
+        # oldest key the next query (at `committed`) sees
+        first_pos = committed // g.window * g.window if g.chunked else committed - g.window + 1
         return max(0, first_pos) // self.page_size
 
     def _logical_pages(self, g: CacheGroup, n_tokens: int) -> int:

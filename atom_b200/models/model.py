@@ -13,7 +13,7 @@ import torch
 from .. import parts as _parts  # noqa: F401  (registers the built-in parts)
 from ..parts import registry
 from ..parts.base import Part, Runtime
-from ..parts.linear import NormedDelta, resolve
+from ..parts.linear import NormedDelta, SumDelta, resolve
 from ..parts.spec import CacheNeed, ModelSpec, PartSpec
 
 
@@ -128,6 +128,9 @@ class Model:
             block = self.blocks[e.layer]
             if e.add_step is not None:
                 self.stream_steps.add(residual, e.add_step)     # (sums commute: the pending delta is added by the next norm)
+            if isinstance(delta, SumDelta) and not getattr(block, "takes_sums", False):
+                delta.add_to(residual)
+                delta = None
             if not getattr(block, "takes_pending", False):
                 delta = resolve(delta)      # (a block may hand its last product on unrun)
             if delta is not None and (scale != 1.0 or getattr(block, "delta_scale", 1.0) != 1.0):
@@ -137,6 +140,9 @@ class Model:
             else:
                 delta = block.run(residual, delta, step, caches.get(e.cache), e.writes_cache)
             scale = getattr(block, "delta_scale", 1.0)
+        if isinstance(delta, SumDelta) and not getattr(self.final_norm, "fuses_sums", False):
+            delta.add_to(residual)
+            delta = None
         if not (isinstance(delta, NormedDelta) and getattr(self.final_norm, "fuses_products", False)):
             delta = resolve(delta)
         kw = {"delta_scale": scale} if scale != 1.0 else {}

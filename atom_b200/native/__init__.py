@@ -79,7 +79,12 @@ _SIGNATURES = {
     "atom_gla_supports": [_i, _i],
     "atom_gla_scan": [_vp, _vp, _vp, _vp, _i, _i64, _vp, _i64, _vp, _i, _f, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
                       _i, _i, _i, _vp],
-    "atom_gla_gate_norm": [_vp, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _i, _f, _vp, _vp],
+    "atom_gla_gate_norm": [_vp, _i64, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _i, _f, _vp, _i, _f, _vp],
+    "atom_add_dynamic_tanh": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _vp],
+    "atom_delta_supports": [_i, _i],
+    "atom_delta_prepare": [_vp, _vp, _vp, _i, _i64, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _i64, _vp, _vp, _vp, _vp, _i, _i,
+                           _i, _i, _i, _f, _f, _vp],
+    "atom_delta_scan": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "atom_pooled_attention_supports": [_i, _i, _i, _i],
     "atom_pooled_attention_split_supports": [_i, _i, _i, _i],
     "atom_pooled_attention_split": [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i,
@@ -115,11 +120,11 @@ _SIGNATURES = {
     "atom_gemm_bf16_batched": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _i64, _i64, _i64, _i64, _i64, _vp, _sz, _vp],
     "atom_relu2": [_vp, _i, _i64, _vp],
     "atom_conv_rope_write": [_vp, _vp, _i, _i64, _i, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i,
-                             _i, _vp, _vp, _i64, _vp, _vp, _i, _i, _f, _vp, _f, _vp, _vp],
+                             _i, _vp, _vp, _i64, _vp, _vp, _i, _i, _f, _vp, _f, _vp, _i, _vp, _vp, _i, _f, _vp],
     "atom_conv_state_update": [_vp, _vp, _i, _i64, _i, _i, _vp, _vp, _i, _vp],
-    "atom_window_attention_merge": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i64, _f, _i64, _vp],
+    "atom_window_attention_merge": [_vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i64, _f, _i64, _i, _f, _f, _vp],
     "atom_window_attention": [_vp, _vp, _i, _vp, _vp, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _i, _vp, _vp,
-                              _i64, _f, _i64, _vp],
+                              _i64, _f, _i64, _i, _i, _f, _f, _vp],
     "atom_lightning_supports": [_i, _i],
     "atom_lightning_scan": [_vp, _vp, _i, _i64, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "atom_lightning_gate_norm": [_vp, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _f, _vp, _vp],
@@ -837,21 +842,28 @@ def conv_rope_write(q_out: torch.Tensor, qkv: torch.Tensor, H: int, G: int, dk: 
                     k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor], status: torch.Tensor,
                     bias: Optional[torch.Tensor] = None, neighbours: bool = False, magnitude: float = 1.0,
                     v_first: Optional[torch.Tensor] = None, v_mix: float = 0.0,
-                    v_keep: Optional[torch.Tensor] = None) -> None:
+                    v_keep: Optional[torch.Tensor] = None, value_heads: Optional[int] = None,
+                    head_norms: Optional[tuple] = None) -> None:
     """Per token of the packed projection [q (H dk) | k (G dk) | v (G dv)]: the short causal convolution over time on
     every channel (conv_w [C, taps]; rows before the step from conv_state [slots, taps - 1, C], which is only read),
     rotation of the first rot_dims numbers of every query and key head by position * freq, queries to q_out
     [T, H dk], keys and values to their pages (csrc/window_attention.cu).  conv_w None: no convolution.  bias [C] is
     added to the projected channels (only without a convolution); neighbours: rotated pairs are (2i, 2i + 1) instead of
     (i, i + rot_dims / 2); magnitude: factor on cos and sin; v_first [T, G dv] dense: values become
-    (1 - v_mix) v + v_mix v_first; v_keep [T, G dv] takes a copy of the values."""
+    (1 - v_mix) v + v_mix v_first; v_keep [T, G dv] takes a copy of the values.  value_heads: value heads where there are
+    not G of them (0, like G = 0, for rows that hold queries only); head_norms (wq, wk, eps): every query and key head is
+    divided by its root mean square and multiplied by wq or wk [dk] before the rotation (only without a convolution)."""
+    GV = G if value_heads is None else value_heads
+    wq, wk, norm_eps = head_norms if head_norms is not None else (None, None, 0.0)
+    _cuda(wq, wk)
+    assert wq is None or (conv_w is None and wq.numel() == dk and (G == 0 or (wk.numel() == dk and wk.dtype == wq.dtype)))
     _cuda(q_out, qkv, conv_w, conv_state, freq, positions, seq_of_token, cu_q, state_slots, block_table, k_pages,
           v_pages, status, bias, v_first, v_keep)
-    assert bias is None or (conv_w is None and bias.numel() >= (H + G) * dk + G * dv and bias.is_contiguous())
+    assert bias is None or (conv_w is None and bias.numel() >= (H + G) * dk + GV * dv and bias.is_contiguous())
     for vt in (v_first, v_keep):
-        assert vt is None or (vt.is_contiguous() and vt.dtype == qkv.dtype and vt.shape == (qkv.shape[0], G * dv))
+        assert vt is None or (vt.is_contiguous() and vt.dtype == qkv.dtype and vt.shape == (qkv.shape[0], GV * dv))
     T = qkv.shape[0]
-    C = (H + G) * dk + G * dv
+    C = (H + G) * dk + GV * dv
     taps = 0 if conv_w is None else conv_w.shape[1]
     assert qkv.stride(1) == 1 and qkv.shape[1] >= C and q_out.is_contiguous() and q_out.shape == (T, H * dk)
     assert q_out.dtype == qkv.dtype and block_table.dtype == torch.int32 and block_table.is_contiguous()
@@ -860,7 +872,7 @@ def conv_rope_write(q_out: torch.Tensor, qkv: torch.Tensor, H: int, G: int, dk: 
                          and tuple(conv_state.shape[1:]) == (taps - 1, C))
     assert rot_dims == 0 or (freq is not None and freq.dtype == torch.float32 and freq.numel() >= rot_dims // 2)
     if k_pages is not None:
-        assert tuple(k_pages.shape[1:]) == (G, page_size, dk) and tuple(v_pages.shape[1:]) == (G, page_size, dv)
+        assert tuple(k_pages.shape[1:]) == (G, page_size, dk) and tuple(v_pages.shape[1:]) == (GV, page_size, dv)
         assert k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.dtype == v_pages.dtype == qkv.dtype
     _check(lib().atom_conv_rope_write(
         q_out.data_ptr(), qkv.data_ptr(), dtype_code(qkv.dtype), qkv.stride(0), T, H, G, dk, dv, _ptr(conv_w),
@@ -869,7 +881,8 @@ def conv_rope_write(q_out: torch.Tensor, qkv: torch.Tensor, H: int, G: int, dk: 
         block_table.data_ptr(), block_table.shape[1], page_size, _ptr(k_pages), _ptr(v_pages),
         k_pages.shape[0] if k_pages is not None else 0, status.data_ptr(), _ptr(bias),
         dtype_code(bias.dtype) if bias is not None else F32, int(neighbours), float(magnitude), _ptr(v_first),
-        float(v_mix), _ptr(v_keep), _stream()), "conv_rope_write")
+        float(v_mix), _ptr(v_keep), GV, _ptr(wq), _ptr(wk), dtype_code(wq.dtype) if wq is not None else F32,
+        float(norm_eps), _stream()), "conv_rope_write")
 
 
 def conv_state_update(conv_state: torch.Tensor, qkv: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
@@ -887,24 +900,30 @@ def window_attention(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tensor, 
                      block_table: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor, nh: int, nkv: int,
                      dk: int, dv: int, scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0,
                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                     out_scale: float = 1.0) -> None:
+                     out_scale: float = 1.0, chunked: bool = False, maps: Optional[tuple] = None) -> None:
     """Causal paged attention, key j seen from position p if j <= p and (p - j < window or j < keep_first); scores
     scale * q.k, then softcap * tanh(score / softcap) if softcap > 0.  q [T, nh dk], out [T, nh dv] (rows may lie further
     apart), any sizes, both precisions (csrc/window_attention.cu).  sink [nh] float32: exp(sink_h) is added to the
-    denominator; gate [T, nh] (a view, activation type): the output times sigmoid(gate); out_scale: times a constant."""
+    denominator; gate [T, nh] (a view, activation type): the output times sigmoid(gate); out_scale: times a constant.
+    chunked: the window is a chunk, keys j <= p with j // window = p // window.  maps (lambda, eps): differential attention,
+    q [T, nh 2 dk] with two queries per head, k_pages with two keys per key head: the first map's output minus lambda times
+    the second's, divided by its root mean square (over dv, eps inside the root)."""
+    n_maps, lam, maps_eps = (2,) + tuple(maps) if maps is not None else (1, 0.0, 0.0)
     _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token, sink, gate)
     _attention_extras(sink, gate, nh, q)
     T = q.shape[0]
     page_size = k_pages.shape[2]
-    assert q.is_contiguous() and out.stride(1) == 1 and q.shape == (T, nh * dk) and out.shape == (T, nh * dv)
+    assert q.is_contiguous() and out.stride(1) == 1 and q.shape == (T, nh * n_maps * dk) and out.shape == (T, nh * dv)
+    assert maps is None or sink is None
     assert out.dtype == q.dtype == k_pages.dtype == v_pages.dtype and k_pages.is_contiguous() and v_pages.is_contiguous()
-    assert tuple(k_pages.shape[1:]) == (nkv, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
+    assert tuple(k_pages.shape[1:]) == (nkv * n_maps, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
     assert block_table.dtype == torch.int32 and block_table.is_contiguous()
     _check(lib().atom_window_attention(
         out.data_ptr(), q.data_ptr(), dtype_code(q.dtype), k_pages.data_ptr(), v_pages.data_ptr(),
         block_table.data_ptr(), block_table.shape[1], page_size, positions.data_ptr(), seq_of_token.data_ptr(), T, nh,
         nkv, dk, dv, float(scale), float(softcap or 0.0), int(window or 0), int(keep_first), _ptr(sink), _ptr(gate),
-        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), _stream()), "window_attention")
+        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), int(chunked), n_maps, float(lam),
+        float(maps_eps), _stream()), "window_attention")
 
 
 def _attention_extras(sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], nh: int, q: torch.Tensor) -> None:
@@ -916,29 +935,34 @@ def _attention_extras(sink: Optional[torch.Tensor], gate: Optional[torch.Tensor]
 # first use
 _watc_libs = {}
 _WATC_SIG = [_vp, _vp, _i64, _vp, _vp, _i64, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _i, _i, _vp, _i, _vp,
-             _vp, _i64, _f, _i64, _vp]
+             _vp, _i64, _f, _i64, _i, _f, _f, _vp]
 WINDOW_TC = True     # False: the plain kernel also where the tensor-core kernel takes the sizes (measurements, tests)
 WINDOW_TC_ROWS = 64  # query rows of a tile
 
 
-def window_attention_tc_supports(dk: int, dv: int, dtype: torch.dtype) -> bool:
+def window_attention_tc_supports(dk: int, dv: int, dtype: torch.dtype, maps: int = 1) -> bool:
     """bfloat16; key and value sizes in steps of 16, keys up to 256 and values up to 128 numbers (a warp keeps its
-    16 x value size output in registers)."""
-    return dtype == torch.bfloat16 and dk % 16 == 0 and dv % 16 == 0 and 16 <= dk <= 256 and 16 <= dv <= 128
+    16 x value size output in registers), queries, keys and values of two stages within shared memory."""
+    smem = 2 * (maps * 64 * (dk + 8) + 2 * (maps * 64 * (dk + 8) + 64 * (dv + 8)))
+    return (dtype == torch.bfloat16 and dk % 16 == 0 and dv % 16 == 0 and 16 <= dk <= 256 and 16 <= dv <= 128
+            and smem <= 227 * 1024)
 
 
-def watc_lib(dk: int, dv: int):
-    key = (dk, dv)
+def watc_lib(dk: int, dv: int, maps: int = 1):
+    key = (dk, dv, maps)
     l = _watc_libs.get(key)
     if l is None:
         with _lock:
             l = _watc_libs.get(key)
             if l is None:
-                path = build_variant("window_attention_tc.cu", {"ATOM_WA_DK": dk, "ATOM_WA_DV": dv})
+                defines = {"ATOM_WA_DK": dk, "ATOM_WA_DV": dv}
+                if maps != 1:
+                    defines["ATOM_WA_MAPS"] = maps
+                path = build_variant("window_attention_tc.cu", defines)
                 l = ctypes.CDLL(path)
                 l.atom_window_attention_tc.argtypes = _WATC_SIG
                 l.atom_window_attention_tc.restype = ctypes.c_int
-                got = [ctypes.c_int() for _ in range(2)]
+                got = [ctypes.c_int() for _ in range(3)]
                 l.atom_watc_sizes(*[ctypes.byref(g) for g in got])
                 if tuple(g.value for g in got) != key:
                     raise NativeBuildError(f"{path} was built for other sizes")
@@ -952,7 +976,7 @@ def window_attention_tc(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tenso
                         softcap: float = 0.0, window: int = 0, keep_first: int = 0, nsplit: int = 1,
                         scratch: Optional[torch.Tensor] = None, heads_rows: bool = False,
                         sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                        out_scale: float = 1.0) -> None:
+                        out_scale: float = 1.0, chunked: bool = False, maps: Optional[tuple] = None) -> None:
     """``window_attention`` on the tensor cores: tiles of 64 consecutive tokens of a request and one head (cu_q:
     [num_seqs + 1] first token row of every request); with nsplit > 1 a tile's keys are shared out among nsplit
     CTAs and put together by a merge kernel.  heads_rows (only for steps in which every request brings ONE token, and
@@ -960,28 +984,31 @@ def window_attention_tc(out: torch.Tensor, q: torch.Tensor, k_pages: torch.Tenso
     keys and values are read once per key head.  Sizes as ``window_attention_tc_supports``."""
     _cuda(out, q, k_pages, v_pages, block_table, positions, seq_of_token, cu_q, scratch, sink, gate)
     _attention_extras(sink, gate, nh, q)
+    n_maps, lam, maps_eps = (2,) + tuple(maps) if maps is not None else (1, 0.0, 0.0)
+    assert maps is None or sink is None
     T = q.shape[0]
     page_size = k_pages.shape[2]
-    assert q.stride(1) == 1 and q.shape[1] == nh * dk and out.stride(1) == 1 and out.shape == (T, nh * dv)
+    assert q.stride(1) == 1 and q.shape[1] == nh * n_maps * dk and out.stride(1) == 1 and out.shape == (T, nh * dv)
     assert out.dtype == q.dtype == k_pages.dtype == v_pages.dtype == torch.bfloat16
-    assert tuple(k_pages.shape[1:]) == (nkv, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
+    assert tuple(k_pages.shape[1:]) == (nkv * n_maps, page_size, dk) and tuple(v_pages.shape[1:]) == (nkv, page_size, dv)
     assert k_pages.is_contiguous() and v_pages.is_contiguous() and cu_q.numel() >= num_seqs + 1
     assert block_table.dtype == torch.int32 and block_table.is_contiguous()
     assert nsplit == 1 or (scratch is not None and scratch.dtype == torch.float32
-                           and scratch.numel() >= attention_mixed_scratch_elems(T, nh, dv, nsplit))
+                           and scratch.numel() >= attention_mixed_scratch_elems(T, nh * n_maps, dv, nsplit))
     assert not heads_rows or nh // nkv <= WINDOW_TC_ROWS
     units = T if heads_rows else -(-T // WINDOW_TC_ROWS) + num_seqs
-    _check(watc_lib(dk, dv).atom_window_attention_tc(
+    _check(watc_lib(dk, dv, n_maps).atom_window_attention_tc(
         out.data_ptr(), q.data_ptr(), q.stride(0), k_pages.data_ptr(), v_pages.data_ptr(), k_pages.shape[0],
         block_table.data_ptr(), block_table.shape[1], page_size, positions.data_ptr(), seq_of_token.data_ptr(),
         cu_q.data_ptr(), num_seqs, units, nh, nkv, float(scale), float(softcap or 0.0), int(window or 0),
         int(keep_first), int(nsplit), _ptr(scratch) if nsplit > 1 else None, int(heads_rows), _ptr(sink), _ptr(gate),
-        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), _stream()), "window_attention_tc")
+        gate.stride(0) if gate is not None else 0, float(out_scale), out.stride(0), int(chunked), float(lam),
+        float(maps_eps), _stream()), "window_attention_tc")
     if nsplit > 1:
         _check(lib().atom_window_attention_merge(out.data_ptr(), dtype_code(out.dtype), scratch.data_ptr(),
                                                  seq_of_token.data_ptr(), T, nh, dv, nsplit, _ptr(sink), _ptr(gate),
                                                  gate.stride(0) if gate is not None else 0, float(out_scale),
-                                                 out.stride(0), _stream()),
+                                                 out.stride(0), n_maps, float(lam), float(maps_eps), _stream()),
                "window_attention_merge")
 
 
@@ -1578,6 +1605,23 @@ def layernorm(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, bias: to
            "layernorm")
 
 
+def add_dynamic_tanh(out: torch.Tensor, residual: torch.Tensor, d0: Optional[torch.Tensor], d1: Optional[torch.Tensor],
+                     weight: torch.Tensor, bias: torch.Tensor, alpha: float, rows: Optional[torch.Tensor] = None,
+                     n_rows: Optional[int] = None) -> None:
+    """residual (+= d0) (+= d1); out = tanh(alpha * residual) * weight + bias, one kernel, 32-bit.  With ``rows`` only those
+    rows, written densely, and residual is left as it is."""
+    _cuda(out, residual, d0, d1, weight, bias, rows)
+    H = residual.shape[-1]
+    assert residual.dtype == torch.float32 and residual.is_contiguous() and out.is_contiguous() and out.shape[-1] == H
+    n = (rows.numel() if n_rows is None else n_rows) if rows is not None else residual.shape[0]
+    for d in (d0, d1):
+        assert d is None or (d.dtype == out.dtype and d.is_contiguous() and d.shape == residual.shape)
+    assert weight.dtype == bias.dtype and weight.numel() == bias.numel() == H and out.shape[0] >= n
+    _check(lib().atom_add_dynamic_tanh(out.data_ptr(), dtype_code(out.dtype), residual.data_ptr(), _ptr(d0), _ptr(d1),
+                                       weight.data_ptr(), bias.data_ptr(), dtype_code(weight.dtype), float(alpha),
+                                       _ptr(rows), n, H, _stream()), "add_dynamic_tanh")
+
+
 def head_gate(x: torch.Tensor, g: torch.Tensor) -> None:
     """x[t, h, :] *= sigmoid(g[t, h]); x [T, H, n] dense, g [T, H] a view whose rows may lie further apart."""
     _cuda(x, g)
@@ -1642,16 +1686,71 @@ def gla_scan(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tenso
 
 
 def gla_gate_norm(y: torch.Tensor, o: torch.Tensor, g: torch.Tensor, w: torch.Tensor, eps: float, H: int, dv: int,
-                  seq_of_token: torch.Tensor) -> None:
-    """y[t, h] = o[t, h] / rms(o[t, h]) * w * silu(g[t, h]): the norm runs over one head's columns, w [dv] is shared by
-    the heads.  o float32 [T, H dv]; g a view whose rows may lie further apart."""
+                  seq_of_token: torch.Tensor, gate: str = "silu", out_scale: float = 1.0) -> None:
+    """y[t, h] = o[t, h] / rms(o[t, h]) * w * gate(g[t, h]) * out_scale: the norm runs over one head's columns, w [dv] is
+    shared by the heads; gate "silu" or "sigmoid".  o float32 [T, H dv]; y and g may be views whose rows lie further apart."""
     _cuda(y, o, g, w, seq_of_token)
     T = o.shape[0]
-    assert o.dtype == torch.float32 and o.is_contiguous() and y.is_contiguous() and y.shape == o.shape == (T, H * dv)
+    assert gate in ("silu", "sigmoid")
+    assert o.dtype == torch.float32 and o.is_contiguous() and y.stride(1) == 1 and y.shape == o.shape == (T, H * dv)
     assert g.dtype == y.dtype and g.stride(1) == 1 and g.shape == (T, H * dv) and w.numel() == dv
-    _check(lib().atom_gla_gate_norm(y.data_ptr(), o.data_ptr(), g.data_ptr(), dtype_code(y.dtype), g.stride(0),
+    _check(lib().atom_gla_gate_norm(y.data_ptr(), y.stride(0), o.data_ptr(), g.data_ptr(), dtype_code(y.dtype), g.stride(0),
                                     w.data_ptr(), dtype_code(w.dtype), T, H, dv, float(eps), seq_of_token.data_ptr(),
-                                    _stream()), "gla_gate_norm")
+                                    int(gate == "sigmoid"), float(out_scale), _stream()), "gla_gate_norm")
+
+
+# ------------------------------------------------------------------ gated delta rule with a decay per key channel
+
+def delta_supports(dk: int, dv: int) -> bool:
+    return bool(lib().atom_delta_supports(dk, dv))
+
+
+def delta_lanes(dk: int) -> int:
+    """Lanes that share a column of the state in ``delta_scan``."""
+    return 4 if dk <= 32 else 8
+
+
+def delta_prepare(u: torch.Tensor, rn: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor],
+                  z: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, beta_in: torch.Tensor, beta: torch.Tensor,
+                  seq_of_token: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, G: int, H: int, dk: int,
+                  dv: int, q_scale: float, unit_eps: float) -> None:
+    """What enters the delta rule, per token: u [T, C] = silu(short causal convolution of x [T, C] with w [C, taps]), channels
+    [q (G dk) | k (G dk) | v (H dv)], rows before the step from ``state`` [slots, taps - 1, C] (only read); rn [T, 2 G]
+    float32 the factors that make q and k heads unit vectors (queries' times q_scale); z [T, H dk] float32 becomes
+    -exp(A_log) softplus(z + dt_bias) log2(e); beta [T, H] float32 = sigmoid(beta_in)."""
+    _cuda(u, rn, x, w, state, z, A_log, dt_bias, beta_in, beta, seq_of_token, cu_q, state_slots)
+    T, C = x.shape
+    taps = w.shape[1]
+    assert C == 2 * G * dk + H * dv and x.stride(1) == 1 and u.is_contiguous() and u.shape == (T, C) and u.dtype == x.dtype
+    assert tuple(w.shape) == (C, taps) and w.is_contiguous() and A_log.dtype == dt_bias.dtype
+    assert A_log.numel() == H and dt_bias.numel() == H * dk and A_log.is_contiguous() and dt_bias.is_contiguous()
+    assert taps == 1 or (state.is_contiguous() and state.dtype == x.dtype and tuple(state.shape[1:]) == (taps - 1, C))
+    for t, n in ((rn, 2 * G), (z, H * dk), (beta, H)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n)
+    assert beta_in.dtype == x.dtype and beta_in.stride(1) == 1 and beta_in.shape == (T, H)
+    _check(lib().atom_delta_prepare(u.data_ptr(), rn.data_ptr(), x.data_ptr(), dtype_code(x.dtype), x.stride(0), w.data_ptr(),
+                                    dtype_code(w.dtype), taps, _ptr(state) if taps > 1 else None, z.data_ptr(),
+                                    A_log.data_ptr(), dt_bias.data_ptr(), dtype_code(A_log.dtype), beta_in.data_ptr(),
+                                    beta_in.stride(0), beta.data_ptr(), seq_of_token.data_ptr(), cu_q.data_ptr(),
+                                    state_slots.data_ptr(), T, G, H, dk, dv, float(q_scale), float(unit_eps), _stream()),
+           "delta_prepare")
+
+
+def delta_scan(out: torch.Tensor, u: torch.Tensor, rn: torch.Tensor, la: torch.Tensor, beta: torch.Tensor,
+               state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, G: int, H: int, dk: int,
+               dv: int, write_state: bool = True, lanes: Optional[int] = None) -> None:
+    """out[t] (float32 [T, H dv]) = S^T q_t with S <- diag(2^la_t) S, then S <- S + k_t (beta_t (v_t - S^T k_t))^T, row by row
+    over every request's rows; u, rn, la, beta as ``delta_prepare`` leaves them; state [slots, H, dk, dv] float32."""
+    _cuda(out, u, rn, la, beta, state, cu_q, state_slots)
+    T, C = u.shape
+    assert C == 2 * G * dk + H * dv and u.is_contiguous() and out.dtype == torch.float32
+    assert out.is_contiguous() and out.shape == (T, H * dv)
+    for t, n in ((rn, 2 * G), (la, H * dk), (beta, H)):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n)
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dk, dv)
+    _check(lib().atom_delta_scan(out.data_ptr(), u.data_ptr(), dtype_code(u.dtype), rn.data_ptr(), la.data_ptr(),
+                                 beta.data_ptr(), state.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, G,
+                                 H, dk, dv, lanes or delta_lanes(dk), int(write_state), _stream()), "delta_scan")
 
 
 # ------------------------------------------------------------------ state-space duality (Mamba-2)

@@ -16,7 +16,8 @@
 // the step's rows alone and changes only the order of 32-bit roundings.  In steps that are cut into runs every CTA
 // of both walks would form the same decays again, so a kernel of its own turns z into the decays in place first.
 //
-//   gla_gate_norm_kernel   y = o / rms(o over a head's columns) * w * silu(g), w shared by the heads
+//   gla_gate_norm_kernel   y = o / rms(o over a head's columns) * w * silu(g) (or sigmoid(g)) * out_scale, w shared by the
+//                          heads
 #include "common.cuh"
 
 namespace atom {
@@ -200,11 +201,11 @@ __global__ void gla_prefix_kernel(float* __restrict__ state, float* __restrict__
   }
 }
 
-// y[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * silu(g[t, h, :]); a warp per (token, head).
-template <typename T>
-__global__ void gla_gate_norm_kernel(T* __restrict__ y, const float* __restrict__ o, const T* __restrict__ g, int64_t ldg,
+// y[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(g[t, h, :]) * out_scale; a warp per (token, head).
+template <typename T, bool SIGMOID>
+__global__ void gla_gate_norm_kernel(T* __restrict__ y, int64_t ldy, const float* __restrict__ o, const T* __restrict__ g, int64_t ldg,
                                      const void* __restrict__ w, int w_dtype, int H, int dv, float eps,
-                                     const int* __restrict__ seq_of_token) {
+                                     const int* __restrict__ seq_of_token, float out_scale) {
   atom::pdl_trigger();
   atom::pdl_wait();
   const int t = blockIdx.x;
@@ -215,11 +216,11 @@ __global__ void gla_gate_norm_kernel(T* __restrict__ y, const float* __restrict_
     float ss = 0.f;
     for (int i = lane; i < dv; i += 32) ss = fmaf(orow[i], orow[i], ss);
     ss = warp_sum(ss);
-    const float rstd = rsqrtf(ss / (float)dv + eps);
+    const float rstd = rsqrtf(ss / (float)dv + eps) * out_scale;
     for (int i = lane; i < dv; i += 32) {
       const float gg = to_float(g[(int64_t)t * ldg + (int64_t)h * dv + i]);
-      y[((int64_t)t * H + h) * dv + i] =
-          from_float<T>(orow[i] * rstd * load_as_float(w, w_dtype, i) * (gg / (1.f + expf(-gg))));
+      y[(int64_t)t * ldy + (int64_t)h * dv + i] =
+          from_float<T>(orow[i] * rstd * load_as_float(w, w_dtype, i) * ((SIGMOID ? 1.f : gg) / (1.f + expf(-gg))));
     }
   }
 }
@@ -303,19 +304,23 @@ ATOM_EXPORT int atom_gla_scan(float* out, const void* q, const void* k, const vo
   return ATOM_ERR_ARG;
 }
 
-ATOM_EXPORT int atom_gla_gate_norm(void* y, const float* o, const void* g, int dtype, int64_t ldg, const void* w,
-                                   int w_dtype, int T, int H, int dv, float eps, const int* seq_of_token,
-                                   cudaStream_t stream) {
+ATOM_EXPORT int atom_gla_gate_norm(void* y, int64_t ldy, const float* o, const void* g, int dtype, int64_t ldg, const void* w,
+                                   int w_dtype, int T, int H, int dv, float eps, const int* seq_of_token, int sigmoid,
+                                   float out_scale, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  if (H <= 0 || dv <= 0 || (w_dtype != ATOM_F32 && w_dtype != ATOM_BF16)) return ATOM_ERR_ARG;
-  const int threads = H >= 8 ? 256 : 32 * H;
-  if (dtype == ATOM_F32)
-    atom::launch_pdl(atom::gla_gate_norm_kernel<float>, dim3(T), dim3(threads), 0, stream, (float*)y, o, (const float*)g,
-                     ldg, w, w_dtype, H, dv, eps, seq_of_token);
-  else if (dtype == ATOM_BF16)
-    atom::launch_pdl(atom::gla_gate_norm_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, (__nv_bfloat16*)y, o,
-                     (const __nv_bfloat16*)g, ldg, w, w_dtype, H, dv, eps, seq_of_token);
-  else
+  if (H <= 0 || dv <= 0 || (w_dtype != ATOM_F32 && w_dtype != ATOM_BF16) || (dtype != ATOM_F32 && dtype != ATOM_BF16))
     return ATOM_ERR_ARG;
+  const int threads = H >= 8 ? 256 : 32 * H;
+#define ATOM_GN(TT, SIG)                                                                                               \
+  atom::launch_pdl(atom::gla_gate_norm_kernel<TT, SIG>, dim3(T), dim3(threads), 0, stream, (TT*)y, ldy, o, (const TT*)g, \
+                   ldg, w, w_dtype, H, dv, eps, seq_of_token, out_scale)
+  if (dtype == ATOM_F32) {
+    if (sigmoid) ATOM_GN(float, true);
+    else ATOM_GN(float, false);
+  } else {
+    if (sigmoid) ATOM_GN(__nv_bfloat16, true);
+    else ATOM_GN(__nv_bfloat16, false);
+  }
+#undef ATOM_GN
   return atom::check_launch();
 }

@@ -8,14 +8,19 @@
 //                             numbers of every query and key head by position * frequency (pairs (i, i + rot_dims/2),
 //                             or neighbours (2i, 2i + 1)), cos and sin times a constant; optionally a bias on every
 //                             channel (without a convolution), and values blended with another layer's values of
-//                             the same token, v <- (1 - mix) v + mix v_first; q to a dense array, k and v to their
-//                             pages (conv_rope_write_vec_kernel: the same for bfloat16 sizes in steps of 8, 16 bytes
-//                             at a time)
+//                             the same token, v <- (1 - mix) v + mix v_first; optionally every query and key head
+//                             divided by its root mean square and times a weight before the rotation; q to a dense
+//                             array, k and v to their pages (conv_rope_write_vec_kernel: the same for bfloat16 sizes
+//                             in steps of 8, 16 bytes at a time).  Keys and values may have head counts of their own.
 //   conv_state_update_kernel  per request: the last taps - 1 projected rows after this step
 //   window_attention_kernel   one CTA per (token, query head): keys j <= p with p - j < window or j < keep_first,
 //                             s = scale * q.k, s <- cap * tanh(s / cap), online softmax in 32-bit; any sizes, both
 //                             precisions; optionally a sink per head (exp(sink_h) is added to the denominator), a
-//                             gate number per head (the output times sigmoid(gate)) and a constant on the output
+//                             gate number per head (the output times sigmoid(gate)) and a constant on the output.
+//                             A window may also be a chunk: keys j <= p with j / window = p / window.
+//                             With two maps (differential attention) every head has two queries and every key head two
+//                             keys, [map 1, map 2], over the same values: o = a1 - lambda a2 with a1, a2 the two maps'
+//                             outputs, divided by its root mean square over the value size
 // Convolution sums, angles, scores, weights and sums are 32-bit in both precisions.
 #include "common.cuh"
 
@@ -48,7 +53,12 @@ struct RopeExtras {
   float mag;             // factor on cos and sin
   const void* v_first;   // [T, G dv] dense, activation type: values to blend in (null: none)
   float v_mix;
-  void* v_keep;          // [T, G dv] dense: takes a copy of this layer's values (null: none)
+  void* v_keep;          // [T, GV dv] dense: takes a copy of this layer's values (null: none)
+  int GV;                // value heads
+  const void* wq;        // [dk] weights of the norm of every query and key head (null: none)
+  const void* wk;
+  int norm_dtype;
+  float norm_eps;
 };
 
 template <typename T>
@@ -67,7 +77,7 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
   if (s < 0) return;
   const int p = positions[t];
   const int first = cu_q[s];
-  const int C = H * dk + G * dk + G * dv;
+  const int C = H * dk + G * dk + x.GV * dv;
   const T* state_row = (conv_state && taps > 1) ? conv_state + (int64_t)state_slots[s] * (taps - 1) * C : nullptr;
   const int lp = p / page_size;
   const int page = lp < max_pages ? block_table[(int64_t)s * max_pages + lp] : -1;
@@ -84,22 +94,40 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
     if (x.bias) y += load_as_float(x.bias, x.bias_dtype, c);
     return y;
   };
+  extern __shared__ __align__(16) float cr_factor[];      // [H + G] with a norm: 1 / root mean square
+  if (x.wq) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int n = warp; n < H + G; n += blockDim.x >> 5) {
+      float ss = 0.f;
+      for (int i = lane; i < dk; i += 32) {
+        const float y = value_at(n * dk + i);
+        ss = fmaf(y, y, ss);
+      }
+      ss = warp_sum(ss);
+      if (lane == 0) cr_factor[n] = rsqrtf(ss / (float)dk + x.norm_eps);
+    }
+    __syncthreads();
+  }
+  auto normed_at = [&](int n, int i) {
+    float y = value_at(n * dk + i);
+    if (x.wq) y *= cr_factor[n] * load_as_float(n < H ? x.wq : x.wk, x.norm_dtype, i);
+    return y;
+  };
   // queries and keys: H + G vectors of dk numbers
   for (int idx = threadIdx.x; idx < (H + G) * dk; idx += blockDim.x) {
     const int n = idx / dk, i = idx - n * dk;
     if (x.neighbours ? (i < rot_dims && (i & 1)) : (i >= half && i < rot_dims)) continue;   // written by the pair's first
-    const int c = n * dk + i;                      // (keys follow the queries in the row)
-    T* dst;
+    T* dst;                                        // (keys follow the queries in the row)
     if (n < H) {
       dst = q_out + ((int64_t)t * H + n) * dk;
     } else {
       if (!writes) continue;
       dst = k_pages + (((int64_t)page * G + (n - H)) * page_size + slot) * dk;
     }
-    const float a = value_at(c);
+    const float a = normed_at(n, i);
     if (i < rot_dims) {
       const int other = x.neighbours ? 1 : half;
-      const float b = value_at(c + other);
+      const float b = normed_at(n, i + other);
       float sn, cs;
       sincosf(pos * freq[x.neighbours ? i >> 1 : i], &sn, &cs);
       sn *= x.mag;
@@ -111,12 +139,12 @@ conv_rope_write_kernel(T* __restrict__ q_out, const T* __restrict__ qkv, int64_t
     }
   }
   const int v0 = (H + G) * dk;
-  for (int idx = threadIdx.x; idx < G * dv; idx += blockDim.x) {
+  for (int idx = threadIdx.x; idx < x.GV * dv; idx += blockDim.x) {
     const int g = idx / dv, i = idx - g * dv;
     float v = value_at(v0 + idx);
-    if (x.v_first) v = (1.f - x.v_mix) * v + x.v_mix * to_float(((const T*)x.v_first)[(int64_t)t * G * dv + idx]);
-    if (x.v_keep) ((T*)x.v_keep)[(int64_t)t * G * dv + idx] = from_float<T>(v);
-    if (writes) v_pages[(((int64_t)page * G + g) * page_size + slot) * dv + i] = from_float<T>(v);
+    if (x.v_first) v = (1.f - x.v_mix) * v + x.v_mix * to_float(((const T*)x.v_first)[(int64_t)t * x.GV * dv + idx]);
+    if (x.v_keep) ((T*)x.v_keep)[(int64_t)t * x.GV * dv + idx] = from_float<T>(v);
+    if (writes) v_pages[(((int64_t)page * x.GV + g) * page_size + slot) * dv + i] = from_float<T>(v);
   }
 }
 
@@ -136,13 +164,13 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
                            int* __restrict__ status, const RopeExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
-  extern __shared__ __align__(16) float cv_y[];      // [C], then cos and sin of the rotated pairs
+  extern __shared__ __align__(16) float cv_y[];      // [C], cos and sin of the rotated pairs
   const int t = blockIdx.x;
   const int s = seq_of_token[t];
   if (s < 0) return;
   const int p = positions[t];
   const int first = cu_q[s];
-  const int C = H * dk + G * dk + G * dv;
+  const int C = H * dk + G * dk + x.GV * dv;
   const __nv_bfloat16* state_row =
       (conv_state && TAPS > 1) ? conv_state + (int64_t)state_slots[s] * (TAPS - 1) * C : nullptr;
   const int lp = p / page_size;
@@ -216,6 +244,17 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
   }
   __syncthreads();
   const int qk_end = (H + G) * dk;
+  if (x.wq) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int n = warp; n < H + G; n += blockDim.x >> 5) {
+      float ss = 0.f;
+      for (int i = lane; i < dk; i += 32) ss = fmaf(cv_y[n * dk + i], cv_y[n * dk + i], ss);
+      ss = warp_sum(ss);
+      const float f = rsqrtf(ss / (float)dk + x.norm_eps);
+      for (int i = lane; i < dk; i += 32) cv_y[n * dk + i] *= f * load_as_float(n < H ? x.wq : x.wk, x.norm_dtype, i);
+    }
+    __syncthreads();
+  }
   for (int g = threadIdx.x; g < groups; g += blockDim.x) {
     const int c = g * 8;
     __nv_bfloat16* dst;
@@ -237,8 +276,8 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
       if (!writes && !x.v_keep) continue;
       const int idx = c - qk_end;
       const int gg = idx / dv;
-      keep_at = (int64_t)t * G * dv + idx;
-      dst = writes ? v_pages + (((int64_t)page * G + gg) * page_size + slot) * dv + (idx - gg * dv) : nullptr;
+      keep_at = (int64_t)t * x.GV * dv + idx;
+      dst = writes ? v_pages + (((int64_t)page * x.GV + gg) * page_size + slot) * dv + (idx - gg * dv) : nullptr;
     }
     if (rotated && x.neighbours) {
 #pragma unroll
@@ -305,7 +344,15 @@ struct AttnExtras {
   int64_t gate_ld;
   float out_mul;
   int64_t out_ld;
+  int chunked;           // 1: the window is a chunk, keys j <= p with j / window = p / window
+  float lambda, maps_eps;     // with two maps: the second map's weight, and what is added to the mean square
 };
+
+// First key that position p sees (kept first tokens apart).
+__device__ __forceinline__ int attn_first_key(int p, int window, int chunked) {
+  if (window <= 0) return 0;
+  return chunked ? p / window * window : max(0, p - window + 1);
+}
 
 template <typename T>
 __device__ __forceinline__ float attn_out_factor(const AttnExtras& x, int t, int h) {
@@ -317,7 +364,9 @@ __device__ __forceinline__ float attn_out_factor(const AttnExtras& x, int t, int
 constexpr int kWinThreads = 128;
 constexpr int kWinChunk = 256;
 
-template <typename T>
+// nh heads; with MAPS maps a head has MAPS queries in a row and a key head MAPS keys: q [T, nh MAPS dk], k_pages
+// [pages, nkv MAPS, page, dk], v_pages [pages, nkv, page, dv].
+template <typename T, int MAPS>
 __global__ void __launch_bounds__(kWinThreads)
 window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ k_pages,
                         const T* __restrict__ v_pages, const int* __restrict__ block_table, int max_pages,
@@ -327,7 +376,7 @@ window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   atom::pdl_trigger();
   atom::pdl_wait();
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  int64_t* row_of = (int64_t*)smem_raw;            // [kWinChunk] (page * nkv + g) * page_size + slot of a key
+  int64_t* row_of = (int64_t*)smem_raw;            // [kWinChunk] (page * nkv + g) * page_size + slot of a key's value
   float* prob = (float*)(row_of + kWinChunk);      // [kWinChunk]
   float* qs = prob + kWinChunk;                    // [dk]
   __shared__ float scratch[32];
@@ -337,124 +386,159 @@ window_attention_kernel(T* __restrict__ out, const T* __restrict__ q, const T* _
   const int g = h / (nh / nkv);
   const int p = positions[t];
   const int* bt = block_table + (int64_t)seq_of_token[t] * max_pages;
-  const T* qrow = q + ((int64_t)t * nh + h) * dk;
-  for (int i = threadIdx.x; i < dk; i += blockDim.x) qs[i] = to_float(qrow[i]);
-
-  int lo = 0;
-  if (window > 0 && p - window + 1 > 0) lo = p - window + 1;
+  const int lo = attn_first_key(p, window, x.chunked);
   const int n_first = min(keep_first, lo);         // kept first tokens that the window itself does not reach
   const int n_keys = n_first + (p - lo + 1);
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
 
-  float acc[4] = {0.f, 0.f, 0.f, 0.f};
-  float m = -INFINITY, l = 0.f;
-  __syncthreads();
-  for (int c0 = 0; c0 < n_keys; c0 += kWinChunk) {
-    const int n = min(kWinChunk, n_keys - c0);
-    float cmax = -INFINITY;
-    for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
-      const int e = c0 + jj;
-      const int j = e < n_first ? e : lo + (e - n_first);
-      const int page = bt[j / page_size];
-      const int64_t row = ((int64_t)page * nkv + g) * page_size + (j % page_size);
-      row_of[jj] = row;
-      const T* kr = k_pages + row * dk;
-      float sc = 0.f;
-      for (int i = 0; i < dk; ++i) sc += qs[i] * to_float(kr[i]);
-      sc *= scale;
-      if (softcap > 0.f) sc = softcap * tanhf(sc * inv_cap);
-      prob[jj] = sc;
-      cmax = fmaxf(cmax, sc);
-    }
-    cmax = block_max(cmax, scratch);
-    const float m_new = fmaxf(m, cmax);
-    const float corr = expf(m - m_new);
-    float lsum = 0.f;
-    for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
-      const float e = expf(prob[jj] - m_new);
-      prob[jj] = e;
-      lsum += e;
-    }
-    lsum = block_sum(lsum, scratch);
-    l = l * corr + lsum;
-    m = m_new;
+  float res[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int a = 0; a < 4; ++a) {
-      const int d = threadIdx.x + a * kWinThreads;
-      if (d < dv) {
-        float sum = acc[a] * corr;
-        for (int jj = 0; jj < n; ++jj) sum += prob[jj] * to_float(v_pages[row_of[jj] * dv + d]);
-        acc[a] = sum;
-      }
-    }
+  for (int map = 0; map < MAPS; ++map) {
+    const T* qrow = q + (((int64_t)t * nh + h) * MAPS + map) * dk;
     __syncthreads();
+    for (int i = threadIdx.x; i < dk; i += blockDim.x) qs[i] = to_float(qrow[i]);
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float m = -INFINITY, l = 0.f;
+    __syncthreads();
+    for (int c0 = 0; c0 < n_keys; c0 += kWinChunk) {
+      const int n = min(kWinChunk, n_keys - c0);
+      float cmax = -INFINITY;
+      for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
+        const int e = c0 + jj;
+        const int j = e < n_first ? e : lo + (e - n_first);
+        const int page = bt[j / page_size];
+        row_of[jj] = ((int64_t)page * nkv + g) * page_size + (j % page_size);
+        const T* kr = k_pages + (((int64_t)page * nkv + g) * MAPS + map) * page_size * dk + (int64_t)(j % page_size) * dk;
+        float sc = 0.f;
+        for (int i = 0; i < dk; ++i) sc += qs[i] * to_float(kr[i]);
+        sc *= scale;
+        if (softcap > 0.f) sc = softcap * tanhf(sc * inv_cap);
+        prob[jj] = sc;
+        cmax = fmaxf(cmax, sc);
+      }
+      cmax = block_max(cmax, scratch);
+      const float m_new = fmaxf(m, cmax);
+      const float corr = expf(m - m_new);
+      float lsum = 0.f;
+      for (int jj = threadIdx.x; jj < n; jj += blockDim.x) {
+        const float e = expf(prob[jj] - m_new);
+        prob[jj] = e;
+        lsum += e;
+      }
+      lsum = block_sum(lsum, scratch);
+      l = l * corr + lsum;
+      m = m_new;
+#pragma unroll
+      for (int a = 0; a < 4; ++a) {
+        const int d = threadIdx.x + a * kWinThreads;
+        if (d < dv) {
+          float sum = acc[a] * corr;
+          for (int jj = 0; jj < n; ++jj) sum += prob[jj] * to_float(v_pages[row_of[jj] * dv + d]);
+          acc[a] = sum;
+        }
+      }
+      __syncthreads();
+    }
+    if (x.sink) l += expf(x.sink[h] - m);
+    const float f = (map == 0 ? 1.f : -x.lambda) / l;
+#pragma unroll
+    for (int a = 0; a < 4; ++a) res[a] = fmaf(acc[a], f, res[a]);
+  }
+  float mul = attn_out_factor<T>(x, t, h);
+  if (MAPS > 1) {
+    float ss = 0.f;
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+      if (threadIdx.x + a * kWinThreads < dv) ss = fmaf(res[a], res[a], ss);
+    mul *= rsqrtf(block_sum(ss, scratch) / (float)dv + x.maps_eps);
   }
   T* orow = out + (int64_t)t * x.out_ld + (int64_t)h * dv;
-  if (x.sink) l += expf(x.sink[h] - m);
-  const float inv = attn_out_factor<T>(x, t, h) / l;
 #pragma unroll
   for (int a = 0; a < 4; ++a) {
     const int d = threadIdx.x + a * kWinThreads;
-    if (d < dv) orow[d] = from_float<T>(acc[a] * inv);
+    if (d < dv) orow[d] = from_float<T>(res[a] * mul);
   }
 }
 
-// Puts together the shares that window_attention_tc.cu left in `part`: per token and share [m (nh) | l (nh) | o (nh dv)],
-// a share's running maximum (natural logarithm), sum and unnormalised output.  One CTA per (token, head).
-template <typename T>
+// Puts together the shares that window_attention_tc.cu left in `part`: per token and share [m (n) | l (n) | o (n dv)] for
+// n = nh MAPS head maps, a share's running maximum (natural logarithm), sum and unnormalised output.  One CTA per (token,
+// head), a thread up to four columns.
+template <typename T, int MAPS>
 __global__ void window_attention_merge_kernel(T* __restrict__ out, const float* __restrict__ part,
                                               const int* __restrict__ seq_of_token, int nh, int dv, int nsplit,
                                               const AttnExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y;
+  __shared__ float scratch[32];
+  const int t = blockIdx.x, h = blockIdx.y, n = nh * MAPS;
   if (seq_of_token[t] < 0) return;
-  const int64_t stride = (int64_t)nh * dv + 2 * nh;
+  const int64_t stride = (int64_t)n * dv + 2 * n;
   const float* pt = part + (int64_t)t * nsplit * stride;
-  float M = -INFINITY;
-  for (int s = 0; s < nsplit; ++s) M = fmaxf(M, pt[s * stride + h]);
-  const float sink = x.sink ? expf(x.sink[h] - M) : 0.f;
-  const float f = attn_out_factor<T>(x, t, h);
-  for (int i = threadIdx.x; i < dv; i += blockDim.x) {
-    float L = 0.f, o = 0.f;
+  float res[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int map = 0; map < MAPS; ++map) {
+    const int hm = h * MAPS + map;
+    float M = -INFINITY;
+    for (int s = 0; s < nsplit; ++s) M = fmaxf(M, pt[s * stride + hm]);
+    float L = x.sink ? expf(x.sink[h] - M) : 0.f;
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
     for (int s = 0; s < nsplit; ++s) {
-      const float m = pt[s * stride + h];
+      const float m = pt[s * stride + hm];
       const float w = (m == -INFINITY) ? 0.f : expf(m - M);      // a share without keys weighs nothing
-      L = fmaf(pt[s * stride + nh + h], w, L);
-      o = fmaf(pt[s * stride + 2 * nh + (int64_t)h * dv + i], w, o);
+      L = fmaf(pt[s * stride + n + hm], w, L);
+#pragma unroll
+      for (int a = 0; a < 4; ++a) {
+        const int d = threadIdx.x + a * blockDim.x;
+        if (d < dv) o[a] = fmaf(pt[s * stride + 2 * n + (int64_t)hm * dv + d], w, o[a]);
+      }
     }
-    out[(int64_t)t * x.out_ld + (int64_t)h * dv + i] = from_float<T>(o * (f / (L + sink)));
+    const float f = (map == 0 ? 1.f : -x.lambda) / L;
+#pragma unroll
+    for (int a = 0; a < 4; ++a) res[a] = fmaf(o[a], f, res[a]);
+  }
+  float mul = attn_out_factor<T>(x, t, h);
+  if (MAPS > 1) {
+    const float ss = res[0] * res[0] + res[1] * res[1] + res[2] * res[2] + res[3] * res[3];
+    mul *= rsqrtf(block_sum(ss, scratch) / (float)dv + x.maps_eps);
+  }
+#pragma unroll
+  for (int a = 0; a < 4; ++a) {
+    const int d = threadIdx.x + a * blockDim.x;
+    if (d < dv) out[(int64_t)t * x.out_ld + (int64_t)h * dv + d] = from_float<T>(res[a] * mul);
   }
 }
 
 }  // namespace atom
 
-// qkv: [T, >= C] rows of [q (H dk) | k (G dk) | v (G dv)], row stride ld; q_out [T, H dk] dense.  conv_w [C, taps]
-// (taps 0: no convolution), conv_state [slots, taps - 1, C] (read only here).  k_pages null: nothing is written.
+// qkv: [T, >= C] rows of [q (H dk) | k (G dk) | v (GV dv)], row stride ld; q_out [T, H dk] dense.  conv_w [C, taps]
+// (taps 0: no convolution), conv_state [slots, taps - 1, C] (read only here).  k_pages null: nothing is written (G and
+// GV may then be 0).  wq, wk [dk]: norm weights of every query and key head (null: no norm; not with a convolution).
 ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, int64_t ld, int T, int H, int G, int dk,
                                      int dv, const void* conv_w, int w_dtype, int taps, const void* conv_state,
                                      const float* freq, int rot_dims, const int* positions, const int* seq_of_token,
                                      const int* cu_q, const int* state_slots, const int* block_table, int max_pages,
                                      int page_size, void* k_pages, void* v_pages, int64_t num_pages, int* status,
                                      const void* bias, int bias_dtype, int neighbours, float mag, const void* v_first,
-                                     float v_mix, void* v_keep, cudaStream_t stream) {
+                                     float v_mix, void* v_keep, int GV, const void* wq, const void* wk, int norm_dtype,
+                                     float norm_eps, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  if (bias && taps > 0) return ATOM_ERR_ARG;
-  const atom::RopeExtras x{bias, bias_dtype, neighbours, mag, v_first, v_mix, v_keep};
-  if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dk || taps < 0 ||
+  if ((bias || wq) && taps > 0) return ATOM_ERR_ARG;
+  const atom::RopeExtras x{bias, bias_dtype, neighbours, mag, v_first, v_mix, v_keep, GV, wq, wk, norm_dtype, norm_eps};
+  if (GV < 0 || (k_pages && (G == 0 || GV == 0)) || (wq && G > 0 && !wk)) return ATOM_ERR_ARG;
+  if (H <= 0 || G < 0 || dk <= 0 || dv <= 0 || rot_dims < 0 || rot_dims % 2 || rot_dims > dk || taps < 0 ||
       page_size <= 0 || (rot_dims > 0 && !freq) || (taps > 0 && !conv_w))
     return ATOM_ERR_ARG;
   if (dtype == ATOM_F32)
-    atom::launch_pdl(atom::conv_rope_write_kernel<float>, dim3(T), dim3(256), 0, stream, (float*)q_out,
+    atom::launch_pdl(atom::conv_rope_write_kernel<float>, dim3(T), dim3(256), (H + G) * sizeof(float), stream, (float*)q_out,
                      (const float*)qkv, ld, H, G, dk, dv, conv_w, w_dtype, taps, (const float*)conv_state, freq,
                      rot_dims, positions, seq_of_token, cu_q, state_slots, block_table, max_pages, page_size,
                      (float*)k_pages, (float*)v_pages, num_pages, status, x);
   else if (dtype == ATOM_BF16 && dk % 8 == 0 && dv % 8 == 0 && rot_dims % (neighbours ? 8 : 16) == 0 && ld % 8 == 0 && taps <= 8 &&
-           (taps == 0 || w_dtype == ATOM_BF16) && ((H + 2 * G) * dk + G * dv) * sizeof(float) <= 48 * 1024 &&
+           (taps == 0 || w_dtype == ATOM_BF16) && ((H + G) * dk + GV * dv + rot_dims) * sizeof(float) <= 48 * 1024 &&
            ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)conv_w % 16) == 0 && ((uintptr_t)conv_state % 16) == 0 &&
            ((uintptr_t)bias % 16) == 0 && ((uintptr_t)v_first % 16) == 0 && ((uintptr_t)v_keep % 16) == 0 &&
            ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0) {
-    const int C = (H + G) * dk + G * dv;
+    const int C = (H + G) * dk + GV * dv;
     const int threads = C / 8 >= 256 ? 256 : ((C / 8 + 31) / 32) * 32;
 #define ATOM_CV(TAPS)                                                                                               \
   atom::launch_pdl(atom::conv_rope_write_vec_kernel<TAPS>, dim3(T), dim3(threads), (C + rot_dims) * sizeof(float), stream, \
@@ -475,7 +559,7 @@ ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, in
     }
 #undef ATOM_CV
   } else if (dtype == ATOM_BF16)
-    atom::launch_pdl(atom::conv_rope_write_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream,
+    atom::launch_pdl(atom::conv_rope_write_kernel<__nv_bfloat16>, dim3(T), dim3(256), (H + G) * sizeof(float), stream,
                      (__nv_bfloat16*)q_out, (const __nv_bfloat16*)qkv, ld, H, G, dk, dv, conv_w, w_dtype, taps,
                      (const __nv_bfloat16*)conv_state, freq, rot_dims, positions, seq_of_token, cu_q, state_slots,
                      block_table, max_pages, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages,
@@ -501,48 +585,55 @@ ATOM_EXPORT int atom_conv_state_update(void* conv_state, const void* qkv, int dt
   return atom::check_launch();
 }
 
-// out: row t at out + t * out_ld, heads packed [nh, dv]; q [T, nh dk] dense.  window <= 0: every earlier key;
-// softcap <= 0: none; sink, gate null: none.
+// out: row t at out + t * out_ld, heads packed [nh, dv]; q [T, nh maps dk] dense.  window <= 0: every earlier key;
+// softcap <= 0: none; sink, gate null: none; maps: 1 or 2.
 ATOM_EXPORT int atom_window_attention(void* out, const void* q, int dtype, const void* k_pages, const void* v_pages,
                                       const int* block_table, int max_pages, int page_size, const int* positions,
                                       const int* seq_of_token, int T, int nh, int nkv, int dk, int dv, float scale,
                                       float softcap, int window, int keep_first, const float* sink, const void* gate,
-                                      int64_t gate_ld, float out_mul, int64_t out_ld, cudaStream_t stream) {
+                                      int64_t gate_ld, float out_mul, int64_t out_ld, int chunked, int maps, float lambda,
+                                      float maps_eps, cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld};
+  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld, chunked, lambda, maps_eps};
   if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || dk <= 0 || dv <= 0 || dv > 4 * atom::kWinThreads || dk > 4096 ||
-      page_size <= 0 || nh > 65535 || keep_first < 0)
+      page_size <= 0 || nh > 65535 || keep_first < 0 || maps < 1 || maps > 2 || (dtype != ATOM_F32 && dtype != ATOM_BF16))
     return ATOM_ERR_ARG;
   const size_t smem = sizeof(float) * (dk + atom::kWinChunk) + sizeof(int64_t) * atom::kWinChunk;
-  dim3 grid(T, nh);
-  if (dtype == ATOM_F32)
-    atom::launch_pdl(atom::window_attention_kernel<float>, grid, dim3(atom::kWinThreads), smem, stream, (float*)out,
-                     (const float*)q, (const float*)k_pages, (const float*)v_pages, block_table, max_pages, page_size,
-                     positions, seq_of_token, nh, nkv, dk, dv, scale, softcap, window, keep_first, x);
-  else if (dtype == ATOM_BF16)
-    atom::launch_pdl(atom::window_attention_kernel<__nv_bfloat16>, grid, dim3(atom::kWinThreads), smem, stream,
-                     (__nv_bfloat16*)out, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages,
-                     (const __nv_bfloat16*)v_pages, block_table, max_pages, page_size, positions, seq_of_token, nh,
-                     nkv, dk, dv, scale, softcap, window, keep_first, x);
-  else
-    return ATOM_ERR_ARG;
+#define ATOM_WIN(TT, MAPS)                                                                                            \
+  atom::launch_pdl(atom::window_attention_kernel<TT, MAPS>, dim3(T, nh), dim3(atom::kWinThreads), smem, stream, (TT*)out, \
+                   (const TT*)q, (const TT*)k_pages, (const TT*)v_pages, block_table, max_pages, page_size, positions, \
+                   seq_of_token, nh, nkv, dk, dv, scale, softcap, window, keep_first, x)
+  if (dtype == ATOM_F32) {
+    if (maps == 1) ATOM_WIN(float, 1);
+    else ATOM_WIN(float, 2);
+  } else {
+    if (maps == 1) ATOM_WIN(__nv_bfloat16, 1);
+    else ATOM_WIN(__nv_bfloat16, 2);
+  }
+#undef ATOM_WIN
   return atom::check_launch();
 }
 
 ATOM_EXPORT int atom_window_attention_merge(void* out, int dtype, const float* part, const int* seq_of_token, int T, int nh,
                                             int dv, int nsplit, const float* sink, const void* gate, int64_t gate_ld,
-                                            float out_mul, int64_t out_ld, cudaStream_t stream) {
+                                            float out_mul, int64_t out_ld, int maps, float lambda, float maps_eps,
+                                            cudaStream_t stream) {
   if (T <= 0) return ATOM_OK;
-  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld};
-  if (nsplit < 1 || part == nullptr || nh <= 0 || nh > 65535 || dv <= 0) return ATOM_ERR_ARG;
-  const int threads = dv >= 128 ? 128 : (dv >= 64 ? 64 : 32);
-  if (dtype == ATOM_F32)
-    atom::launch_pdl(atom::window_attention_merge_kernel<float>, dim3(T, nh), dim3(threads), 0, stream, (float*)out, part,
-                     seq_of_token, nh, dv, nsplit, x);
-  else if (dtype == ATOM_BF16)
-    atom::launch_pdl(atom::window_attention_merge_kernel<__nv_bfloat16>, dim3(T, nh), dim3(threads), 0, stream,
-                     (__nv_bfloat16*)out, part, seq_of_token, nh, dv, nsplit, x);
-  else
+  const atom::AttnExtras x{sink, gate, gate_ld, out_mul, out_ld, 0, lambda, maps_eps};
+  if (nsplit < 1 || part == nullptr || nh <= 0 || nh > 65535 || dv <= 0 || dv > 512 || maps < 1 || maps > 2 ||
+      (dtype != ATOM_F32 && dtype != ATOM_BF16))
     return ATOM_ERR_ARG;
+  const int threads = dv >= 128 ? 128 : (dv >= 64 ? 64 : 32);
+#define ATOM_WIN(TT, MAPS)                                                                                            \
+  atom::launch_pdl(atom::window_attention_merge_kernel<TT, MAPS>, dim3(T, nh), dim3(threads), 0, stream, (TT*)out, part, \
+                   seq_of_token, nh, dv, nsplit, x)
+  if (dtype == ATOM_F32) {
+    if (maps == 1) ATOM_WIN(float, 1);
+    else ATOM_WIN(float, 2);
+  } else {
+    if (maps == 1) ATOM_WIN(__nv_bfloat16, 1);
+    else ATOM_WIN(__nv_bfloat16, 2);
+  }
+#undef ATOM_WIN
   return atom::check_launch();
 }

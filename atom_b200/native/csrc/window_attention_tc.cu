@@ -1,6 +1,6 @@
 // Causal paged attention with capped scores and a sliding window that keeps a request's first tokens
 // (the formulas stand in window_attention.cu), in bfloat16 on the tensor cores, compiled for one pair of sizes:
-//   -DATOM_WA_DK (key size) -DATOM_WA_DV (value size), both multiples of 16.
+//   -DATOM_WA_DK (key size) -DATOM_WA_DV (value size), both multiples of 16, and optionally -DATOM_WA_MAPS=2.
 //
 // A CTA of 4 warps takes a tile of up to 64 consecutive tokens of one request and one query head (a warp 16 rows)
 // and walks the keys it can see in tiles of 64: first the tiles of the kept first tokens that lie before the window,
@@ -14,22 +14,36 @@
 // In a step of single tokens a CTA's rows are the query heads that share one key head, so a request's keys and values
 // are read once per key head.
 // A sink per head adds exp(sink_h) to the denominator; a gate number per (token, head) and a constant multiply the
-// output, whose rows may lie further apart (with shares the merge kernel does all of this).
+// output, whose rows may lie further apart (with shares the merge kernel does all of this).  The window may be a chunk.
+// With two maps (differential attention: two queries per head, two keys per key head, the same values) the CTA has four
+// warps per map, which share the value tiles; at the end the second map's outputs pass through shared memory to the
+// warps of the first, which subtract them and divide every row by its root mean square.
 #include "common.cuh"
 
 #if !defined(ATOM_WA_DK) || !defined(ATOM_WA_DV)
 #error "compile with -DATOM_WA_DK= -DATOM_WA_DV="
 #endif
 
+#if !defined(ATOM_WA_MAPS)
+#define ATOM_WA_MAPS 1
+#endif
+
 namespace atom {
 namespace watc {
 
+constexpr int MAPS = ATOM_WA_MAPS;
+static_assert(MAPS == 1 || MAPS == 2, "maps");
+
 constexpr int DK = ATOM_WA_DK, DV = ATOM_WA_DV;
-constexpr int BM = 64, BN = 64, WARPS = 4, THREADS = WARPS * 32;
+constexpr int BM = 64, BN = 64, WARPS = 4 * MAPS, THREADS = WARPS * 32;
 constexpr int LDK = DK + 8, LDV = DV + 8;                 // bf16 elements per row in shared memory (16 bytes of padding)
 static_assert(DK % 16 == 0 && DV % 16 == 0 && DK <= 256 && DV <= 128, "sizes");
 
-constexpr size_t kSmemBytes = sizeof(__nv_bfloat16) * ((size_t)BM * LDK + 2 * ((size_t)BN * LDK + (size_t)BN * LDV));
+constexpr int KTILE = MAPS * BN * LDK, STAGE = KTILE + BN * LDV;      // a stage: the maps' key tiles, the value tile
+constexpr int LDX = DV + 4;                                            // floats per row of the exchange between maps
+constexpr size_t kLoopBytes = sizeof(__nv_bfloat16) * ((size_t)MAPS * BM * LDK + 2 * (size_t)STAGE);
+constexpr size_t kExchBytes = MAPS > 1 ? sizeof(float) * (size_t)BM * LDX : 0;
+constexpr size_t kSmemBytes = kLoopBytes > kExchBytes ? kLoopBytes : kExchBytes;
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem) {
   const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -105,14 +119,23 @@ struct Params {
   const __nv_bfloat16* gate;       // [T, nh] rows at stride gate_ld, or null
   int64_t gate_ld, out_ld;
   float out_mul;
+  int chunked;                     // 1: the window is a chunk, keys j <= p with j / window = p / window
+  float lambda, maps_eps;          // with two maps: the second map's weight, what is added to the mean square
 };
 
-// Two threads per key row: the page is looked up once per row and tile, the row's 16-byte pieces alternate between them.
+// First key that position p sees (kept first tokens apart).
+__device__ __forceinline__ int first_key(const Params& p, int pos) {
+  if (p.window <= 0) return 0;
+  return p.chunked ? pos / p.window * p.window : max(0, pos - p.window + 1);
+}
+
+// 2 MAPS threads per key row: the page is looked up once per thread and tile, the row's 16-byte pieces alternate between
+// the threads.
 __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* Ks, __nv_bfloat16* Vs, const Params& p, const int* bt, int g,
                                              int j0, int p_last) {
-  constexpr int KC = DK / 8, VC = DV / 8;
-  static_assert(THREADS == 2 * BN, "two threads per key row");
-  const int r = threadIdx.x >> 1, half = threadIdx.x & 1;
+  constexpr int KC = DK / 8, VC = DV / 8, PER = 2 * MAPS;
+  static_assert(THREADS == PER * BN, "threads per key row");
+  const int r = threadIdx.x / PER, sub = threadIdx.x % PER;
   const int j = j0 + r;
   int page = -1;
   if (j <= p_last) {
@@ -120,25 +143,32 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* Ks, __nv_bfloat16* V
     if (lp < p.max_pages) page = bt[lp];
   }
   const bool valid = page >= 0 && page < p.num_pages;
-  const int64_t row = valid ? ((int64_t)page * p.nkv + g) * p.page_size + (j % p.page_size) : 0;
-  const __nv_bfloat16* ksrc = p.k_pages + row * DK;
-  const __nv_bfloat16* vsrc = p.v_pages + row * DV;
+  const int slot = j % p.page_size;
+  const int64_t head = valid ? (int64_t)page * p.nkv + g : 0;
+  const __nv_bfloat16* ksrc = p.k_pages + (valid ? (head * MAPS * p.page_size + slot) * DK : 0);
+  const __nv_bfloat16* vsrc = p.v_pages + (valid ? (head * p.page_size + slot) * DV : 0);
+  const int64_t map_stride = valid ? (int64_t)p.page_size * DK : 0;
 #pragma unroll
-  for (int c = 0; c < KC / 2; ++c) cp_async16(Ks + r * LDK + (2 * c + half) * 8, ksrc + (2 * c + half) * 8, valid);
+  for (int c = 0; c < MAPS * KC / PER; ++c) {
+    const int idx = c * PER + sub, map = MAPS > 1 ? idx / KC : 0, cc = idx - map * KC;
+    cp_async16(Ks + (map * BN + r) * LDK + cc * 8, ksrc + map * map_stride + cc * 8, valid);
+  }
 #pragma unroll
-  for (int c = 0; c < VC / 2; ++c) cp_async16(Vs + r * LDV + (2 * c + half) * 8, vsrc + (2 * c + half) * 8, valid);
+  for (int c = 0; c < (VC + PER - 1) / PER; ++c) {
+    const int cc = c * PER + sub;
+    if (VC % PER == 0 || cc < VC) cp_async16(Vs + r * LDV + cc * 8, vsrc + cc * 8, valid);
+  }
 }
 
 // HEADS: a step of single tokens.  A CTA's rows are the query heads of ONE key head for one token (they share the
 // keys and values, which are then read once for the group), blockIdx = (token, key head, share).
 template <bool HEADS>
-__global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const Params p) {
+__global__ void __launch_bounds__(THREADS, 2 / MAPS) window_attention_tc_kernel(const Params p) {
   atom::pdl_trigger();
   atom::pdl_wait();
   extern __shared__ __align__(16) unsigned char wa_smem[];
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(wa_smem);
-  __nv_bfloat16* KVs = Qs + BM * LDK;                          // two stages of [K tile | V tile]
-  constexpr int STAGE = BN * LDK + BN * LDV;
+  __nv_bfloat16* KVs = Qs + MAPS * BM * LDK;                   // two stages of [K tiles | V tile]
 
   int s, r, h, g, t0, rows;
   const int z = blockIdx.z;
@@ -159,10 +189,11 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
   const int p0 = p.positions[t0];
   const int p_last = HEADS ? p0 : p0 + rows - 1;
   const int* bt = p.block_table + (int64_t)s * p.max_pages;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int lane = threadIdx.x & 31;
+  const int map = MAPS > 1 ? (int)(threadIdx.x >> 7) : 0, warp = (threadIdx.x >> 5) & 3;      // (a warp's map, its rows)
 
   // key tiles: the kept first tokens' that lie before the window's first tile, then the window's
-  const int lo = p.window > 0 ? max(0, p0 - p.window + 1) : 0;
+  const int lo = first_key(p, p0);
   const int jt_lo = lo / BN, n_tiles = p_last / BN + 1;
   const int nk = p.window > 0 ? min((p.keep + BN - 1) / BN, jt_lo) : 0;
   const int n = nk + n_tiles - jt_lo;
@@ -172,13 +203,14 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
 
   // the queries of the tile, and the first key tile
   constexpr int KC = DK / 8;
-  for (int idx = threadIdx.x; idx < BM * KC; idx += THREADS) {
-    const int rr = idx / KC, c = idx - rr * KC;
+  for (int idx = threadIdx.x; idx < MAPS * BM * KC; idx += THREADS) {
+    const int qr = idx / KC, c = idx - qr * KC;
+    const int qm = MAPS > 1 ? qr / BM : 0, rr = qr - qm * BM;
     const bool valid = rr < rows;
     const int qt = HEADS ? t0 : t0 + (valid ? rr : 0), qh = HEADS ? h + (valid ? rr : 0) : h;
-    cp_async16(Qs + rr * LDK + c * 8, p.q + (int64_t)qt * p.q_stride + (int64_t)qh * DK + c * 8, valid);
+    cp_async16(Qs + qr * LDK + c * 8, p.q + (int64_t)qt * p.q_stride + (int64_t)(qh * MAPS + qm) * DK + c * 8, valid);
   }
-  if (i_begin < i_end) load_kv_tile(KVs, KVs + BN * LDK, p, bt, g, tile_of(i_begin) * BN, p_last);
+  if (i_begin < i_end) load_kv_tile(KVs, KVs + KTILE, p, bt, g, tile_of(i_begin) * BN, p_last);
   cp_async_commit();
 
   float o[DV / 8][4];
@@ -187,17 +219,19 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const bool active = warp * 16 < rows;                        // a warp without rows only helps to load
   const int row_a = warp * 16 + (lane >> 2), row_b = row_a + 8;
+  const int lo_last = first_key(p, p_last);
+  const int lo_row[2] = {first_key(p, HEADS ? p0 : p0 + row_a), first_key(p, HEADS ? p0 : p0 + row_b)};
   // with a cap: score = cap2 * tanh(sum * in_mul); without: sum * in_mul; both in units of log 2
   const float in_mul = p.cap > 0.f ? p.scale / p.cap : p.scale * kLog2e;
   const float cap2 = p.cap * kLog2e;
 
   for (int i = i_begin; i < i_end; ++i) {
     const int stage = (i - i_begin) & 1;
-    __nv_bfloat16* Ks = KVs + stage * STAGE;
-    __nv_bfloat16* Vs = Ks + BN * LDK;
+    const __nv_bfloat16* Ks = KVs + stage * STAGE + map * BN * LDK;
+    const __nv_bfloat16* Vs = KVs + stage * STAGE + KTILE;
     if (i + 1 < i_end) {
       __nv_bfloat16* Kn = KVs + (stage ^ 1) * STAGE;
-      load_kv_tile(Kn, Kn + BN * LDK, p, bt, g, tile_of(i + 1) * BN, p_last);
+      load_kv_tile(Kn, Kn + KTILE, p, bt, g, tile_of(i + 1) * BN, p_last);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -212,7 +246,7 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
 #pragma unroll
       for (int kk = 0; kk < DK / 16; ++kk) {
         uint32_t a[4];
-        ldmatrix_x4(a, Qs + (warp * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDK + kk * 16 + (lane >> 4) * 8);
+        ldmatrix_x4(a, Qs + (map * BM + warp * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * LDK + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
         for (int np = 0; np < BN / 16; ++np) {
           uint32_t b[4];
@@ -225,7 +259,7 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
       // tiles at an edge need (the diagonal, the window's far end, the end of the kept tokens, a tile of few rows);
       // the tile's maximum per row
       const bool interior = !HEADS && rows == BM && j0 + BN - 1 <= p0 &&
-                            (p.window <= 0 || p_last - j0 < p.window || j0 + BN <= p.keep);
+                            (j0 >= lo_last || j0 + BN <= p.keep);
 #pragma unroll
       for (int nt = 0; nt < BN / 8; ++nt) {
 #pragma unroll
@@ -240,7 +274,7 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
             const int j = j0 + nt * 8 + (lane & 3) * 2 + (e & 1);
             const int row = (e < 2) ? row_a : row_b;
             const int pi = HEADS ? p0 : p0 + row;
-            const bool seen = row < rows && j <= pi && (p.window <= 0 || pi - j < p.window || j < p.keep);
+            const bool seen = row < rows && j <= pi && (j >= lo_row[e >> 1] || j < p.keep);
             if (!seen) sc[nt][e] = -INFINITY;
           }
         }
@@ -308,9 +342,52 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
     __syncthreads();                                            // the stage is free for the tile after the next
   }
   if (i_begin >= i_end) cp_async_wait<0>();
-  if (!active) return;
 
   const int col = (lane & 3) * 2;
+  if (MAPS > 1 && p.nsplit == 1) {
+    // (no sink here: the maps' softmaxes are plain) the second map's outputs to the first one's warps
+    __syncthreads();                                            // queries and stages are no longer read or written
+    float* xch = reinterpret_cast<float*>(wa_smem);
+    if (active && map == 1) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const float f = l_run[k] > 0.f ? p.lambda / l_run[k] : 0.f;
+        float* dst = xch + (k ? row_b : row_a) * LDX;
+#pragma unroll
+        for (int nt = 0; nt < DV / 8; ++nt)
+          *reinterpret_cast<float2*>(dst + nt * 8 + col) = make_float2(o[nt][2 * k] * f, o[nt][2 * k + 1] * f);
+      }
+    }
+    __syncthreads();
+    if (!active || map != 0) return;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int row = k ? row_b : row_a;
+      const float inv = l_run[k] > 0.f ? 1.f / l_run[k] : 0.f;
+      const float* src = xch + row * LDX;
+      float ss = 0.f;
+#pragma unroll
+      for (int nt = 0; nt < DV / 8; ++nt) {
+        const float2 b = *reinterpret_cast<const float2*>(src + nt * 8 + col);
+        o[nt][2 * k] = fmaf(o[nt][2 * k], inv, -b.x);
+        o[nt][2 * k + 1] = fmaf(o[nt][2 * k + 1], inv, -b.y);
+        ss = fmaf(o[nt][2 * k], o[nt][2 * k], fmaf(o[nt][2 * k + 1], o[nt][2 * k + 1], ss));
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (row >= rows) continue;
+      const int tt = HEADS ? t0 : t0 + row, hh = HEADS ? h + row : h;
+      float mul = p.out_mul * rsqrtf(ss / (float)DV + p.maps_eps);
+      if (p.gate) mul = __fdividef(mul, 1.f + ex2(-kLog2e * __bfloat162float(p.gate[(int64_t)tt * p.gate_ld + hh])));
+      __nv_bfloat16* dst = p.out + (int64_t)tt * p.out_ld + (int64_t)hh * DV;
+#pragma unroll
+      for (int nt = 0; nt < DV / 8; ++nt)
+        *reinterpret_cast<__nv_bfloat162*>(dst + nt * 8 + col) =
+            __floats2bfloat162_rn(o[nt][2 * k] * mul, o[nt][2 * k + 1] * mul);
+    }
+    return;
+  }
+  if (!active) return;
   if (p.nsplit == 1) {
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
@@ -328,18 +405,18 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
             __floats2bfloat162_rn(o[nt][2 * k] * inv, o[nt][2 * k + 1] * inv);
     }
   } else {
-    const int stride = p.nh * DV + 2 * p.nh;
+    const int n_all = p.nh * MAPS, stride = n_all * DV + 2 * n_all;
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       const int row = k ? row_b : row_a;
       if (row >= rows) continue;
       float* dst = p.part + ((int64_t)(HEADS ? t0 : t0 + row) * p.nsplit + z) * stride;
-      const int hh = HEADS ? h + row : h;
+      const int hh = (HEADS ? h + row : h) * MAPS + map;
       if ((lane & 3) == 0) {
         dst[hh] = m_run[k] * kLn2;                               // the merge kernel takes natural logarithms
-        dst[p.nh + hh] = l_run[k];
+        dst[n_all + hh] = l_run[k];
       }
-      float* od = dst + 2 * p.nh + (int64_t)hh * DV;
+      float* od = dst + 2 * n_all + (int64_t)hh * DV;
 #pragma unroll
       for (int nt = 0; nt < DV / 8; ++nt)
         *reinterpret_cast<float2*>(od + nt * 8 + col) = make_float2(o[nt][2 * k], o[nt][2 * k + 1]);
@@ -350,26 +427,27 @@ __global__ void __launch_bounds__(THREADS, 2) window_attention_tc_kernel(const P
 }  // namespace watc
 }  // namespace atom
 
-ATOM_EXPORT void atom_watc_sizes(int* dk, int* dv) {
+ATOM_EXPORT void atom_watc_sizes(int* dk, int* dv, int* maps) {
   *dk = atom::watc::DK;
   *dv = atom::watc::DV;
+  *maps = atom::watc::MAPS;
 }
 
-// out: row t at out + t * out_ld, heads packed [nh, DV]; q: row t at q + t * q_stride, heads packed [nh, DK]; k_pages [pages, nkv, page, DK]; v_pages
+// out: row t at out + t * out_ld, heads packed [nh, DV]; q: row t at q + t * q_stride, heads packed [nh, MAPS, DK]; k_pages [pages, nkv, MAPS, page, DK]; v_pages
 // [pages, nkv, page, DV]; units: an upper bound of the step's tiles (ceil(T / 64) + num_seqs), or with heads_rows (a
 // step of single tokens: a CTA's rows are the query heads of one key head) the step's tokens.  nsplit > 1: part holds
-// T * nsplit * nh * (DV + 2) floats, which attention_mixed.cu's merge kernel puts together.
+// T * nsplit * nh * MAPS * (DV + 2) floats, which window_attention.cu's merge kernel puts together.
 ATOM_EXPORT int atom_window_attention_tc(void* out, const void* q, int64_t q_stride, const void* k_pages,
                                          const void* v_pages, int64_t num_pages, const int* block_table, int max_pages,
                                          int page_size, const int* positions, const int* seq_of_token, const int* cu_q,
                                          int num_seqs, int units, int nh, int nkv, float scale, float cap, int window,
                                          int keep, int nsplit, float* part, int heads_rows, const float* sink,
-                                         const void* gate, int64_t gate_ld, float out_mul, int64_t out_ld,
-                                         cudaStream_t stream) {
+                                         const void* gate, int64_t gate_ld, float out_mul, int64_t out_ld, int chunked,
+                                         float lambda, float maps_eps, cudaStream_t stream) {
   using namespace atom::watc;
   if (units <= 0) return ATOM_OK;
   if (nh <= 0 || nkv <= 0 || nh % nkv || page_size <= 0 || nsplit < 1 || nsplit > 65535 || nh > 65535 ||
-      (nsplit > 1 && part == nullptr) || (q_stride % 8) != 0 || (out_ld % 2) != 0 || (heads_rows && nh / nkv > BM))
+      (nsplit > 1 && part == nullptr) || (MAPS > 1 && sink) || (q_stride % 8) != 0 || (out_ld % 2) != 0 || (heads_rows && nh / nkv > BM))
     return ATOM_ERR_ARG;
   Params p;
   p.out = (__nv_bfloat16*)out;
@@ -398,6 +476,9 @@ ATOM_EXPORT int atom_window_attention_tc(void* out, const void* q, int64_t q_str
   p.gate_ld = gate_ld;
   p.out_ld = out_ld;
   p.out_mul = out_mul;
+  p.chunked = chunked;
+  p.lambda = lambda;
+  p.maps_eps = maps_eps;
   static bool attr_set = false;
   if (!attr_set) {
     if (cudaFuncSetAttribute(window_attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,

@@ -17,6 +17,8 @@ by whoever comes next (``delta_scale`` tells the model the factor of what ``run`
 
 "parallel" has one norm whose output both the mixer and the feed-forward read, and adds both to the residual:
    r += delta;  h = norm(r);  r += mixer(h) + ffn(h)        (a layer may have no feed-forward).
+Where the norm says ``fuses_sums`` both outputs are left (a ``SumDelta``) to the kernel of the norm that reads the stream
+next.
 
 "sandwich" puts a norm before and after each sub-block (the feed-forward and its two norms optional):
    r += delta;  a = norm1(r);  r += m * norm1b(mixer(a));  [b = norm2(r);  r += m * norm2b(ffn(b))]
@@ -31,7 +33,7 @@ own; a part that says nothing gets and gives plain tensors.
 from __future__ import annotations
 
 from .. import native
-from .linear import NormedDelta, resolve
+from .linear import NormedDelta, SumDelta, resolve
 from .registry import register
 
 
@@ -136,10 +138,12 @@ class ParallelBlock:
 
     def __init__(self, norm, mixer, ffn=None):
         self.norm, self.mixer, self.ffn = norm, mixer, ffn
+        self.takes_sums = getattr(norm, "fuses_sums", False)      # delta may be a SumDelta
 
     def run(self, residual, delta, step, cache, writes_cache):
         """The sum goes into the 32-bit residual here (a mixer that says ``adds_to_residual`` does it in
-        its own last kernel), so there is nothing left for the next norm to add: returns None."""
+        its own last kernel), so there is nothing left for the next norm to add, and None is returned; or, with norms
+        that add two outputs themselves, both are."""
         h = self.norm.add_norm(residual, delta, "norm.parallel")
         if getattr(self.mixer, "adds_to_residual", False):
             # (the mixer calls the feed-forward when it suits it: beside a member that runs on a stream of its own)
@@ -148,5 +152,7 @@ class ParallelBlock:
         else:
             f = self.ffn.forward(h, step) if self.ffn is not None else None
             m = self.mixer.forward(h, step, cache, writes_cache)
+            if self.takes_sums:
+                return m if f is None else SumDelta(m, f)
             native.pair_rmsnorm_add(residual[: m.shape[0]], m, None, None, None, f, 0.0)
         return None

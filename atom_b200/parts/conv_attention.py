@@ -35,14 +35,15 @@ def rotation_options(position) -> dict:
     return {"neighbours": getattr(position, "neighbours", False), "magnitude": getattr(position, "magnitude", 1.0)}
 
 
-def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int], keep_first: int, dtype):
+def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int], keep_first: int, dtype, maps: int = 1):
     """(into how many shares the tensor-core kernel cuts the key tiles of every unit, or 0 for the plain kernel;
     whether a unit is a token with the query heads of one key head as rows, which steps of single tokens use, or
-    a tile of 64 tokens with one head), for attention over a window that keeps first tokens (or over all keys)."""
-    key = ("window_attention", nh, nkv, dk, dv, window or 0, keep_first)
+    a tile of 64 tokens with one head), for attention over a window that keeps first tokens (or over all keys); maps:
+    attention maps per head."""
+    key = ("window_attention", nh, nkv, dk, dv, window or 0, keep_first, maps)
     plan = step.plans.get(key)
     if plan is None:
-        if native.WINDOW_TC and native.window_attention_tc_supports(dk, dv, dtype):
+        if native.WINDOW_TC and native.window_attention_tc_supports(dk, dv, dtype, maps):
             longest = min(step.max_ctx_len, window + keep_first) if window else step.max_ctx_len
             heads_rows = step.max_q_len <= 1 and nh // nkv <= native.WINDOW_TC_ROWS
             if heads_rows:
@@ -51,9 +52,9 @@ def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int]
                 units = step.num_tokens * nh
             else:
                 units = (-(-step.num_tokens // native.WINDOW_TC_ROWS) + step.num_seqs - 1) * nh
-            # (two CTAs fit an SM; steps with prompt portions fill it once before their keys are shared out: the
+            # (two CTAs of one map fit an SM; steps with prompt portions fill it once before their keys are shared out: the
             # shares cost a pass over 32-bit partial outputs of every row)
-            plan = (native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 else 1,
+            plan = (native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 and maps == 1 else 1,
                                                   min_share=128), heads_rows)
         else:
             plan = (0, False)
@@ -63,13 +64,14 @@ def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int]
 
 def attend(plan, ws, o, q, cache, step, nh: int, nkv: int, dk: int, dv: int, scale: float, softcap: float,
            window: Optional[int], keep_first: int, **extras) -> None:
-    """Runs the attention of ``plan`` (``window_plan``) over the cache's pages; extras: sink, gate, out_scale."""
+    """Runs the attention of ``plan`` (``window_plan``) over the cache's pages; extras: sink, gate, out_scale, chunked,
+    maps (lambda, eps)."""
     bt = step.block_tables[cache.group]
     nsplit, heads_rows = plan
     if nsplit:
         scratch = None
         if nsplit > 1:
-            scratch = ws.get("cwa.splits", (native.attention_mixed_scratch_elems(q.shape[0], nh, dv, nsplit),), torch.float32)
+            scratch = ws.get("cwa.splits", (native.attention_mixed_scratch_elems(q.shape[0], nh * (2 if extras.get("maps") else 1), dv, nsplit),), torch.float32)
         native.window_attention_tc(o, q, cache.k_pages, cache.v_pages, bt, step.positions, step.seq_of_token,
                                    step.cu_q, step.num_seqs, nh, nkv, dk, dv, scale, softcap, window or 0, keep_first,
                                    nsplit, scratch, heads_rows, **extras)

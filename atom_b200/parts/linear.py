@@ -61,6 +61,18 @@ class NormedDelta:
         return self.norm.normalise(self.x, self.out, self.x_bias)
 
 
+class SumDelta:
+    """The outputs of two sub-blocks that run side by side, to be added to the residual stream together: a norm that says
+    ``fuses_sums`` adds both in its own kernel; otherwise ``add_to`` does, in 32-bit."""
+    __slots__ = ("a", "b")
+
+    def __init__(self, a, b):
+        self.a, self.b = a, b
+
+    def add_to(self, residual) -> None:
+        native.pair_rmsnorm_add(residual[: self.a.shape[0]], self.a, None, None, None, self.b, 0.0)
+
+
 def resolve(delta):
     """The tensor of a part's output, whether it came as one or as work still to run."""
     return delta.run() if isinstance(delta, (PendingProduct, NormedDelta)) else delta

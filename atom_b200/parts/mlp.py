@@ -4,7 +4,8 @@ Dense with the xIELU activation:  y = W_down act(W_up x),
    act(z) = softplus(p) z^2 + z/2 for z > 0,  (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2 otherwise,
 with the two numbers (p, q) a parameter of the layer.
 GELU-gated:  y = W_down (gelu_tanh(W_gate x) * (W_up x)),  gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
-Dense with the square of relu:  y = W_down relu(W_up x)^2."""
+Dense with the square of relu:  y = W_down relu(W_up x)^2.
+Gated with clamps:  y = W_down (g sigmoid(1.702 g) (u + 1)),  g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit)."""
 from __future__ import annotations
 
 import math
@@ -62,6 +63,30 @@ class GatedGeluMLP(FeedForward):
         ws, dt = self.rt.workspace, self.rt.dtype
         f = gated_linear(x, self.w_gate_up_weight, ws.get("ffn.act", (T, self.intermediate_size), dt),
                          lambda m, n: ws.get("ffn.gate_up", (m, n), dt), act="gelu_tanh")
+        out = ws.get("ffn.out", (T, self.hidden_size), dt)
+        if defer and may_defer(f, self.w_down_weight):
+            return PendingProduct(f, self.w_down_weight, None, out)
+        return linear(f, self.w_down_weight, None, out)
+
+
+@register("ffn", "gated_clamped")
+class GatedClampedMLP(FeedForward):
+    graph_safe = True
+    takes_scaled_rows = True      # x may be ScaledRows: the first product finishes the norm
+    defers_output = True          # forward(..., defer=True) may hand the last product on unrun
+
+    def __init__(self, hidden_size: int, intermediate_size: int, limit: float):
+        self.hidden_size, self.intermediate_size, self.limit = hidden_size, intermediate_size, float(limit)
+
+    def params(self) -> Dict[str, ParamSpec]:
+        H, I = self.hidden_size, self.intermediate_size
+        return {"gate_up.weight": ParamSpec((2 * I, H), rows=(I, I)), "down.weight": ParamSpec((H, I))}
+
+    def forward(self, x, step, defer=False):
+        T = x.shape[0]
+        ws, dt = self.rt.workspace, self.rt.dtype
+        f = gated_linear(x, self.w_gate_up_weight, ws.get("ffn.act", (T, self.intermediate_size), dt),
+                         lambda m, n: ws.get("ffn.gate_up", (m, n), dt), "clamped", self.limit)
         out = ws.get("ffn.out", (T, self.hidden_size), dt)
         if defer and may_defer(f, self.w_down_weight):
             return PendingProduct(f, self.w_down_weight, None, out)

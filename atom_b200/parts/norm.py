@@ -16,7 +16,7 @@ import torch
 from .. import native
 from . import linear as _linear
 from .base import Norm
-from .linear import NormedDelta, PendingProduct, ScaledRows
+from .linear import NormedDelta, PendingProduct, ScaledRows, SumDelta
 from .registry import register
 from .spec import ParamSpec
 
@@ -112,4 +112,30 @@ class LayerNorm(Norm):
     def normalise(self, x, out, x_bias=None):
         """out = norm(x (+ x_bias)) of rows that are no part of the stream."""
         native.layernorm(out, x, self.w_weight, self.w_bias, self.eps, x_bias)
+        return out
+
+
+@register("norm", "dynamic_tanh")
+class DynamicTanh(Norm):
+    """tanh(alpha * r) * w + b with a number alpha of the norm's own, no mean and no variance; the add in front of it, of one
+    sub-block's output or of two that run side by side (``SumDelta``), is the same kernel."""
+    graph_safe = True
+    fuses_sums = True
+
+    def __init__(self, size: int):
+        self.size = size
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {"weight": ParamSpec((self.size,), role="vector", init="norm"),
+                "bias": ParamSpec((self.size,), role="vector", init="normal"),
+                "alpha": ParamSpec((1,), role="vector", init="norm", rows=(1,), members_lack_axis=True)}
+
+    def after_load(self) -> None:
+        self._alpha = float(self.w_alpha.float().cpu()[0])
+
+    def add_norm(self, residual, delta, tag, rows=None, n_rows=None):
+        a, b = (delta.a, delta.b) if isinstance(delta, SumDelta) else (_linear.resolve(delta), None)
+        n = residual.shape[0] if rows is None else (rows.numel() if n_rows is None else n_rows)
+        out = self.rt.workspace.get(tag, (n, self.size), self.rt.dtype)
+        native.add_dynamic_tanh(out, residual, a, b, self.w_weight, self.w_bias, self._alpha, rows, n)
         return out

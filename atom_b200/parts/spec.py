@@ -128,7 +128,8 @@ class CacheNeed:
 
     kind "pages": ``entries`` for every position (or for the last ``window`` positions, and with
                   ``keep_first`` also for the request's first positions, which a window never drops),
-                  held in pages.  Giving ``num_kv_heads`` and ``head_dim`` instead stands for the two
+                  held in pages.  With ``chunked`` the window is a chunk: a position's queries see only keys of
+                  its own chunk of ``window`` positions, so a chunk that is over is no longer held.  Giving ``num_kv_heads`` and ``head_dim`` instead stands for the two
                   entries "k" and "v" of that shape each.
     kind "state": one array of fixed shape per request, held in a slot.
     A need of pages may also keep ``block_entries``: one row of these arrays for every whole block of ``block``
@@ -145,6 +146,7 @@ class CacheNeed:
     head_dim: int = 0
     window: Optional[int] = None
     keep_first: int = 0
+    chunked: bool = False
     state_shape: Tuple[int, ...] = ()
     state_dtype: str = "float32"
     entries: Tuple[CacheEntry, ...] = ()
@@ -173,7 +175,8 @@ class CacheNeed:
 
     def group_key(self) -> Tuple:
         if self.kind == "pages":
-            return ("pages", self.entries, self.window) + ((self.keep_first,) if self.window and self.keep_first else ())
+            return (("pages", self.entries, self.window) + ((self.keep_first,) if self.window and self.keep_first else ())
+                    + (("chunked",) if self.window and self.chunked else ()))
         return ("state", self.state_shape, self.state_dtype)
 
     @property
@@ -198,7 +201,7 @@ class CacheNeed:
             states += [CacheEntry(f"{n}.{e.name}", e.shape, e.dtype) for e in c.states]
         if pages:
             c = pages[0][1]
-            return CacheNeed("pages", window=c.window, keep_first=c.keep_first, entries=c.entries, states=tuple(states),
+            return CacheNeed("pages", window=c.window, keep_first=c.keep_first, chunked=c.chunked, entries=c.entries, states=tuple(states),
                              block=c.block, block_entries=c.block_entries)
         if states:
             return CacheNeed("state", states=tuple(states))
