@@ -1,5 +1,5 @@
-"""Prefill and decode throughput of the Nurinex, Mugulorn, Simivik, Kibotar and Vudezen designs beside Qwen3 dense at equal
-sizes.
+"""Prefill and decode throughput of the Nurinex, Mugulorn, Simivik, Kibotar, Vudezen and Vunepel designs beside Qwen3 dense at
+equal sizes.
 
     python -m atom_b200.benchmarks.designs [--sizes 1024x8,2048x16] [--layers 4] [--prefill 2048]
                                            [--batch 8] [--context 2048] [--kernels] [--only qwen3,vudezen]
@@ -24,7 +24,11 @@ whose layers (layer norms before and after every sub-block) are in turn attentio
 all 128 numbers rotated in neighbouring pairs, a sink and a gate per head, biases) beside a state-space recurrence
 (width / 64 heads of 64 numbers, a state of 128, 4 groups, a convolution of 4 taps), and attention over all earlier
 tokens (the same heads, YaRN, blended values), all with 16 experts of the width's size and 4 identity experts in 4
-groups, of which 2 groups are kept and 2 experts used, beside a shared one.  Measured on the device with CUDA events: one prompt of ``--prefill`` tokens through
+groups, of which 2 groups are kept and 2 experts used, beside a shared one; and Vunepel, whose layers (one dynamic tanh,
+both sub-blocks beside each other) are in turn a gated delta rule (the same heads, 128 numbers per key and value, ranks of
+128, a convolution of 4 taps) and differential attention within chunks of 1024 (the same heads, two maps of 64 numbers,
+values of 128; every second such layer reads the keys of the one before), the first with a dense feed-forward, the others
+with 16 experts of the width's size of which 2 are used beside a shared one.  Measured on the device with CUDA events: one prompt of ``--prefill`` tokens through
 one step, and decode steps of ``--batch`` requests whose caches hold ``--context`` tokens (captured graphs,
 as the engine runs them).  With ``--kernels`` the kernels of one prefill step and of one decode step are
 listed with their summed device time (the engine's profiler hook), which is what the per-kernel rooflines
@@ -127,6 +131,27 @@ def vudezen_config(width: int, heads: int, layers: int) -> dict:
     return {"architecture": "Vudezen", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
             "logit_scale": 0.5, "logit_softcap": 50.0,
             "layers": [{"type": t, "mixer": m, "mlp": moe} for t, m in (kinds[i % 2] for i in range(layers))]}
+
+
+def vunepel_config(width: int, heads: int, layers: int) -> dict:
+    delta = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.4,
+           "rot": {"base": 1000000.0, "dims": 64}, "mask": {"size": 1024}}
+    dense = {"kind": "dense", "ff": 3 * width, "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": 16, "top": 2, "scale": 1.5}, "expert": {"ff": width, "limit": 7.0},
+           "shared": {"ff": width, "limit": 7.0}}
+    out, owner = [], None
+    for i in range(layers):
+        mlp = dense if i == 0 else moe
+        if i % 2 == 0:
+            out.append({"type": "channel_delta", "mixer": delta, "mlp": mlp})
+        elif owner is None:
+            out.append({"type": "attention", "mixer": att, "mlp": mlp})
+            owner = i
+        else:
+            out.append({"type": "attention", "mixer": dict(att, kv_from=owner), "mlp": mlp})
+            owner = None
+    return {"architecture": "Vunepel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": out}
 
 
 def _runner(cfg: dict, pages: int, max_len: int, batch: int):
@@ -246,10 +271,10 @@ def main(argv=None) -> int:
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=2048)
     ap.add_argument("--kernels", action="store_true", help="list the kernels of one prefill and one decode step")
-    ap.add_argument("--only", default="qwen3,nurinex,mugulorn,simivik,kibotar,vudezen", help="the designs to measure, comma-separated")
+    ap.add_argument("--only", default="qwen3,nurinex,mugulorn,simivik,kibotar,vudezen,vunepel", help="the designs to measure, comma-separated")
     args = ap.parse_args(argv)
     configs = {"qwen3": qwen3_config, "nurinex": nurinex_config, "mugulorn": mugulorn_config, "simivik": simivik_config,
-               "kibotar": kibotar_config, "vudezen": vudezen_config}
+               "kibotar": kibotar_config, "vudezen": vudezen_config, "vunepel": vunepel_config}
     chosen = [d for d in args.only.split(",") if d]
     if any(d not in configs for d in chosen):
         ap.error(f"--only takes {sorted(configs)}")

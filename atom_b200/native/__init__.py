@@ -1710,6 +1710,17 @@ def delta_lanes(dk: int) -> int:
     return 4 if dk <= 32 else 8
 
 
+DELTA_TC = True      # False: row by row also where the tensor-core kernels take the sizes (measurements, tests)
+
+
+def delta_chunk_supports(dk: int, dv: int, dtype: torch.dtype) -> bool:
+    return False
+
+
+def delta_scratch_elems(T: int, num_seqs: int, H: int, dk: int, dv: int, dtype: torch.dtype, max_q_len: int) -> int:
+    return 0
+
+
 def delta_prepare(u: torch.Tensor, rn: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor],
                   z: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, beta_in: torch.Tensor, beta: torch.Tensor,
                   seq_of_token: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, G: int, H: int, dk: int,
@@ -1738,7 +1749,8 @@ def delta_prepare(u: torch.Tensor, rn: torch.Tensor, x: torch.Tensor, w: torch.T
 
 def delta_scan(out: torch.Tensor, u: torch.Tensor, rn: torch.Tensor, la: torch.Tensor, beta: torch.Tensor,
                state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, G: int, H: int, dk: int,
-               dv: int, write_state: bool = True, lanes: Optional[int] = None) -> None:
+               dv: int, write_state: bool = True, lanes: Optional[int] = None, scratch: Optional[torch.Tensor] = None,
+               max_q_len: int = 0) -> None:
     """out[t] (float32 [T, H dv]) = S^T q_t with S <- diag(2^la_t) S, then S <- S + k_t (beta_t (v_t - S^T k_t))^T, row by row
     over every request's rows; u, rn, la, beta as ``delta_prepare`` leaves them; state [slots, H, dk, dv] float32."""
     _cuda(out, u, rn, la, beta, state, cu_q, state_slots)
