@@ -11,7 +11,7 @@
 //                           beta[t] = sigmoid(raw)   per head
 //   delta_scan_kernel     the recurrence over every request's rows, the state (32-bit) carried in the request's slot.
 //                         Every column of the state runs by itself: a CTA owns (a request, a head, 128 / LPC value columns),
-//                         LPC neighbouring lanes share a column's key channels and hold them in registers.  Two more warps
+//                         LPC neighbouring lanes share a column's key channels and hold them in registers.  Four more warps
 //                         bring the next rows into shared memory (unit vectors and decays formed on the way) while
 //                         the four compute warps walk the present ones.
 // Head h reads q and k head h / (H / G).
@@ -151,7 +151,7 @@ __global__ void __launch_bounds__(256) delta_prepare_vec_kernel(const DeltaPrep 
 
 // ------------------------------------------------------------------ the recurrence, row by row
 
-constexpr int kDrCompute = 128, kDrStagers = 64;      // threads
+constexpr int kDrCompute = 128, kDrStagers = 128;      // threads
 constexpr int kDrRows = 8;                             // rows staged at a time, in two buffers
 
 struct DeltaScan {
@@ -165,6 +165,15 @@ struct DeltaScan {
   const int* state_slots;
   int num_seqs, G, H, dk, dv, write_state;
 };
+
+__device__ __forceinline__ float4 dr_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 dr_load4(const __nv_bfloat16* p) {
+  const uint2 q = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 dr_scale4(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
 
 __device__ __forceinline__ float dr_ex2(float x) {
   float y;
@@ -189,6 +198,7 @@ __global__ void __launch_bounds__(kDrCompute + kDrStagers) delta_scan_kernel(con
   const int dk = p.dk, dv = p.dv, G = p.G, H = p.H;
   const int C = 2 * G * dk + H * dv, g = hd / (H / G);
   const T* u = (const T*)p.u;
+  const bool vec = dk % 4 == 0 && C % 4 == 0 && ((uintptr_t)p.u % 16) == 0 && ((uintptr_t)p.la % 16) == 0;
 
   auto stage = [&](int c0, float* buf, int tid, int nthreads) {
     const int n = min(kDrRows, t1 - c0);
@@ -197,18 +207,37 @@ __global__ void __launch_bounds__(kDrCompute + kDrStagers) delta_scan_kernel(con
     float* a_s = k_s + kDrRows * DKP;
     float* v_s = a_s + kDrRows * DKP;
     float* b_s = v_s + kDrRows * COLS;
-    for (int e = tid; e < n * DKP; e += nthreads) {
-      const int row = e / DKP, i = e - row * DKP;
-      const int64_t t = c0 + row;
-      float qq = 0.f, kk = 0.f, aa = 1.f;
-      if (i < dk) {
-        qq = to_float(u[t * C + g * dk + i]) * p.rn[t * 2 * G + g];
-        kk = to_float(u[t * C + (G + g) * dk + i]) * p.rn[t * 2 * G + G + g];
-        aa = dr_ex2(p.la[(t * H + hd) * dk + i]);
+    if (vec) {                                            // four channels at a time
+      constexpr int Q = DKP / 4;
+#pragma unroll 4
+      for (int e = tid; e < n * Q; e += nthreads) {
+        const int row = e / Q, i = (e - row * Q) * 4;
+        const int64_t t = c0 + row;
+        float4 qq = make_float4(0.f, 0.f, 0.f, 0.f), kk = qq, aa = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (i < dk) {
+          qq = dr_scale4(dr_load4(u + t * C + g * dk + i), p.rn[t * 2 * G + g]);
+          kk = dr_scale4(dr_load4(u + t * C + (G + g) * dk + i), p.rn[t * 2 * G + G + g]);
+          aa = dr_load4(p.la + (t * H + hd) * dk + i);
+          aa = make_float4(dr_ex2(aa.x), dr_ex2(aa.y), dr_ex2(aa.z), dr_ex2(aa.w));
+        }
+        *reinterpret_cast<float4*>(q_s + row * DKP + i) = qq;
+        *reinterpret_cast<float4*>(k_s + row * DKP + i) = kk;
+        *reinterpret_cast<float4*>(a_s + row * DKP + i) = aa;
       }
-      q_s[e] = qq;
-      k_s[e] = kk;
-      a_s[e] = aa;
+    } else {
+      for (int e = tid; e < n * DKP; e += nthreads) {
+        const int row = e / DKP, i = e - row * DKP;
+        const int64_t t = c0 + row;
+        float qq = 0.f, kk = 0.f, aa = 1.f;
+        if (i < dk) {
+          qq = to_float(u[t * C + g * dk + i]) * p.rn[t * 2 * G + g];
+          kk = to_float(u[t * C + (G + g) * dk + i]) * p.rn[t * 2 * G + G + g];
+          aa = dr_ex2(p.la[(t * H + hd) * dk + i]);
+        }
+        q_s[e] = qq;
+        k_s[e] = kk;
+        a_s[e] = aa;
+      }
     }
     for (int e = tid; e < n * COLS; e += nthreads) {
       const int row = e / COLS, c = e - row * COLS;
