@@ -82,6 +82,9 @@ _SIGNATURES = {
     "atom_gla_gate_norm": [_vp, _i64, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _i, _f, _vp, _i, _f, _vp],
     "atom_add_dynamic_tanh": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _vp],
     "atom_delta_supports": [_i, _i],
+    "atom_delta_chunk_supports": [_i, _i],
+    "atom_delta_chunk_floats": [_i, _i],
+    "atom_delta_chunks": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "atom_delta_prepare": [_vp, _vp, _vp, _i, _i64, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _i64, _vp, _vp, _vp, _vp, _i, _i,
                            _i, _i, _i, _f, _f, _vp],
     "atom_delta_scan": [_vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
@@ -1713,12 +1716,24 @@ def delta_lanes(dk: int) -> int:
 DELTA_TC = True      # False: row by row also where the tensor-core kernels take the sizes (measurements, tests)
 
 
+DELTA_CHUNK_ROWS = 64     # rows of a chunk
+DELTA_CHUNK_MIN = 96      # rows of a request in the step from which the step runs in chunks
+
+
 def delta_chunk_supports(dk: int, dv: int, dtype: torch.dtype) -> bool:
-    return False
+    return dtype == torch.bfloat16 and bool(lib().atom_delta_chunk_supports(dk, dv))
+
+
+def delta_chunks_pay(dk: int, dv: int, dtype: torch.dtype, max_q_len: int) -> bool:
+    """Whether ``delta_scan`` runs a step whose longest portion has max_q_len rows in chunks on the tensor cores."""
+    return DELTA_TC and max_q_len >= DELTA_CHUNK_MIN and delta_chunk_supports(dk, dv, dtype)
 
 
 def delta_scratch_elems(T: int, num_seqs: int, H: int, dk: int, dv: int, dtype: torch.dtype, max_q_len: int) -> int:
-    return 0
+    """Floats of scratch that ``delta_scan`` needs (0: none)."""
+    if not delta_chunks_pay(dk, dv, dtype, max_q_len):
+        return 0
+    return (-(-T // DELTA_CHUNK_ROWS) + num_seqs) * H * lib().atom_delta_chunk_floats(dk, dv)
 
 
 def delta_prepare(u: torch.Tensor, rn: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor],
@@ -1752,7 +1767,9 @@ def delta_scan(out: torch.Tensor, u: torch.Tensor, rn: torch.Tensor, la: torch.T
                dv: int, write_state: bool = True, lanes: Optional[int] = None, scratch: Optional[torch.Tensor] = None,
                max_q_len: int = 0) -> None:
     """out[t] (float32 [T, H dv]) = S^T q_t with S <- diag(2^la_t) S, then S <- S + k_t (beta_t (v_t - S^T k_t))^T, row by row
-    over every request's rows; u, rn, la, beta as ``delta_prepare`` leaves them; state [slots, H, dk, dv] float32."""
+    over every request's rows; u, rn, la, beta as ``delta_prepare`` leaves them; state [slots, H, dk, dv] float32.  Steps
+    that bring a long portion (max_q_len rows; ``delta_chunks_pay``) run in chunks on the tensor cores and take ``scratch``
+    (``delta_scratch_elems`` floats)."""
     _cuda(out, u, rn, la, beta, state, cu_q, state_slots)
     T, C = u.shape
     assert C == 2 * G * dk + H * dv and u.is_contiguous() and out.dtype == torch.float32
@@ -1760,6 +1777,15 @@ def delta_scan(out: torch.Tensor, u: torch.Tensor, rn: torch.Tensor, la: torch.T
     for t, n in ((rn, 2 * G), (la, H * dk), (beta, H)):
         assert t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, n)
     assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dk, dv)
+    if delta_chunks_pay(dk, dv, u.dtype, max_q_len):
+        assert scratch is not None and scratch.dtype == torch.float32
+        assert scratch.numel() >= delta_scratch_elems(T, num_seqs, H, dk, dv, u.dtype, max_q_len)
+        _cuda(scratch)
+        _check(lib().atom_delta_chunks(out.data_ptr(), u.data_ptr(), rn.data_ptr(), la.data_ptr(), beta.data_ptr(),
+                                       state.data_ptr(), scratch.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(), num_seqs,
+                                       T, G, H, dk, dv, int(write_state), _stream()), "delta_chunks")
+        add_launches(1)      # (what does not need the state, then the walk)
+        return
     _check(lib().atom_delta_scan(out.data_ptr(), u.data_ptr(), dtype_code(u.dtype), rn.data_ptr(), la.data_ptr(),
                                  beta.data_ptr(), state.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, T, G,
                                  H, dk, dv, lanes or delta_lanes(dk), int(write_state), _stream()), "delta_scan")

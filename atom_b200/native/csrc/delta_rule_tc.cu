@@ -1,0 +1,543 @@
+// The gated delta rule of delta_rule.cu over long portions, in chunks of 64 rows on the tensor cores (bfloat16 q, k, v).
+//
+// With G_i the sum of the decays' logarithms over a chunk's rows up to i (per key channel), S the state the chunk begins
+// with, and  A_ij = sum_c k_i k_j 2^(G_i - G_j),  B_ij = sum_c q_i k_j 2^(G_i - G_j)  (j <= i), the recurrence
+//   S <- diag(g_i) S;  u_i = beta_i (v_i - S^T k_i);  S <- S + k_i u_i^T;  o_i = S^T q_i
+// over the chunk is, with k~_i = 2^(G_i) k_i, q~_i = 2^(G_i) q_i and k^_j = 2^(G_last - G_j) k_j,
+//   (I + diag(beta) A_strictly_lower) [U_v | W] = diag(beta) [V | K~]
+//   U = U_v - W S;    O = Q~ S + B_lower U;    S <- diag(2^(G_last)) S + K^T U
+//   delta_chunk_prepare_kernel  a CTA per (chunk, head), all chunks side by side: everything that does not need the state.
+//       No exponent is above zero: blocks of A and B below the diagonal's 16 x 16 blocks take the row before the block's
+//       first as reference (both factors are then powers of sums of decays), the blocks on the diagonal form 2^(G_i - G_j)
+//       for every pair.  Sums run within a block of 16 rows and over whole blocks, so that no difference is one of two large
+//       sums (a decay's logarithm counts as -32 at least: 2^-32 of a state is below its last bit).  The triangular system is
+//       solved column by column in 32-bit.
+//   delta_chunk_scan_kernel     a CTA per (request, head, 16 value columns) walks the chunks in order.  The transposed state
+//       (16 columns x key channels) lies in the accumulators of four warps, a quarter of the channels each, and is the left
+//       operand of the products with W and Q~ as it stands (the order of a product's inner index is free, so a lane's
+//       accumulators are its operand); partial sums over the quarters meet in shared memory.  The next operands arrive by
+//       cp.async meanwhile.
+// Products run on mma.sync m16n8k8 in tf32 with every 32-bit operand as two numbers (hi + lo, three products), 32-bit
+// sums; state, decays, sums of decays and the system are 32-bit.
+#include "common.cuh"
+
+namespace atom {
+namespace drtc {
+
+constexpr int C = 64;                    // rows of a chunk
+constexpr int PT = 256;                  // threads of the prepare kernel
+constexpr int ST = 128;                  // threads of the scan kernel
+constexpr int COLS = 16;                 // value columns of a scan CTA
+constexpr int LB = C + 8;                // floats per row of B and K^ (transposed)
+
+template <int DKP>
+struct Blob {                            // what a (chunk, head) leaves for the scan, in floats
+  static constexpr int LW = DKP + 8;
+  static constexpr int W = 0;
+  static constexpr int Q = W + C * LW;
+  static constexpr int KT = Q + C * LW;
+  static constexpr int B = KT + DKP * LB;
+  static constexpr int GL = B + C * LB;
+  static constexpr int UV = GL + DKP;    // [dv][C]
+};
+template <int DKP>
+__host__ __device__ constexpr int64_t blob_floats(int dv) { return Blob<DKP>::UV + (int64_t)dv * C; }
+
+struct Params {
+  float* out;                // [T, H dv]
+  const __nv_bfloat16* u;    // [T, 2 G dk + H dv]
+  const float* rn;           // [T, 2 G]
+  const float* la;           // [T, H dk]
+  const float* beta;         // [T, H]
+  float* state;              // [slots, H, dk, dv]
+  float* blobs;              // [chunk slots, H, blob]
+  const int* cu_q;
+  const int* state_slots;
+  int num_seqs, G, H, dk, dv, write_state;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// x = hi + lo with hi and lo of ten mantissa bits (what the tf32 product reads).
+__device__ __forceinline__ void split(float x, uint32_t& hi, uint32_t& lo) {
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
+}
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// d += a b with a and b as two numbers each (the product of the two small parts is left out).
+__device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], float b0, float b1) {
+  uint32_t h0, l0, h1, l1;
+  split(b0, h0, l0);
+  split(b1, h1, l1);
+  mma_tf32(d, ah, l0, l1);
+  mma_tf32(d, al, h0, h1);
+  mma_tf32(d, ah, h0, h1);
+}
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(gmem));
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
+
+// ------------------------------------------------------------------ what does not need the state
+
+template <int DKP>
+struct PrepSmem {
+  static constexpr int LG = DKP + 4, LK = DKP + 8;
+  float g[C * LG];                       // sums of the decays' logarithms from the row's block of 16 rows on
+  float tot[4 * DKP], pre[4 * DKP], suf[4 * DKP];      // the blocks' sums; over the blocks before; over the blocks behind
+  float a[C * LB];                       // A, then transposed and times beta: at[j][i] = beta_i A_ij, i > j
+  float b[C * LB];
+  __nv_bfloat16 k[C * LK], q[C * LK];
+  float rk[C], rq[C], beta[C];
+};
+
+template <int DKP>
+__global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params p) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  extern __shared__ __align__(16) unsigned char dc_smem[];
+  PrepSmem<DKP>& sm = *reinterpret_cast<PrepSmem<DKP>*>(dc_smem);
+  constexpr int LG = PrepSmem<DKP>::LG, LK = PrepSmem<DKP>::LK;
+  using BL = Blob<DKP>;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int hd = blockIdx.y, H = p.H, G = p.G, dk = p.dk, dv = p.dv, g = hd / (H / G);
+  int s, r = 0, acc = 0;
+  for (s = 0; s < p.num_seqs; ++s) {
+    const int n_chunks = (p.cu_q[s + 1] - p.cu_q[s] + C - 1) / C;
+    if ((int)blockIdx.x < acc + n_chunks) {
+      r = blockIdx.x - acc;
+      break;
+    }
+    acc += n_chunks;
+  }
+  if (s >= p.num_seqs) return;
+  const int64_t t0 = p.cu_q[s] + r * C;
+  const int n = min(C, p.cu_q[s + 1] - (int)t0);
+  const int nb = (n + 15) / 16;                             // 16-row blocks with rows
+  const int64_t CU = 2 * (int64_t)G * dk + (int64_t)H * dv;
+  float* blob = p.blobs + ((int64_t)blockIdx.x * H + hd) * blob_floats<DKP>(dv);
+
+  // rows into shared memory; rows behind the last and channels behind dk are zero (no decay, no write)
+  for (int e = tid; e < C * DKP; e += PT) {
+    const int i = e / DKP, c = e - i * DKP;
+    const bool in = i < n && c < dk;
+    const int64_t t = t0 + (in ? i : 0);
+    sm.g[i * LG + c] = in ? fmaxf(p.la[(t * H + hd) * dk + c], -32.f) : 0.f;
+    sm.q[i * LK + c] = in ? p.u[t * CU + (int64_t)g * dk + c] : __float2bfloat16_rn(0.f);
+    sm.k[i * LK + c] = in ? p.u[t * CU + (int64_t)(G + g) * dk + c] : __float2bfloat16_rn(0.f);
+  }
+  for (int i = tid; i < C; i += PT) {
+    const int64_t t = t0 + i;
+    sm.rq[i] = i < n ? p.rn[t * 2 * G + g] : 0.f;
+    sm.rk[i] = i < n ? p.rn[t * 2 * G + G + g] : 0.f;
+    sm.beta[i] = i < n ? p.beta[t * H + hd] : 0.f;
+  }
+  for (int e = tid; e < C * LB; e += PT) {
+    sm.a[e] = 0.f;
+    sm.b[e] = 0.f;
+  }
+  __syncthreads();
+  for (int e = tid; e < 4 * DKP; e += PT) {
+    const int b = e / DKP, c = e - b * DKP;
+    float v[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) v[i] = sm.g[(b * 16 + i) * LG + c];
+#pragma unroll
+    for (int i = 1; i < 16; ++i) v[i] += v[i - 1];
+#pragma unroll
+    for (int i = 1; i < 16; ++i) sm.g[(b * 16 + i) * LG + c] = v[i];
+    sm.tot[e] = v[15];
+  }
+  __syncthreads();
+  for (int e = tid; e < 4 * DKP; e += PT) {
+    const int b = e / DKP, c = e - b * DKP;
+    float before = 0.f, behind = 0.f;
+    for (int q = 0; q < b; ++q) before += sm.tot[q * DKP + c];
+    for (int q = b + 1; q < 4; ++q) behind += sm.tot[q * DKP + c];
+    sm.pre[e] = before;
+    sm.suf[e] = behind;
+  }
+  __syncthreads();
+
+  // A and B below the blocks on the diagonal: jobs (row block I, 8 columns); reference: the row before block I
+  for (int job = warp; job < 12; job += PT / 32) {
+    const int I = job < 2 ? 1 : (job < 6 ? 2 : 3);
+    const int j0 = (job - (I == 1 ? 0 : (I == 2 ? 2 : 6))) * 8;
+    if (I >= nb) continue;
+    const int gq = lane >> 2, tq = lane & 3;
+    const int J = j0 / 16;
+    const int ia = 16 * I + gq, ib = ia + 8, jc = j0 + gq;
+    float da[4] = {0.f, 0.f, 0.f, 0.f}, db[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+    for (int kk = 0; kk < DKP; kk += 8) {
+      uint32_t kh[4], kl[4], qh[4], ql[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = (e & 1) ? ib : ia, c = kk + tq + (e >> 1) * 4;
+        const float f = ex2(sm.g[i * LG + c]);
+        split(__bfloat162float(sm.k[i * LK + c]) * f, kh[e], kl[e]);
+        split(__bfloat162float(sm.q[i * LK + c]) * f, qh[e], ql[e]);
+      }
+      float bv[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int c = kk + tq + e * 4;
+        float d = sm.tot[J * DKP + c] - sm.g[jc * LG + c];
+        for (int b = J + 1; b < I; ++b) d += sm.tot[b * DKP + c];
+        bv[e] = __bfloat162float(sm.k[jc * LK + c]) * ex2(d);
+      }
+      mma_split(da, kh, kl, bv[0], bv[1]);
+      mma_split(db, qh, ql, bv[0], bv[1]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int i = e < 2 ? ia : ib, j = j0 + 2 * tq + (e & 1);
+      sm.a[j * LB + i] = da[e] * sm.rk[i] * sm.rk[j] * sm.beta[i];
+      sm.b[i * LB + j] = db[e] * sm.rq[i] * sm.rk[j];
+    }
+  }
+  // the blocks on the diagonal: every pair j <= i of a block, its channels shared by two neighbouring lanes
+  for (int e = tid; e < 4 * 136 * 2; e += PT) {          // (a whole number of warps: 1088 = 34 * 32)
+    const int half = e & 1, pr = e >> 1, blk = pr / 136, id = pr - blk * 136;
+    int ii = (int)((sqrtf(8.f * (float)id + 1.f) - 1.f) * 0.5f);
+    ii += (ii + 1) * (ii + 2) / 2 <= id ? 1 : 0;
+    ii -= ii * (ii + 1) / 2 > id ? 1 : 0;
+    const int jj = id - ii * (ii + 1) / 2;
+    const int i = blk * 16 + ii, j = blk * 16 + jj;
+    float sa = 0.f, sb = 0.f;
+    if (blk < nb) {
+      const float* gi = sm.g + i * LG;
+      const float* gj = sm.g + j * LG;
+      const __nv_bfloat16 *ki = sm.k + i * LK, *kj = sm.k + j * LK, *qi = sm.q + i * LK;
+#pragma unroll 2
+      for (int c = half * 4; c < DKP; c += 8) {
+        const float4 x = *reinterpret_cast<const float4*>(gi + c), y = *reinterpret_cast<const float4*>(gj + c);
+        const uint2 kiv = *reinterpret_cast<const uint2*>(ki + c), kjv = *reinterpret_cast<const uint2*>(kj + c);
+        const uint2 qiv = *reinterpret_cast<const uint2*>(qi + c);
+        const float2 ki0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kiv.x));
+        const float2 ki1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kiv.y));
+        const float2 kj0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kjv.x));
+        const float2 kj1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kjv.y));
+        const float2 qi0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qiv.x));
+        const float2 qi1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qiv.y));
+        const float w0 = kj0.x * ex2(x.x - y.x), w1 = kj0.y * ex2(x.y - y.y);
+        const float w2 = kj1.x * ex2(x.z - y.z), w3 = kj1.y * ex2(x.w - y.w);
+        sa = fmaf(ki0.x, w0, fmaf(ki0.y, w1, fmaf(ki1.x, w2, fmaf(ki1.y, w3, sa))));
+        sb = fmaf(qi0.x, w0, fmaf(qi0.y, w1, fmaf(qi1.x, w2, fmaf(qi1.y, w3, sb))));
+      }
+    }
+    sa += __shfl_xor_sync(0xffffffffu, sa, 1);
+    sb += __shfl_xor_sync(0xffffffffu, sb, 1);
+    if (blk < nb && half == 0) {
+      if (i > j) sm.a[j * LB + i] = sa * sm.rk[i] * sm.rk[j] * sm.beta[i];
+      sm.b[i * LB + j] = sb * sm.rq[i] * sm.rk[j];
+    }
+  }
+  __syncthreads();
+
+  // (I + L) X = diag(beta) [K~ | V], a thread per column: once x_j stands, every later row loses L_ij x_j
+  for (int col = tid; col < DKP + dv; col += PT) {
+    float x[C];
+    if (col < DKP) {
+#pragma unroll
+      for (int i = 0; i < C; ++i)
+        x[i] = __bfloat162float(sm.k[i * LK + col]) * sm.rk[i] * ex2(sm.pre[(i / 16) * DKP + col] + sm.g[i * LG + col]) * sm.beta[i];
+    } else {
+      const __nv_bfloat16* v = p.u + t0 * CU + 2 * (int64_t)G * dk + (int64_t)hd * dv + (col - DKP);
+#pragma unroll
+      for (int i = 0; i < C; ++i) x[i] = i < n ? __bfloat162float(v[(int64_t)i * CU]) * sm.beta[i] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < C - 1; ++j) {
+#pragma unroll
+      for (int i4 = (j + 1) / 4; i4 < C / 4; ++i4) {
+        const float4 l = *reinterpret_cast<const float4*>(sm.a + j * LB + i4 * 4);      // (zero where i <= j)
+        x[4 * i4] = fmaf(-l.x, x[j], x[4 * i4]);
+        x[4 * i4 + 1] = fmaf(-l.y, x[j], x[4 * i4 + 1]);
+        x[4 * i4 + 2] = fmaf(-l.z, x[j], x[4 * i4 + 2]);
+        x[4 * i4 + 3] = fmaf(-l.w, x[j], x[4 * i4 + 3]);
+      }
+    }
+    if (col < DKP) {
+#pragma unroll
+      for (int i = 0; i < C; ++i) blob[BL::W + i * BL::LW + col] = x[i];
+    } else {
+      float* dst = blob + BL::UV + (int64_t)(col - DKP) * C;
+#pragma unroll
+      for (int i = 0; i < C; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+    }
+  }
+  // Q~, K^ transposed, B, the whole chunk's decays
+  for (int e = tid; e < C * DKP; e += PT) {
+    const int i = e / DKP, c = e - i * DKP;
+    blob[BL::Q + i * BL::LW + c] = __bfloat162float(sm.q[i * LK + c]) * sm.rq[i] * ex2(sm.pre[(i / 16) * DKP + c] + sm.g[i * LG + c]);
+  }
+  for (int e = tid; e < C * DKP; e += PT) {
+    const int c = e / C, j = e - c * C;
+    const int b = (j / 16) * DKP + c;
+    blob[BL::KT + c * LB + j] = __bfloat162float(sm.k[j * LK + c]) * sm.rk[j] * ex2(sm.tot[b] - sm.g[j * LG + c] + sm.suf[b]);
+  }
+  for (int e = tid; e < C * C; e += PT) {
+    const int i = e / C, j = e - i * C;
+    blob[BL::B + i * LB + j] = sm.b[i * LB + j];
+  }
+  for (int c = tid; c < DKP; c += PT) blob[BL::GL + c] = ex2(sm.pre[3 * DKP + c] + sm.tot[3 * DKP + c]);
+}
+
+// ------------------------------------------------------------------ the walk over the chunks
+
+template <int DKP>
+struct ScanSmem {
+  float wq[2][2 * C * (DKP + 8)];        // W and Q~ of two chunks
+  float kb[DKP * LB + C * LB + DKP];     // K^ transposed, B, decays of one
+  float part[4 * COLS * LB];             // partial sums of -U, a warp each
+  float opart[4 * COLS * LB];            // partial outputs
+};
+
+template <int DKP>
+__global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  extern __shared__ __align__(16) unsigned char dc_smem[];
+  ScanSmem<DKP>& sm = *reinterpret_cast<ScanSmem<DKP>*>(dc_smem);
+  using BL = Blob<DKP>;
+  constexpr int LW = BL::LW, KS = DKP / 32;                 // 8-channel steps of a warp's quarter
+  const int s = blockIdx.x, hd = blockIdx.y, col0 = blockIdx.z * COLS;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, tq = lane & 3;
+  const int first = p.cu_q[s], len = p.cu_q[s + 1] - first;
+  if (len <= 0) return;
+  const int H = p.H, dk = p.dk, dv = p.dv;
+  int x0 = 0;
+  for (int q = 0; q < s; ++q) x0 += (p.cu_q[q + 1] - p.cu_q[q] + C - 1) / C;
+  const int n_chunks = (len + C - 1) / C;
+  const int64_t bf = blob_floats<DKP>(dv);
+  const float* blob0 = p.blobs + ((int64_t)x0 * H + hd) * bf;
+  auto blob_of = [&](int c) { return blob0 + (int64_t)c * H * bf; };
+
+  auto load = [&](float* dst, const float* src, int floats) {
+    for (int e = tid * 4; e < floats; e += ST * 4) cp_async16(dst + e, src + e);
+  };
+  load(sm.wq[0], blob_of(0) + BL::W, 2 * C * LW);
+  cp_async_commit();
+
+  // the transposed state: rows (value columns) gq and gq + 8, channels c0 + 8 nt + 2 tq and the next
+  const int c0 = warp * (DKP / 4);
+  const int ja = col0 + gq, jb = ja + 8;
+  float* S_g = p.state + ((int64_t)p.state_slots[s] * H + hd) * dk * dv;
+  float S[KS][4];
+#pragma unroll
+  for (int nt = 0; nt < KS; ++nt) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = c0 + 8 * nt + 2 * tq + (e & 1), j = e < 2 ? ja : jb;
+      S[nt][e] = c < dk && j < dv ? S_g[(int64_t)c * dv + j] : 0.f;
+    }
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+
+  for (int ch = 0; ch < n_chunks; ++ch) {
+    const float* blob = blob_of(ch);
+    load(sm.kb, blob + BL::KT, DKP * LB + C * LB + DKP);
+    cp_async_commit();
+    if (ch + 1 < n_chunks) load(sm.wq[(ch + 1) & 1], blob_of(ch + 1) + BL::W, 2 * C * LW);
+    cp_async_commit();
+    const float* Ws = sm.wq[ch & 1];
+    const float* Qs = Ws + C * LW;
+
+    // -U and O over the warp's quarter of the channels; a warp also takes -U_v of a quarter of the rows
+    float u[C / 8][4], o[C / 8][4];
+#pragma unroll
+    for (int nt = 0; nt < C / 8; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) u[nt][e] = o[nt][e] = 0.f;
+#pragma unroll
+    for (int nt = 0; nt < C / 8; ++nt) {
+      if (nt / 2 == warp) {
+        const float* uv = blob + BL::UV + 8 * nt + 2 * tq;
+        if (ja < dv) {
+          const float2 v = *reinterpret_cast<const float2*>(uv + (int64_t)ja * C);
+          u[nt][0] = -v.x;
+          u[nt][1] = -v.y;
+        }
+        if (jb < dv) {
+          const float2 v = *reinterpret_cast<const float2*>(uv + (int64_t)jb * C);
+          u[nt][2] = -v.x;
+          u[nt][3] = -v.y;
+        }
+      }
+    }
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+      uint32_t ah[4], al[4];
+      split(S[ks][0], ah[0], al[0]);
+      split(S[ks][2], ah[1], al[1]);
+      split(S[ks][1], ah[2], al[2]);
+      split(S[ks][3], ah[3], al[3]);
+      const int at = c0 + 8 * ks + 2 * tq;
+#pragma unroll
+      for (int nt = 0; nt < C / 8; ++nt) {
+        const float2 w = *reinterpret_cast<const float2*>(Ws + (8 * nt + gq) * LW + at);
+        mma_split(u[nt], ah, al, w.x, w.y);
+        const float2 q = *reinterpret_cast<const float2*>(Qs + (8 * nt + gq) * LW + at);
+        mma_split(o[nt], ah, al, q.x, q.y);
+      }
+    }
+    float* mine = sm.part + warp * COLS * LB;
+#pragma unroll
+    for (int nt = 0; nt < C / 8; ++nt) {
+      *reinterpret_cast<float2*>(mine + gq * LB + 8 * nt + 2 * tq) = make_float2(u[nt][0], u[nt][1]);
+      *reinterpret_cast<float2*>(mine + (gq + 8) * LB + 8 * nt + 2 * tq) = make_float2(u[nt][2], u[nt][3]);
+    }
+    cp_async_wait<1>();
+    __syncthreads();                                        // partial sums stand, K^ and B are here
+
+    const float* KTs = sm.kb;
+    const float* Bs = KTs + DKP * LB;
+    const float* GLs = Bs + C * LB;
+#pragma unroll
+    for (int nt = 0; nt < KS; ++nt) {
+      const float2 gl = *reinterpret_cast<const float2*>(GLs + c0 + 8 * nt + 2 * tq);
+      S[nt][0] *= gl.x;
+      S[nt][1] *= gl.y;
+      S[nt][2] *= gl.x;
+      S[nt][3] *= gl.y;
+    }
+#pragma unroll
+    for (int js = 0; js < C / 8; ++js) {
+      float2 a = make_float2(0.f, 0.f), b = a;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float2 x = *reinterpret_cast<const float2*>(sm.part + (w * COLS + gq) * LB + 8 * js + 2 * tq);
+        const float2 y = *reinterpret_cast<const float2*>(sm.part + (w * COLS + gq + 8) * LB + 8 * js + 2 * tq);
+        a.x -= x.x;
+        a.y -= x.y;
+        b.x -= y.x;
+        b.y -= y.y;
+      }
+      uint32_t ah[4], al[4];
+      split(a.x, ah[0], al[0]);
+      split(b.x, ah[1], al[1]);
+      split(a.y, ah[2], al[2]);
+      split(b.y, ah[3], al[3]);
+      const int at = 8 * js + 2 * tq;
+#pragma unroll
+      for (int nt = 0; nt < KS; ++nt) {
+        const float2 k = *reinterpret_cast<const float2*>(KTs + (c0 + 8 * nt + gq) * LB + at);
+        mma_split(S[nt], ah, al, k.x, k.y);
+      }
+      // O += B_lower U: the warp's row blocks are warp and 7 - warp
+#pragma unroll
+      for (int nt = 0; nt < C / 8; ++nt) {
+        if ((nt == warp || nt == 7 - warp) && js <= nt) {
+          const float2 k = *reinterpret_cast<const float2*>(Bs + (8 * nt + gq) * LB + at);
+          mma_split(o[nt], ah, al, k.x, k.y);
+        }
+      }
+    }
+    float* omine = sm.opart + warp * COLS * LB;
+#pragma unroll
+    for (int nt = 0; nt < C / 8; ++nt) {
+      *reinterpret_cast<float2*>(omine + gq * LB + 8 * nt + 2 * tq) = make_float2(o[nt][0], o[nt][1]);
+      *reinterpret_cast<float2*>(omine + (gq + 8) * LB + 8 * nt + 2 * tq) = make_float2(o[nt][2], o[nt][3]);
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                        // outputs stand, K^ and B are free, the next W and Q~ are here
+    {
+      const int i = tid & (C - 1), half = tid / C;          // a row, 8 of the 16 columns
+      const int row = ch * C + i;
+      if (row < len) {
+        float r[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          r[e] = 0.f;
+#pragma unroll
+          for (int w = 0; w < 4; ++w) r[e] += sm.opart[(w * COLS + half * 8 + e) * LB + i];
+        }
+        float* dst = p.out + ((int64_t)(first + row) * H + hd) * dv + col0 + half * 8;
+        if (col0 + half * 8 + 8 <= dv && dv % 4 == 0) {
+          *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
+          *reinterpret_cast<float4*>(dst + 4) = make_float4(r[4], r[5], r[6], r[7]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (col0 + half * 8 + e < dv) dst[e] = r[e];
+        }
+      }
+    }
+  }
+  if (!p.write_state) return;
+#pragma unroll
+  for (int nt = 0; nt < KS; ++nt) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = c0 + 8 * nt + 2 * tq + (e & 1), j = e < 2 ? ja : jb;
+      if (c < dk && j < dv) S_g[(int64_t)c * dv + j] = S[nt][e];
+    }
+  }
+}
+
+template <int DKP>
+static int launch(const Params& p, int T, cudaStream_t stream) {
+  const int slots = (T + C - 1) / C + p.num_seqs;           // an upper bound of the chunks
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(delta_chunk_prepare_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             (int)sizeof(PrepSmem<DKP>)) != cudaSuccess ||
+        cudaFuncSetAttribute(delta_chunk_scan_kernel<DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             (int)sizeof(ScanSmem<DKP>)) != cudaSuccess)
+      return ATOM_ERR_LAUNCH;
+    attr_set = true;
+  }
+  atom::launch_pdl(delta_chunk_prepare_kernel<DKP>, dim3(slots, p.H), dim3(PT), sizeof(PrepSmem<DKP>), stream, p);
+  atom::launch_pdl(delta_chunk_scan_kernel<DKP>, dim3(p.num_seqs, p.H, (p.dv + COLS - 1) / COLS), dim3(ST),
+                   sizeof(ScanSmem<DKP>), stream, p);
+  return atom::check_launch();
+}
+
+static int pad_of(int dk) { return dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 96 ? 96 : 128)); }
+
+}  // namespace drtc
+}  // namespace atom
+
+ATOM_EXPORT int atom_delta_chunk_supports(int dk, int dv) { return dk > 0 && dk <= 128 && dv > 0 ? 1 : 0; }
+
+// Floats that a (chunk, head) leaves in the scratch.
+ATOM_EXPORT int atom_delta_chunk_floats(int dk, int dv) {
+  using namespace atom::drtc;
+  switch (pad_of(dk)) {
+    case 32: return (int)blob_floats<32>(dv);
+    case 64: return (int)blob_floats<64>(dv);
+    case 96: return (int)blob_floats<96>(dv);
+    default: return (int)blob_floats<128>(dv);
+  }
+}
+
+// blobs: (ceil(T / 64) + num_seqs) * H * atom_delta_chunk_floats(dk, dv) floats, 16-byte aligned; u: bfloat16.
+ATOM_EXPORT int atom_delta_chunks(float* out, const void* u, const float* rn, const float* la, const float* beta, float* state,
+                                  float* blobs, const int* cu_q, const int* state_slots, int num_seqs, int T, int G, int H,
+                                  int dk, int dv, int write_state, cudaStream_t stream) {
+  using namespace atom::drtc;
+  if (T <= 0 || num_seqs <= 0) return ATOM_OK;
+  if (!atom_delta_chunk_supports(dk, dv) || G <= 0 || H <= 0 || H % G || H > 65535 || !blobs || ((uintptr_t)blobs % 16) ||
+      ((uintptr_t)out % 16))
+    return ATOM_ERR_ARG;
+  const Params p{out, (const __nv_bfloat16*)u, rn, la, beta, state, blobs, cu_q, state_slots, num_seqs, G, H, dk, dv, write_state};
+  switch (pad_of(dk)) {
+    case 32: return launch<32>(p, T, stream);
+    case 64: return launch<64>(p, T, stream);
+    case 96: return launch<96>(p, T, stream);
+    default: return launch<128>(p, T, stream);
+  }
+}

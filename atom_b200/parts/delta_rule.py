@@ -82,6 +82,7 @@ class ChannelDeltaRule(ProjectedMixer):
         if conv is not None and writes_cache:
             native.conv_state_update(conv, rows, step.cu_q, step.state_slots, step.num_seqs)
         o = ws.get("dr.o", (T, H * dv), f32)
+        n = native.delta_scratch_elems(T, step.num_seqs, H, dk, dv, dt, step.max_q_len)
         native.delta_scan(o, u, rn, la, beta, cache.states["S"], step.cu_q, step.state_slots, step.num_seqs, G, H, dk, dv,
-                          writes_cache)
+                          writes_cache, scratch=ws.get("dr.chunks", (n,), f32) if n else None, max_q_len=step.max_q_len)
         native.gla_gate_norm(y, o, gate, self.w_norm, self.norm_eps, H, dv, step.seq_of_token, "sigmoid", y_scale)
