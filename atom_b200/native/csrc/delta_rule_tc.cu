@@ -7,11 +7,13 @@
 //   (I + diag(beta) A_strictly_lower) [U_v | W] = diag(beta) [V | K~]
 //   U = U_v - W S;    O = Q~ S + B_lower U;    S <- diag(2^(G_last)) S + K^T U
 //   delta_chunk_prepare_kernel  a CTA per (chunk, head), all chunks side by side: everything that does not need the state.
-//       No exponent is above zero: blocks of A and B below the diagonal's 16 x 16 blocks take the row before the block's
-//       first as reference (both factors are then powers of sums of decays), the blocks on the diagonal form 2^(G_i - G_j)
-//       for every pair.  Sums run within a block of 16 rows and over whole blocks, so that no difference is one of two large
-//       sums (a decay's logarithm counts as -32 at least: 2^-32 of a state is below its last bit).  The triangular system is
-//       solved column by column in 32-bit.
+//       Rows of 16-row block I of A and B take the row before the block as reference: the rows' factor is 2^(sum from the
+//       block's first row on), the columns' 2^(sum from the column's next row to the block before) in earlier blocks, and its
+//       inverse counterpart 2^-(sum up to the column) within the block, where that stays below 2^60; a block whose decays
+//       reach further forms 2^(G_i - G_j) for every pair instead.  Sums run within a block of 16 rows and over whole blocks,
+//       so that no difference is one of two large sums (a decay's logarithm counts as -32 at least: 2^-32 of a state is below
+//       its last bit).  T = (I + diag(beta) A_strictly_lower)^-1 is formed column by column in 32-bit, [W | U_v] is T times
+//       diag(beta) [K~ | V].
 //   delta_chunk_scan_kernel     a CTA per (request, head, 16 value columns) walks the chunks in order.  The transposed state
 //       (16 columns x key channels) lies in the accumulators of four warps, a quarter of the channels each, and is the left
 //       operand of the products with W and Q~ as it stands (the order of a product's inner index is free, so a lane's
@@ -67,19 +69,28 @@ __device__ __forceinline__ void split(float x, uint32_t& hi, uint32_t& lo) {
   lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
 }
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
+  asm(
       "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-// d += a b with a and b as two numbers each (the product of the two small parts is left out).
-__device__ __forceinline__ void mma_split(float (&d)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], float b0, float b1) {
-  uint32_t h0, l0, h1, l1;
-  split(b0, h0, l0);
-  split(b1, h1, l1);
-  mma_tf32(d, ah, l0, l1);
-  mma_tf32(d, al, h0, h1);
-  mma_tf32(d, ah, h0, h1);
+// d[i] += a b[i] with a and the b[i] as two numbers each (the product of the two small parts is left out); the products of
+// one accumulator stand apart.
+template <int N>
+__device__ __forceinline__ void mma_split(float (*const (&d)[N])[4], const uint32_t (&ah)[4], const uint32_t (&al)[4],
+                                          const float2 (&b)[N]) {
+  uint32_t h0[N], l0[N], h1[N], l1[N];
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    split(b[i].x, h0[i], l0[i]);
+    split(b[i].y, h1[i], l1[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < N; ++i) mma_tf32(*d[i], ah, l0[i], l1[i]);
+#pragma unroll
+  for (int i = 0; i < N; ++i) mma_tf32(*d[i], al, h0[i], h1[i]);
+#pragma unroll
+  for (int i = 0; i < N; ++i) mma_tf32(*d[i], ah, h0[i], h1[i]);
 }
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -93,13 +104,14 @@ __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_gr
 
 template <int DKP>
 struct PrepSmem {
-  static constexpr int LG = DKP + 4, LK = DKP + 8;
+  static constexpr int LG = DKP + 4, LK = DKP + 8, LT = C + 4;
   float g[C * LG];                       // sums of the decays' logarithms from the row's block of 16 rows on
   float tot[4 * DKP], pre[4 * DKP], suf[4 * DKP];      // the blocks' sums; over the blocks before; over the blocks behind
-  float a[C * LB];                       // A, then transposed and times beta: at[j][i] = beta_i A_ij, i > j
-  float b[C * LB];
+  float a[C * LB];                       // [j][i] = beta_i A_ij for i > j, zero for the other i of j's 16-row block
+  float t[C * LT];                       // T
   __nv_bfloat16 k[C * LK], q[C * LK];
   float rk[C], rq[C], beta[C];
+  int strong[4];                         // a channel of the block decays beyond 2^-60
 };
 
 template <int DKP>
@@ -129,23 +141,43 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
   float* blob = p.blobs + ((int64_t)blockIdx.x * H + hd) * blob_floats<DKP>(dv);
 
   // rows into shared memory; rows behind the last and channels behind dk are zero (no decay, no write)
-  for (int e = tid; e < C * DKP; e += PT) {
-    const int i = e / DKP, c = e - i * DKP;
-    const bool in = i < n && c < dk;
-    const int64_t t = t0 + (in ? i : 0);
-    sm.g[i * LG + c] = in ? fmaxf(p.la[(t * H + hd) * dk + c], -32.f) : 0.f;
-    sm.q[i * LK + c] = in ? p.u[t * CU + (int64_t)g * dk + c] : __float2bfloat16_rn(0.f);
-    sm.k[i * LK + c] = in ? p.u[t * CU + (int64_t)(G + g) * dk + c] : __float2bfloat16_rn(0.f);
+  if (tid < 4) sm.strong[tid] = 0;
+  if (dk % 8 == 0 && CU % 8 == 0 && ((uintptr_t)p.u % 16) == 0 && ((uintptr_t)p.la % 16) == 0) {
+#pragma unroll 4
+    for (int e = tid; e < C * DKP / 8; e += PT) {
+      const int i = e / (DKP / 8), c = (e - i * (DKP / 8)) * 8;
+      const bool in = i < n && c < dk;
+      const int64_t t = t0 + (in ? i : 0);
+      uint4 qv = make_uint4(0u, 0u, 0u, 0u), kv = qv;
+      float4 l0 = make_float4(0.f, 0.f, 0.f, 0.f), l1 = l0;
+      if (in) {
+        qv = *reinterpret_cast<const uint4*>(p.u + t * CU + (int64_t)g * dk + c);
+        kv = *reinterpret_cast<const uint4*>(p.u + t * CU + (int64_t)(G + g) * dk + c);
+        l0 = *reinterpret_cast<const float4*>(p.la + (t * H + hd) * dk + c);
+        l1 = *reinterpret_cast<const float4*>(p.la + (t * H + hd) * dk + c + 4);
+      }
+      *reinterpret_cast<uint4*>(sm.q + i * LK + c) = qv;
+      *reinterpret_cast<uint4*>(sm.k + i * LK + c) = kv;
+      *reinterpret_cast<float4*>(sm.g + i * LG + c) =
+          make_float4(fmaxf(l0.x, -32.f), fmaxf(l0.y, -32.f), fmaxf(l0.z, -32.f), fmaxf(l0.w, -32.f));
+      *reinterpret_cast<float4*>(sm.g + i * LG + c + 4) =
+          make_float4(fmaxf(l1.x, -32.f), fmaxf(l1.y, -32.f), fmaxf(l1.z, -32.f), fmaxf(l1.w, -32.f));
+    }
+  } else {
+    for (int e = tid; e < C * DKP; e += PT) {
+      const int i = e / DKP, c = e - i * DKP;
+      const bool in = i < n && c < dk;
+      const int64_t t = t0 + (in ? i : 0);
+      sm.g[i * LG + c] = in ? fmaxf(p.la[(t * H + hd) * dk + c], -32.f) : 0.f;
+      sm.q[i * LK + c] = in ? p.u[t * CU + (int64_t)g * dk + c] : __float2bfloat16_rn(0.f);
+      sm.k[i * LK + c] = in ? p.u[t * CU + (int64_t)(G + g) * dk + c] : __float2bfloat16_rn(0.f);
+    }
   }
   for (int i = tid; i < C; i += PT) {
     const int64_t t = t0 + i;
     sm.rq[i] = i < n ? p.rn[t * 2 * G + g] : 0.f;
     sm.rk[i] = i < n ? p.rn[t * 2 * G + G + g] : 0.f;
     sm.beta[i] = i < n ? p.beta[t * H + hd] : 0.f;
-  }
-  for (int e = tid; e < C * LB; e += PT) {
-    sm.a[e] = 0.f;
-    sm.b[e] = 0.f;
   }
   __syncthreads();
   for (int e = tid; e < 4 * DKP; e += PT) {
@@ -158,6 +190,7 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
 #pragma unroll
     for (int i = 1; i < 16; ++i) sm.g[(b * 16 + i) * LG + c] = v[i];
     sm.tot[e] = v[15];
+    if (v[15] < -60.f) sm.strong[b] = 1;
   }
   __syncthreads();
   for (int e = tid; e < 4 * DKP; e += PT) {
@@ -168,96 +201,89 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
     sm.pre[e] = before;
     sm.suf[e] = behind;
   }
-  __syncthreads();
 
-  // A and B below the blocks on the diagonal: jobs (row block I, 8 columns); reference: the row before block I
-  for (int job = warp; job < 12; job += PT / 32) {
-    const int I = job < 2 ? 1 : (job < 6 ? 2 : 3);
-    const int j0 = (job - (I == 1 ? 0 : (I == 2 ? 2 : 6))) * 8;
-    if (I >= nb) continue;
-    const int gq = lane >> 2, tq = lane & 3;
-    const int J = j0 / 16;
-    const int ia = 16 * I + gq, ib = ia + 8, jc = j0 + gq;
-    float da[4] = {0.f, 0.f, 0.f, 0.f}, db[4] = {0.f, 0.f, 0.f, 0.f};
+  // A and B: a warp takes up to three tiles of 8 columns of one row block (block 3: 8 tiles, 2: 6, 1: 4, 0: 2)
+  const int gq = lane >> 2, tq = lane & 3;
+  {
+    const int I = warp < 3 ? 3 : (warp < 5 ? 2 : (warp < 7 ? 1 : 0));
+    const int jt0 = warp < 3 ? 3 * warp : (warp < 5 ? 3 * (warp - 3) : (warp < 7 ? 2 * (warp - 5) : 0));
+    const int tiles = warp == 2 || warp >= 5 ? 2 : 3;
+    const bool strong = sm.strong[I] != 0;
+    const int ia = 16 * I + gq, ib = ia + 8;
+    float da[3][4], db[3][4];
+#pragma unroll
+    for (int x = 0; x < 3; ++x)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) da[x][e] = db[x][e] = 0.f;
+    if (I < nb) {
 #pragma unroll 2
-    for (int kk = 0; kk < DKP; kk += 8) {
-      uint32_t kh[4], kl[4], qh[4], ql[4];
+      for (int kk = 0; kk < DKP; kk += 8) {
+        uint32_t kh[4], kl[4], qh[4], ql[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = (e & 1) ? ib : ia, c = kk + tq + (e >> 1) * 4;
-        const float f = ex2(sm.g[i * LG + c]);
-        split(__bfloat162float(sm.k[i * LK + c]) * f, kh[e], kl[e]);
-        split(__bfloat162float(sm.q[i * LK + c]) * f, qh[e], ql[e]);
-      }
-      float bv[2];
+        for (int e = 0; e < 4; ++e) {
+          const int i = (e & 1) ? ib : ia, c = kk + tq + (e >> 1) * 4;
+          const float f = ex2(sm.g[i * LG + c]);
+          split(__bfloat162float(sm.k[i * LK + c]) * f, kh[e], kl[e]);
+          split(__bfloat162float(sm.q[i * LK + c]) * f, qh[e], ql[e]);
+        }
+        float2 bv[3];
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int c = kk + tq + e * 4;
-        float d = sm.tot[J * DKP + c] - sm.g[jc * LG + c];
-        for (int b = J + 1; b < I; ++b) d += sm.tot[b * DKP + c];
-        bv[e] = __bfloat162float(sm.k[jc * LK + c]) * ex2(d);
+        for (int x = 0; x < 3; ++x) {
+          const int jt = min(jt0 + x, 2 * I + 1), J = jt >> 1, jc = jt * 8 + gq;
+          float w[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int c = kk + tq + e * 4;
+            float d = -sm.g[jc * LG + c];
+            if (J < I) d += sm.tot[J * DKP + c];
+            if (J == 0 && I >= 2) d += sm.tot[DKP + c];
+            if (J <= 1 && I == 3) d += sm.tot[2 * DKP + c];
+            if (J == I && strong) d = 0.f;                  // (formed pair by pair below)
+            w[e] = __bfloat162float(sm.k[jc * LK + c]) * ex2(d);
+          }
+          bv[x] = make_float2(w[0], w[1]);
+        }
+        mma_split<3>({&da[0], &da[1], &da[2]}, kh, kl, bv);
+        mma_split<3>({&db[0], &db[1], &db[2]}, qh, ql, bv);
       }
-      mma_split(da, kh, kl, bv[0], bv[1]);
-      mma_split(db, qh, ql, bv[0], bv[1]);
     }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int i = e < 2 ? ia : ib, j = j0 + 2 * tq + (e & 1);
-      sm.a[j * LB + i] = da[e] * sm.rk[i] * sm.rk[j] * sm.beta[i];
-      sm.b[i * LB + j] = db[e] * sm.rq[i] * sm.rk[j];
+    for (int x = 0; x < 3; ++x) {
+      if (x < tiles && !(strong && (jt0 + x) >> 1 == I)) {
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = h ? ib : ia, j = (jt0 + x) * 8 + 2 * tq;
+          float2 bo;
+          sm.a[j * LB + i] = i > j ? da[x][2 * h] * sm.rk[i] * sm.rk[j] * sm.beta[i] : 0.f;
+          sm.a[(j + 1) * LB + i] = i > j + 1 ? da[x][2 * h + 1] * sm.rk[i] * sm.rk[j + 1] * sm.beta[i] : 0.f;
+          bo.x = i >= j ? db[x][2 * h] * sm.rq[i] * sm.rk[j] : 0.f;
+          bo.y = i >= j + 1 ? db[x][2 * h + 1] * sm.rq[i] * sm.rk[j + 1] : 0.f;
+          *reinterpret_cast<float2*>(blob + BL::B + i * LB + j) = bo;
+        }
+      }
     }
   }
-  // the blocks on the diagonal: every pair j <= i of a block, its channels shared by two neighbouring lanes
-  for (int e = tid; e < 4 * 136 * 2; e += PT) {          // (a whole number of warps: 1088 = 34 * 32)
-    const int half = e & 1, pr = e >> 1, blk = pr / 136, id = pr - blk * 136;
-    int ii = (int)((sqrtf(8.f * (float)id + 1.f) - 1.f) * 0.5f);
-    ii += (ii + 1) * (ii + 2) / 2 <= id ? 1 : 0;
-    ii -= ii * (ii + 1) / 2 > id ? 1 : 0;
-    const int jj = id - ii * (ii + 1) / 2;
-    const int i = blk * 16 + ii, j = blk * 16 + jj;
+  for (int blk = 0; blk < 4; ++blk) {
+    if (!sm.strong[blk]) continue;                          // (the same for all threads)
+    const int i = blk * 16 + (tid >> 4), j = blk * 16 + (tid & 15);
     float sa = 0.f, sb = 0.f;
-    if (blk < nb) {
-      const float* gi = sm.g + i * LG;
-      const float* gj = sm.g + j * LG;
-      const __nv_bfloat16 *ki = sm.k + i * LK, *kj = sm.k + j * LK, *qi = sm.q + i * LK;
-#pragma unroll 2
-      for (int c = half * 4; c < DKP; c += 8) {
-        const float4 x = *reinterpret_cast<const float4*>(gi + c), y = *reinterpret_cast<const float4*>(gj + c);
-        const uint2 kiv = *reinterpret_cast<const uint2*>(ki + c), kjv = *reinterpret_cast<const uint2*>(kj + c);
-        const uint2 qiv = *reinterpret_cast<const uint2*>(qi + c);
-        const float2 ki0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kiv.x));
-        const float2 ki1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kiv.y));
-        const float2 kj0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kjv.x));
-        const float2 kj1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kjv.y));
-        const float2 qi0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qiv.x));
-        const float2 qi1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qiv.y));
-        const float w0 = kj0.x * ex2(x.x - y.x), w1 = kj0.y * ex2(x.y - y.y);
-        const float w2 = kj1.x * ex2(x.z - y.z), w3 = kj1.y * ex2(x.w - y.w);
-        sa = fmaf(ki0.x, w0, fmaf(ki0.y, w1, fmaf(ki1.x, w2, fmaf(ki1.y, w3, sa))));
-        sb = fmaf(qi0.x, w0, fmaf(qi0.y, w1, fmaf(qi1.x, w2, fmaf(qi1.y, w3, sb))));
+    if (j <= i) {
+      for (int c = 0; c < DKP; ++c) {
+        const float w = __bfloat162float(sm.k[j * LK + c]) * ex2(sm.g[i * LG + c] - sm.g[j * LG + c]);
+        sa = fmaf(__bfloat162float(sm.k[i * LK + c]), w, sa);
+        sb = fmaf(__bfloat162float(sm.q[i * LK + c]), w, sb);
       }
     }
-    sa += __shfl_xor_sync(0xffffffffu, sa, 1);
-    sb += __shfl_xor_sync(0xffffffffu, sb, 1);
-    if (blk < nb && half == 0) {
-      if (i > j) sm.a[j * LB + i] = sa * sm.rk[i] * sm.rk[j] * sm.beta[i];
-      sm.b[i * LB + j] = sb * sm.rq[i] * sm.rk[j];
-    }
+    sm.a[j * LB + i] = i > j ? sa * sm.rk[i] * sm.rk[j] * sm.beta[i] : 0.f;
+    blob[BL::B + i * LB + j] = sb * sm.rq[i] * sm.rk[j];
   }
   __syncthreads();
 
-  // (I + L) X = diag(beta) [K~ | V], a thread per column: once x_j stands, every later row loses L_ij x_j
-  for (int col = tid; col < DKP + dv; col += PT) {
+  if (warp < 2) {
+    // T, a thread per column: once x_j stands, every later row loses beta_i A_ij x_j
     float x[C];
-    if (col < DKP) {
 #pragma unroll
-      for (int i = 0; i < C; ++i)
-        x[i] = __bfloat162float(sm.k[i * LK + col]) * sm.rk[i] * ex2(sm.pre[(i / 16) * DKP + col] + sm.g[i * LG + col]) * sm.beta[i];
-    } else {
-      const __nv_bfloat16* v = p.u + t0 * CU + 2 * (int64_t)G * dk + (int64_t)hd * dv + (col - DKP);
-#pragma unroll
-      for (int i = 0; i < C; ++i) x[i] = i < n ? __bfloat162float(v[(int64_t)i * CU]) * sm.beta[i] : 0.f;
-    }
+    for (int i = 0; i < C; ++i) x[i] = i == tid ? 1.f : 0.f;
 #pragma unroll
     for (int j = 0; j < C - 1; ++j) {
 #pragma unroll
@@ -269,30 +295,103 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
         x[4 * i4 + 3] = fmaf(-l.w, x[j], x[4 * i4 + 3]);
       }
     }
-    if (col < DKP) {
 #pragma unroll
-      for (int i = 0; i < C; ++i) blob[BL::W + i * BL::LW + col] = x[i];
-    } else {
-      float* dst = blob + BL::UV + (int64_t)(col - DKP) * C;
+    for (int i = 0; i < C; ++i) sm.t[i * PrepSmem<DKP>::LT + tid] = x[i];
+  } else {
+    // meanwhile: Q~, K^ transposed, the whole chunk's decays
+    const int w = tid - 64;
+    constexpr int NW = PT - 64;
+#pragma unroll 2
+    for (int e = w; e < C * DKP / 4; e += NW) {
+      const int i = e / (DKP / 4), c = (e - i * (DKP / 4)) * 4;
+      const float4 gl = *reinterpret_cast<const float4*>(sm.g + i * LG + c);
+      const float4 pr = *reinterpret_cast<const float4*>(sm.pre + (i / 16) * DKP + c);
+      const uint2 qv = *reinterpret_cast<const uint2*>(sm.q + i * LK + c);
+      const float2 q0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qv.x));
+      const float2 q1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qv.y));
+      const float f = sm.rq[i];
+      *reinterpret_cast<float4*>(blob + BL::Q + i * BL::LW + c) =
+          make_float4(q0.x * f * ex2(pr.x + gl.x), q0.y * f * ex2(pr.y + gl.y), q1.x * f * ex2(pr.z + gl.z),
+                      q1.y * f * ex2(pr.w + gl.w));
+    }
+#pragma unroll 1
+    for (int e = w; e < DKP * (C / 8); e += NW) {
+      const int j8 = e / DKP, c = e - j8 * DKP;             // (eight rows of one block)
+      const float d = sm.tot[(j8 / 2) * DKP + c], suf = sm.suf[(j8 / 2) * DKP + c];
+      float o[8];
 #pragma unroll
-      for (int i = 0; i < C; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+      for (int x = 0; x < 8; ++x) {
+        const int j = j8 * 8 + x;
+        o[x] = __bfloat162float(sm.k[j * LK + c]) * sm.rk[j] * ex2(d - sm.g[j * LG + c] + suf);
+      }
+      float* dst = blob + BL::KT + c * LB + j8 * 8;
+      *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
+      *reinterpret_cast<float4*>(dst + 4) = make_float4(o[4], o[5], o[6], o[7]);
+    }
+    for (int c = w; c < DKP; c += NW) blob[BL::GL + c] = ex2(sm.pre[3 * DKP + c] + sm.tot[3 * DKP + c]);
+  }
+  __syncthreads();
+
+  // [W | U_v] = T diag(beta) [K~ | V]: a warp four tiles of 8 columns at a time, all rows
+  for (int base = warp * 32; base < DKP + dv; base += PT) {
+    const bool keys = base < DKP;
+    float acc[4][4][4];
+#pragma unroll
+    for (int I = 0; I < 4; ++I)
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[I][x][e] = 0.f;
+    const __nv_bfloat16* v = p.u + t0 * CU + 2 * (int64_t)G * dk + (int64_t)hd * dv - DKP;
+#pragma unroll
+    for (int ks = 0; ks < C / 8; ++ks) {
+      float2 bv[4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int col = base + 8 * x + gq;
+        float w[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int j = 8 * ks + tq + 4 * e;
+          if (keys)
+            w[e] = __bfloat162float(sm.k[j * LK + col]) * sm.rk[j] * ex2(sm.pre[(j / 16) * DKP + col] + sm.g[j * LG + col]);
+          else
+            w[e] = j < n && col < DKP + dv ? __bfloat162float(v[(int64_t)j * CU + col]) : 0.f;
+          w[e] *= sm.beta[j];
+        }
+        bv[x] = make_float2(w[0], w[1]);
+      }
+#pragma unroll
+      for (int I = ks / 2; I < 4; ++I) {
+        uint32_t th[4], tl[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          split(sm.t[(16 * I + gq + (e & 1) * 8) * PrepSmem<DKP>::LT + 8 * ks + tq + (e >> 1) * 4], th[e], tl[e]);
+        mma_split<4>({&acc[I][0], &acc[I][1], &acc[I][2], &acc[I][3]}, th, tl, bv);
+      }
+    }
+#pragma unroll
+    for (int I = 0; I < 4; ++I) {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int col = base + 8 * x + 2 * tq, i = 16 * I + gq;
+        if (keys) {
+          *reinterpret_cast<float2*>(blob + BL::W + i * BL::LW + col) = make_float2(acc[I][x][0], acc[I][x][1]);
+          *reinterpret_cast<float2*>(blob + BL::W + (i + 8) * BL::LW + col) = make_float2(acc[I][x][2], acc[I][x][3]);
+        } else {
+          float* dst = blob + BL::UV + (int64_t)(col - DKP) * C + i;
+          if (col < DKP + dv) {
+            dst[0] = acc[I][x][0];
+            dst[8] = acc[I][x][2];
+          }
+          if (col + 1 < DKP + dv) {
+            dst[C] = acc[I][x][1];
+            dst[C + 8] = acc[I][x][3];
+          }
+        }
+      }
     }
   }
-  // Q~, K^ transposed, B, the whole chunk's decays
-  for (int e = tid; e < C * DKP; e += PT) {
-    const int i = e / DKP, c = e - i * DKP;
-    blob[BL::Q + i * BL::LW + c] = __bfloat162float(sm.q[i * LK + c]) * sm.rq[i] * ex2(sm.pre[(i / 16) * DKP + c] + sm.g[i * LG + c]);
-  }
-  for (int e = tid; e < C * DKP; e += PT) {
-    const int c = e / C, j = e - c * C;
-    const int b = (j / 16) * DKP + c;
-    blob[BL::KT + c * LB + j] = __bfloat162float(sm.k[j * LK + c]) * sm.rk[j] * ex2(sm.tot[b] - sm.g[j * LG + c] + sm.suf[b]);
-  }
-  for (int e = tid; e < C * C; e += PT) {
-    const int i = e / C, j = e - i * C;
-    blob[BL::B + i * LB + j] = sm.b[i * LB + j];
-  }
-  for (int c = tid; c < DKP; c += PT) blob[BL::GL + c] = ex2(sm.pre[3 * DKP + c] + sm.tot[3 * DKP + c]);
 }
 
 // ------------------------------------------------------------------ the walk over the chunks
@@ -344,6 +443,22 @@ __global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p)
       S[nt][e] = c < dk && j < dv ? S_g[(int64_t)c * dv + j] : 0.f;
     }
   }
+  // U_v of a warp's quarter of the rows, one chunk ahead
+  float uv[2][4];
+  auto load_uv = [&](int c) {
+    const float* src = blob_of(c) + BL::UV + 16 * warp + 2 * tq;
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      float2 a = make_float2(0.f, 0.f), b = a;
+      if (ja < dv) a = *reinterpret_cast<const float2*>(src + (int64_t)ja * C + 8 * x);
+      if (jb < dv) b = *reinterpret_cast<const float2*>(src + (int64_t)jb * C + 8 * x);
+      uv[x][0] = a.x;
+      uv[x][1] = a.y;
+      uv[x][2] = b.x;
+      uv[x][3] = b.y;
+    }
+  };
+  load_uv(0);
   cp_async_wait<0>();
   __syncthreads();
 
@@ -361,23 +476,10 @@ __global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p)
 #pragma unroll
     for (int nt = 0; nt < C / 8; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) u[nt][e] = o[nt][e] = 0.f;
-#pragma unroll
-    for (int nt = 0; nt < C / 8; ++nt) {
-      if (nt / 2 == warp) {
-        const float* uv = blob + BL::UV + 8 * nt + 2 * tq;
-        if (ja < dv) {
-          const float2 v = *reinterpret_cast<const float2*>(uv + (int64_t)ja * C);
-          u[nt][0] = -v.x;
-          u[nt][1] = -v.y;
-        }
-        if (jb < dv) {
-          const float2 v = *reinterpret_cast<const float2*>(uv + (int64_t)jb * C);
-          u[nt][2] = -v.x;
-          u[nt][3] = -v.y;
-        }
+      for (int e = 0; e < 4; ++e) {
+        u[nt][e] = nt / 2 == warp ? -uv[nt & 1][e] : 0.f;
+        o[nt][e] = 0.f;
       }
-    }
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
       uint32_t ah[4], al[4];
@@ -387,11 +489,15 @@ __global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p)
       split(S[ks][3], ah[3], al[3]);
       const int at = c0 + 8 * ks + 2 * tq;
 #pragma unroll
-      for (int nt = 0; nt < C / 8; ++nt) {
-        const float2 w = *reinterpret_cast<const float2*>(Ws + (8 * nt + gq) * LW + at);
-        mma_split(u[nt], ah, al, w.x, w.y);
-        const float2 q = *reinterpret_cast<const float2*>(Qs + (8 * nt + gq) * LW + at);
-        mma_split(o[nt], ah, al, q.x, q.y);
+      for (int nt = 0; nt < C / 8; nt += 4) {
+        float2 w[4], q[4];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          w[x] = *reinterpret_cast<const float2*>(Ws + (8 * (nt + x) + gq) * LW + at);
+          q[x] = *reinterpret_cast<const float2*>(Qs + (8 * (nt + x) + gq) * LW + at);
+        }
+        mma_split<4>({&u[nt], &u[nt + 1], &u[nt + 2], &u[nt + 3]}, ah, al, w);
+        mma_split<4>({&o[nt], &o[nt + 1], &o[nt + 2], &o[nt + 3]}, ah, al, q);
       }
     }
     float* mine = sm.part + warp * COLS * LB;
@@ -403,6 +509,7 @@ __global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p)
     cp_async_wait<1>();
     __syncthreads();                                        // partial sums stand, K^ and B are here
 
+    if (ch + 1 < n_chunks) load_uv(ch + 1);
     const float* KTs = sm.kb;
     const float* Bs = KTs + DKP * LB;
     const float* GLs = Bs + C * LB;
@@ -432,17 +539,20 @@ __global__ void __launch_bounds__(ST, 1) delta_chunk_scan_kernel(const Params p)
       split(a.y, ah[2], al[2]);
       split(b.y, ah[3], al[3]);
       const int at = 8 * js + 2 * tq;
+      // the state, and O += B_lower U for the warp's row blocks: warp and 7 - warp
+      float2 k[KS];
+      float(*d[KS])[4];
 #pragma unroll
       for (int nt = 0; nt < KS; ++nt) {
-        const float2 k = *reinterpret_cast<const float2*>(KTs + (c0 + 8 * nt + gq) * LB + at);
-        mma_split(S[nt], ah, al, k.x, k.y);
+        k[nt] = *reinterpret_cast<const float2*>(KTs + (c0 + 8 * nt + gq) * LB + at);
+        d[nt] = &S[nt];
       }
-      // O += B_lower U: the warp's row blocks are warp and 7 - warp
+      mma_split<KS>(d, ah, al, k);
 #pragma unroll
       for (int nt = 0; nt < C / 8; ++nt) {
         if ((nt == warp || nt == 7 - warp) && js <= nt) {
-          const float2 k = *reinterpret_cast<const float2*>(Bs + (8 * nt + gq) * LB + at);
-          mma_split(o[nt], ah, al, k.x, k.y);
+          const float2 x[1] = {*reinterpret_cast<const float2*>(Bs + (8 * nt + gq) * LB + at)};
+          mma_split<1>({&o[nt]}, ah, al, x);
         }
       }
     }
