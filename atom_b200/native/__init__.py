@@ -82,6 +82,9 @@ _SIGNATURES = {
     "atom_gla_gate_norm": [_vp, _i64, _vp, _vp, _i, _i64, _vp, _i, _i, _i, _i, _f, _vp, _i, _f, _vp],
     "atom_add_dynamic_tanh": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _vp],
     "atom_delta_supports": [_i, _i],
+    "atom_delta_step_supports": [_i, _i],
+    "atom_delta_step": [_vp, _i64, _vp, _i, _i64, _vp, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _i64, _vp, _i64, _vp, _i, _f, _f, _vp,
+                        _vp, _vp, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
     "atom_delta_chunk_supports": [_i, _i],
     "atom_delta_chunk_floats": [_i, _i],
     "atom_delta_chunks": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
@@ -1760,6 +1763,38 @@ def delta_prepare(u: torch.Tensor, rn: torch.Tensor, x: torch.Tensor, w: torch.T
                                     beta_in.stride(0), beta.data_ptr(), seq_of_token.data_ptr(), cu_q.data_ptr(),
                                     state_slots.data_ptr(), T, G, H, dk, dv, float(q_scale), float(unit_eps), _stream()),
            "delta_prepare")
+
+
+DELTA_STEP = True     # False: single rows run through delta_prepare, delta_scan and gla_gate_norm too (measurements, tests)
+
+
+def delta_step_supports(dk: int, dv: int) -> bool:
+    return DELTA_STEP and bool(lib().atom_delta_step_supports(dk, dv))
+
+
+def delta_step(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], z: torch.Tensor,
+               A_log: torch.Tensor, dt_bias: torch.Tensor, beta_in: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor,
+               norm_eps: float, y_scale: float, S: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, num_seqs: int,
+               G: int, H: int, dk: int, dv: int, q_scale: float, unit_eps: float, write_state: bool = True) -> None:
+    """One row per request: ``delta_prepare``, ``delta_scan`` and ``gla_gate_norm`` with a sigmoid gate in one kernel (arguments
+    as theirs).  With G = H the convolution's rows in ``state`` are brought up to date too; otherwise that is
+    ``conv_state_update``'s, afterwards."""
+    _cuda(y, x, w, state, z, A_log, dt_bias, beta_in, gate, norm, S, cu_q, state_slots)
+    T, C = x.shape
+    taps = w.shape[1]
+    assert C == 2 * G * dk + H * dv and x.stride(1) == 1 and tuple(w.shape) == (C, taps) and w.is_contiguous()
+    assert y.stride(1) == 1 and y.shape == gate.shape == (T, H * dv) and gate.stride(1) == 1 and y.dtype == gate.dtype == x.dtype
+    assert A_log.dtype == dt_bias.dtype and A_log.numel() == H and dt_bias.numel() == H * dk and norm.numel() == dv
+    assert z.dtype == torch.float32 and z.is_contiguous() and z.shape == (T, H * dk)
+    assert taps == 1 or (state.is_contiguous() and state.dtype == x.dtype and tuple(state.shape[1:]) == (taps - 1, C))
+    assert beta_in.dtype == x.dtype and beta_in.stride(1) == 1 and beta_in.shape == (T, H)
+    assert S.dtype == torch.float32 and S.is_contiguous() and tuple(S.shape[1:]) == (H, dk, dv)
+    _check(lib().atom_delta_step(y.data_ptr(), y.stride(0), x.data_ptr(), dtype_code(x.dtype), x.stride(0), w.data_ptr(),
+                                 dtype_code(w.dtype), taps, _ptr(state) if taps > 1 else None, z.data_ptr(), A_log.data_ptr(),
+                                 dt_bias.data_ptr(), dtype_code(A_log.dtype), beta_in.data_ptr(), beta_in.stride(0),
+                                 gate.data_ptr(), gate.stride(0), norm.data_ptr(), dtype_code(norm.dtype), float(norm_eps),
+                                 float(y_scale), S.data_ptr(), cu_q.data_ptr(), state_slots.data_ptr(), num_seqs, G, H, dk, dv,
+                                 float(q_scale), float(unit_eps), int(write_state), _stream()), "delta_step")
 
 
 def delta_scan(out: torch.Tensor, u: torch.Tensor, rn: torch.Tensor, la: torch.Tensor, beta: torch.Tensor,

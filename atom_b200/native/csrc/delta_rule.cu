@@ -14,6 +14,10 @@
 //                         LPC neighbouring lanes share a column's key channels and hold them in registers.  Four more warps
 //                         bring the next rows into shared memory (unit vectors and decays formed on the way) while
 //                         the four compute warps walk the present ones.
+//   delta_step_kernel     a step in which every request brings one row, everything from the projected rows to the gated
+//                         output in one kernel: a CTA per (request, head), four lanes to a column of the state.  With as
+//                         many q/k heads as heads it also brings the convolution's rows up to date (every channel is then
+//                         one CTA's).
 // Head h reads q and k head h / (H / G).
 #include "common.cuh"
 
@@ -22,6 +26,7 @@ namespace atom {
 constexpr float kDrLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float dr_silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float dr_silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }      // (before a rounding to bfloat16)
 __device__ __forceinline__ float dr_softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 struct DeltaPrep {
@@ -46,13 +51,30 @@ struct DeltaPrep {
   float q_scale, unit_eps;
 };
 
+__device__ __forceinline__ void delta_decays4(const DeltaPrep& p, float* z, int i, const __nv_bfloat16* bias) {
+  float4 v = *reinterpret_cast<const float4*>(z + i);
+  const uint2 q = *reinterpret_cast<const uint2*>(bias + i);
+  const float2 b0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+  const float2 b1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+  const float a = -expf(load_as_float(p.A_log, p.v_dtype, i / p.dk)) * kDrLog2e;
+  v.x = a * dr_softplus(v.x + b0.x);
+  v.y = a * dr_softplus(v.y + b0.y);
+  v.z = a * dr_softplus(v.z + b1.x);
+  v.w = a * dr_softplus(v.w + b1.y);
+  *reinterpret_cast<float4*>(z + i) = v;
+}
+
 template <typename T>
 __device__ __forceinline__ void delta_decays(const DeltaPrep& p, int t) {
   const int n = p.H * p.dk;
   float* z = p.z + (int64_t)t * n;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float a = expf(load_as_float(p.A_log, p.v_dtype, i / p.dk));
-    z[i] = -a * dr_softplus(z[i] + load_as_float(p.dt_bias, p.v_dtype, i)) * kDrLog2e;
+  if (p.dk % 4 == 0 && p.v_dtype == ATOM_BF16 && (((uintptr_t)p.z | (uintptr_t)p.dt_bias) % 16) == 0) {
+    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) delta_decays4(p, z, i, (const __nv_bfloat16*)p.dt_bias);
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+      const float a = expf(load_as_float(p.A_log, p.v_dtype, i / p.dk));
+      z[i] = -a * kDrLog2e * dr_softplus(z[i] + load_as_float(p.dt_bias, p.v_dtype, i));
+    }
   }
   for (int h = threadIdx.x; h < p.H; h += blockDim.x) {
     const float b = to_float(((const T*)p.beta_in)[(int64_t)t * p.ldb + h]);
@@ -132,7 +154,7 @@ __global__ void __launch_bounds__(256) delta_prepare_vec_kernel(const DeltaPrep 
     float ss = 0.f;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      h2[e] = __floats2bfloat162_rn(dr_silu(y[2 * e]), dr_silu(y[2 * e + 1]));
+      h2[e] = __floats2bfloat162_rn(dr_silu_fast(y[2 * e]), dr_silu_fast(y[2 * e + 1]));
       const float2 f = __bfloat1622float2(h2[e]);
       ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
     }
@@ -326,6 +348,146 @@ __global__ void __launch_bounds__(kDrCompute + kDrStagers) delta_scan_kernel(con
   }
 }
 
+// ------------------------------------------------------------------ one row per request
+
+struct DeltaStep {
+  DeltaPrep in;            // (u, rn and beta are not used; z holds the raw decay inputs; state is brought up to date)
+  float* S;                // [slots, H, dk, dv]
+  void* y;                 // [T, H dv] rows at stride ldy
+  int64_t ldy;
+  const void* gate;        // [T, H dv] rows at stride ldg
+  int64_t ldg;
+  const void* norm;        // [dv]
+  int norm_dtype;
+  float norm_eps, y_scale;
+  int write_state;
+};
+
+template <typename T, int KPT>
+__global__ void __launch_bounds__(512) delta_step_kernel(const DeltaStep d) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  constexpr int DKP = 4 * KPT;
+  __shared__ __align__(16) float q_s[DKP], k_s[DKP], a_s[DKP];
+  __shared__ float v_s[128], f_s[2], scratch[32];
+  const DeltaPrep& p = d.in;
+  const int s = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x;
+  const int t = p.cu_q[s];
+  if (p.cu_q[s + 1] - t <= 0) return;
+  const int dk = p.dk, dv = p.dv, G = p.G, H = p.H, g = hd / (H / G);
+  const int C = 2 * G * dk + H * dv, slot = p.state_slots[s];
+  const int col = tid >> 2, slice = tid & 3;
+  float* S_g = d.S + ((int64_t)slot * H + hd) * dk * dv;
+  float S[KPT];
+#pragma unroll
+  for (int m = 0; m < KPT; ++m) {
+    const int ch = dr_channel<4>(slice, m);
+    S[m] = (ch < dk && col < dv) ? S_g[(int64_t)ch * dv + col] : 0.f;
+  }
+  T* st = p.taps > 1 ? (T*)p.state + (int64_t)slot * (p.taps - 1) * C : nullptr;
+  const bool shift = st && d.write_state && H == G;
+  for (int e = tid; e < 2 * dk + dv; e += blockDim.x) {
+    const int c = e < dk ? g * dk + e : (e < 2 * dk ? (G + g) * dk + e - dk : 2 * G * dk + hd * dv + e - 2 * dk);
+    const T now = ((const T*)p.x)[(int64_t)t * p.ldx + c];
+    float y = 0.f;
+    for (int j = 0; j < p.taps - 1; ++j) {
+      const T old = st[(int64_t)j * C + c];
+      y = fmaf(load_as_float(p.w, p.w_dtype, (int64_t)c * p.taps + j), to_float(old), y);
+      if (shift && j > 0) st[(int64_t)(j - 1) * C + c] = old;
+    }
+    if (shift) st[(int64_t)(p.taps - 2) * C + c] = now;
+    y = fmaf(load_as_float(p.w, p.w_dtype, (int64_t)c * p.taps + p.taps - 1), to_float(now), y);
+    const float o = to_float(from_float<T>(dr_silu(y)));
+    if (e < dk) q_s[e] = o;
+    else if (e < 2 * dk) k_s[e - dk] = o;
+    else v_s[e - 2 * dk] = o;
+  }
+  for (int i = tid; i < DKP; i += blockDim.x) {
+    float a = 1.f;
+    if (i < dk) {
+      const int64_t at = (int64_t)hd * dk + i;
+      const float A = expf(load_as_float(p.A_log, p.v_dtype, hd));
+      a = dr_ex2(-A * kDrLog2e * dr_softplus(p.z[(int64_t)t * H * dk + at] + load_as_float(p.dt_bias, p.v_dtype, at)));
+    } else {
+      q_s[i] = k_s[i] = 0.f;
+    }
+    a_s[i] = a;
+  }
+  const float beta = 1.f / (1.f + expf(-to_float(((const T*)p.beta_in)[(int64_t)t * p.ldb + hd])));
+  __syncthreads();
+  const int warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+  for (int n = warp; n < 2; n += warps) {
+    const float* x = n ? k_s : q_s;
+    float ss = 0.f;
+    for (int i = lane; i < dk; i += 32) ss = fmaf(x[i], x[i], ss);
+    ss = warp_sum(ss);
+    if (lane == 0) f_s[n] = rsqrtf(ss + p.unit_eps) * (n ? 1.f : p.q_scale);
+  }
+  __syncthreads();
+  const float fq = f_s[0], fk = f_s[1];
+  float p0 = 0.f, p1 = 0.f, p2 = 0.f, p3 = 0.f;
+#pragma unroll
+  for (int m4 = 0; m4 < KPT / 4; ++m4) {
+    const float4 a4 = *reinterpret_cast<const float4*>(a_s + slice * 4 + m4 * 16);
+    const float4 k4 = *reinterpret_cast<const float4*>(k_s + slice * 4 + m4 * 16);
+    S[4 * m4] *= a4.x;
+    S[4 * m4 + 1] *= a4.y;
+    S[4 * m4 + 2] *= a4.z;
+    S[4 * m4 + 3] *= a4.w;
+    p0 = fmaf(S[4 * m4], k4.x, p0);
+    p1 = fmaf(S[4 * m4 + 1], k4.y, p1);
+    p2 = fmaf(S[4 * m4 + 2], k4.z, p2);
+    p3 = fmaf(S[4 * m4 + 3], k4.w, p3);
+  }
+  float pk = ((p0 + p1) + (p2 + p3)) * fk;
+  pk += __shfl_xor_sync(0xffffffffu, pk, 1);
+  pk += __shfl_xor_sync(0xffffffffu, pk, 2);
+  const float ku = col < dv ? beta * (v_s[col] - pk) * fk : 0.f;
+  p0 = p1 = p2 = p3 = 0.f;
+#pragma unroll
+  for (int m4 = 0; m4 < KPT / 4; ++m4) {
+    const float4 k4 = *reinterpret_cast<const float4*>(k_s + slice * 4 + m4 * 16);
+    const float4 q4 = *reinterpret_cast<const float4*>(q_s + slice * 4 + m4 * 16);
+    S[4 * m4] = fmaf(k4.x, ku, S[4 * m4]);
+    S[4 * m4 + 1] = fmaf(k4.y, ku, S[4 * m4 + 1]);
+    S[4 * m4 + 2] = fmaf(k4.z, ku, S[4 * m4 + 2]);
+    S[4 * m4 + 3] = fmaf(k4.w, ku, S[4 * m4 + 3]);
+    p0 = fmaf(S[4 * m4], q4.x, p0);
+    p1 = fmaf(S[4 * m4 + 1], q4.y, p1);
+    p2 = fmaf(S[4 * m4 + 2], q4.z, p2);
+    p3 = fmaf(S[4 * m4 + 3], q4.w, p3);
+  }
+  float o = ((p0 + p1) + (p2 + p3)) * fq;
+  o += __shfl_xor_sync(0xffffffffu, o, 1);
+  o += __shfl_xor_sync(0xffffffffu, o, 2);
+  if (d.write_state) {
+#pragma unroll
+    for (int m = 0; m < KPT; ++m) {
+      const int ch = dr_channel<4>(slice, m);
+      if (ch < dk && col < dv) S_g[(int64_t)ch * dv + col] = S[m];
+    }
+  }
+  const bool own = slice == 0 && col < dv;
+  const float ss = block_sum(own ? o * o : 0.f, scratch);
+  if (own) {
+    const float z = to_float(((const T*)d.gate)[(int64_t)t * d.ldg + (int64_t)hd * dv + col]);
+    ((T*)d.y)[(int64_t)t * d.ldy + (int64_t)hd * dv + col] =
+        from_float<T>(o * rsqrtf(ss / (float)dv + d.norm_eps) * d.y_scale * load_as_float(d.norm, d.norm_dtype, col) /
+                      (1.f + expf(-z)));
+  }
+}
+
+template <typename T>
+static int launch_delta_step(const DeltaStep& d, int num_seqs, cudaStream_t stream) {
+  const dim3 grid(num_seqs, d.in.H), block((d.in.dv + 7) / 8 * 32);
+  const int dk = d.in.dk;
+  if (dk <= 32) launch_pdl(delta_step_kernel<T, 8>, grid, block, 0, stream, d);
+  else if (dk <= 64) launch_pdl(delta_step_kernel<T, 16>, grid, block, 0, stream, d);
+  else if (dk <= 96) launch_pdl(delta_step_kernel<T, 24>, grid, block, 0, stream, d);
+  else launch_pdl(delta_step_kernel<T, 32>, grid, block, 0, stream, d);
+  return check_launch();
+}
+
 template <typename T, int KPT, int LPC>
 static int launch_delta_scan(const DeltaScan& p, cudaStream_t stream) {
   constexpr int DKP = LPC * KPT, COLS = kDrCompute / LPC;
@@ -361,6 +523,27 @@ static int dispatch_delta_scan(const DeltaScan& p, int lanes, cudaStream_t strea
 }  // namespace atom
 
 ATOM_EXPORT int atom_delta_supports(int dk, int dv) { return dk > 0 && dk <= 256 && dv > 0 ? 1 : 0; }
+
+ATOM_EXPORT int atom_delta_step_supports(int dk, int dv) { return dk > 0 && dk <= 128 && dv > 0 && dv <= 128 ? 1 : 0; }
+
+ATOM_EXPORT int atom_delta_step(void* y, int64_t ldy, const void* x, int dtype, int64_t ldx, const void* w, int w_dtype,
+                                int taps, void* state, const float* z, const void* A_log, const void* dt_bias, int v_dtype,
+                                const void* beta_in, int64_t ldb, const void* gate, int64_t ldg, const void* norm,
+                                int norm_dtype, float norm_eps, float y_scale, float* S, const int* cu_q,
+                                const int* state_slots, int num_seqs, int G, int H, int dk, int dv, float q_scale,
+                                float unit_eps, int write_state, cudaStream_t stream) {
+  if (num_seqs <= 0) return ATOM_OK;
+  if (!atom_delta_step_supports(dk, dv) || G <= 0 || H <= 0 || H % G || H > 65535 || taps < 1 || (taps > 1 && !state) ||
+      (w_dtype != ATOM_F32 && w_dtype != ATOM_BF16) || (v_dtype != ATOM_F32 && v_dtype != ATOM_BF16) ||
+      (norm_dtype != ATOM_F32 && norm_dtype != ATOM_BF16))
+    return ATOM_ERR_ARG;
+  const atom::DeltaPrep in{nullptr, nullptr, x,   ldx,     w,       w_dtype, taps,        state, const_cast<float*>(z), A_log,
+                           dt_bias, v_dtype, beta_in, ldb, nullptr, nullptr, cu_q, state_slots, G, H, dk, dv, q_scale, unit_eps};
+  const atom::DeltaStep d{in, S, y, ldy, gate, ldg, norm, norm_dtype, norm_eps, y_scale, write_state};
+  if (dtype == ATOM_F32) return atom::launch_delta_step<float>(d, num_seqs, stream);
+  if (dtype == ATOM_BF16) return atom::launch_delta_step<__nv_bfloat16>(d, num_seqs, stream);
+  return ATOM_ERR_ARG;
+}
 
 ATOM_EXPORT int atom_delta_prepare(void* u, float* rn, const void* x, int dtype, int64_t ldx, const void* w, int w_dtype,
                                    int taps, const void* state, float* z, const void* A_log, const void* dt_bias,

@@ -106,13 +106,15 @@ template <int DKP>
 struct PrepSmem {
   static constexpr int LG = DKP + 4, LK = DKP + 8, LT = C + 4;
   float g[C * LG];                       // sums of the decays' logarithms from the row's block of 16 rows on
-  float tot[4 * DKP], pre[4 * DKP], suf[4 * DKP];      // the blocks' sums; over the blocks before; over the blocks behind
+  float off[14 * DKP];                   // rows (I, J), J < I <= 4: the sum over blocks J .. I-1; then over the blocks before I
   float a[C * LB];                       // [j][i] = beta_i A_ij for i > j, zero for the other i of j's 16-row block
   float t[C * LT];                       // T
   __nv_bfloat16 k[C * LK], q[C * LK];
-  float rk[C], rq[C], beta[C];
+  float rk[C], rq[C], rb[C], beta[C];    // rb: rk * beta
   int strong[4];                         // a channel of the block decays beyond 2^-60
 };
+
+__device__ __forceinline__ constexpr int off_row(int I, int J) { return I * (I - 1) / 2 + J; }
 
 template <int DKP>
 __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params p) {
@@ -178,6 +180,7 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
     sm.rq[i] = i < n ? p.rn[t * 2 * G + g] : 0.f;
     sm.rk[i] = i < n ? p.rn[t * 2 * G + G + g] : 0.f;
     sm.beta[i] = i < n ? p.beta[t * H + hd] : 0.f;
+    sm.rb[i] = sm.rk[i] * sm.beta[i];
   }
   __syncthreads();
   for (int e = tid; e < 4 * DKP; e += PT) {
@@ -189,18 +192,27 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
     for (int i = 1; i < 16; ++i) v[i] += v[i - 1];
 #pragma unroll
     for (int i = 1; i < 16; ++i) sm.g[(b * 16 + i) * LG + c] = v[i];
-    sm.tot[e] = v[15];
     if (v[15] < -60.f) sm.strong[b] = 1;
   }
   __syncthreads();
-  for (int e = tid; e < 4 * DKP; e += PT) {
-    const int b = e / DKP, c = e - b * DKP;
-    float before = 0.f, behind = 0.f;
-    for (int q = 0; q < b; ++q) before += sm.tot[q * DKP + c];
-    for (int q = b + 1; q < 4; ++q) behind += sm.tot[q * DKP + c];
-    sm.pre[e] = before;
-    sm.suf[e] = behind;
+  for (int c = tid; c < DKP; c += PT) {
+    float tot[4], before = 0.f;
+#pragma unroll
+    for (int b = 0; b < 4; ++b) tot[b] = sm.g[(16 * b + 15) * LG + c];
+#pragma unroll
+    for (int b = 0; b < 4; ++b) {
+      sm.off[(10 + b) * DKP + c] = before;
+      before += tot[b];
+      float sum = 0.f;
+#pragma unroll
+      for (int I = b + 1; I <= 4; ++I) {
+        sum += tot[I - 1];
+        sm.off[off_row(I, b) * DKP + c] = sum;
+      }
+    }
   }
+  __syncthreads();
+  const float* pre = sm.off + 10 * DKP;                     // (row 10 is zero)
 
   // A and B: a warp takes up to three tiles of 8 columns of one row block (block 3: 8 tiles, 2: 6, 1: 4, 0: 2)
   const int gq = lane >> 2, tq = lane & 3;
@@ -216,33 +228,36 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
 #pragma unroll
       for (int e = 0; e < 4; ++e) da[x][e] = db[x][e] = 0.f;
     if (I < nb) {
+      const float *orow[3], *grow[3];
+      const __nv_bfloat16* krow[3];
+      float live[3];
+#pragma unroll
+      for (int x = 0; x < 3; ++x) {
+        const int jt = min(jt0 + x, 2 * I + 1), J = jt >> 1, jc = jt * 8 + gq;
+        orow[x] = J < I ? sm.off + off_row(I, J) * DKP + tq : pre + tq;
+        grow[x] = sm.g + jc * LG + tq;
+        krow[x] = sm.k + jc * LK + tq;
+        live[x] = J == I && strong ? 0.f : 1.f;             // (then formed pair by pair below)
+      }
+      const float *ga = sm.g + ia * LG + tq, *gb = sm.g + ib * LG + tq;
+      const __nv_bfloat16 *ka = sm.k + ia * LK + tq, *kb = sm.k + ib * LK + tq;
+      const __nv_bfloat16 *qa = sm.q + ia * LK + tq, *qb = sm.q + ib * LK + tq;
 #pragma unroll 2
       for (int kk = 0; kk < DKP; kk += 8) {
         uint32_t kh[4], kl[4], qh[4], ql[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = (e & 1) ? ib : ia, c = kk + tq + (e >> 1) * 4;
-          const float f = ex2(sm.g[i * LG + c]);
-          split(__bfloat162float(sm.k[i * LK + c]) * f, kh[e], kl[e]);
-          split(__bfloat162float(sm.q[i * LK + c]) * f, qh[e], ql[e]);
+        for (int h = 0; h < 2; ++h) {
+          const float fa = ex2(ga[kk + 4 * h]), fb = ex2(gb[kk + 4 * h]);
+          split(__bfloat162float(ka[kk + 4 * h]) * fa, kh[2 * h], kl[2 * h]);
+          split(__bfloat162float(kb[kk + 4 * h]) * fb, kh[2 * h + 1], kl[2 * h + 1]);
+          split(__bfloat162float(qa[kk + 4 * h]) * fa, qh[2 * h], ql[2 * h]);
+          split(__bfloat162float(qb[kk + 4 * h]) * fb, qh[2 * h + 1], ql[2 * h + 1]);
         }
         float2 bv[3];
 #pragma unroll
-        for (int x = 0; x < 3; ++x) {
-          const int jt = min(jt0 + x, 2 * I + 1), J = jt >> 1, jc = jt * 8 + gq;
-          float w[2];
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int c = kk + tq + e * 4;
-            float d = -sm.g[jc * LG + c];
-            if (J < I) d += sm.tot[J * DKP + c];
-            if (J == 0 && I >= 2) d += sm.tot[DKP + c];
-            if (J <= 1 && I == 3) d += sm.tot[2 * DKP + c];
-            if (J == I && strong) d = 0.f;                  // (formed pair by pair below)
-            w[e] = __bfloat162float(sm.k[jc * LK + c]) * ex2(d);
-          }
-          bv[x] = make_float2(w[0], w[1]);
-        }
+        for (int x = 0; x < 3; ++x)
+          bv[x] = make_float2(__bfloat162float(krow[x][kk]) * ex2((orow[x][kk] - grow[x][kk]) * live[x]),
+                              __bfloat162float(krow[x][kk + 4]) * ex2((orow[x][kk + 4] - grow[x][kk + 4]) * live[x]));
         mma_split<3>({&da[0], &da[1], &da[2]}, kh, kl, bv);
         mma_split<3>({&db[0], &db[1], &db[2]}, qh, ql, bv);
       }
@@ -305,7 +320,7 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
     for (int e = w; e < C * DKP / 4; e += NW) {
       const int i = e / (DKP / 4), c = (e - i * (DKP / 4)) * 4;
       const float4 gl = *reinterpret_cast<const float4*>(sm.g + i * LG + c);
-      const float4 pr = *reinterpret_cast<const float4*>(sm.pre + (i / 16) * DKP + c);
+      const float4 pr = *reinterpret_cast<const float4*>(pre + (i / 16) * DKP + c);
       const uint2 qv = *reinterpret_cast<const uint2*>(sm.q + i * LK + c);
       const float2 q0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qv.x));
       const float2 q1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&qv.y));
@@ -317,18 +332,36 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
 #pragma unroll 1
     for (int e = w; e < DKP * (C / 8); e += NW) {
       const int j8 = e / DKP, c = e - j8 * DKP;             // (eight rows of one block)
-      const float d = sm.tot[(j8 / 2) * DKP + c], suf = sm.suf[(j8 / 2) * DKP + c];
+      const float d = sm.off[off_row(4, j8 / 2) * DKP + c];
       float o[8];
 #pragma unroll
       for (int x = 0; x < 8; ++x) {
         const int j = j8 * 8 + x;
-        o[x] = __bfloat162float(sm.k[j * LK + c]) * sm.rk[j] * ex2(d - sm.g[j * LG + c] + suf);
+        o[x] = __bfloat162float(sm.k[j * LK + c]) * sm.rk[j] * ex2(d - sm.g[j * LG + c]);
       }
       float* dst = blob + BL::KT + c * LB + j8 * 8;
       *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
       *reinterpret_cast<float4*>(dst + 4) = make_float4(o[4], o[5], o[6], o[7]);
     }
-    for (int c = w; c < DKP; c += NW) blob[BL::GL + c] = ex2(sm.pre[3 * DKP + c] + sm.tot[3 * DKP + c]);
+    // the values into the place of the queries
+    asm volatile("bar.sync 1, %0;\n" ::"n"(PT - 64) : "memory");
+    const __nv_bfloat16* v = p.u + t0 * CU + 2 * (int64_t)G * dk + (int64_t)hd * dv;
+    const int dvs = min(dv, DKP);
+    if (dk % 4 == 0 && dv % 8 == 0 && ((uintptr_t)p.u % 16) == 0) {
+#pragma unroll 4
+      for (int e = w; e < C * DKP / 8; e += NW) {
+        const int i = e / (DKP / 8), c = (e - i * (DKP / 8)) * 8;
+        if (c < dvs)
+          *reinterpret_cast<uint4*>(sm.q + i * LK + c) =
+              i < n ? *reinterpret_cast<const uint4*>(v + (int64_t)i * CU + c) : make_uint4(0u, 0u, 0u, 0u);
+      }
+    } else {
+      for (int e = w; e < C * DKP; e += NW) {
+        const int i = e / DKP, c = e - i * DKP;
+        if (c < dvs) sm.q[i * LK + c] = i < n ? v[(int64_t)i * CU + c] : __float2bfloat16_rn(0.f);
+      }
+    }
+    for (int c = w; c < DKP; c += NW) blob[BL::GL + c] = ex2(sm.off[off_row(4, 0) * DKP + c]);
   }
   __syncthreads();
 
@@ -354,10 +387,11 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
         for (int e = 0; e < 2; ++e) {
           const int j = 8 * ks + tq + 4 * e;
           if (keys)
-            w[e] = __bfloat162float(sm.k[j * LK + col]) * sm.rk[j] * ex2(sm.pre[(j / 16) * DKP + col] + sm.g[j * LG + col]);
+            w[e] = __bfloat162float(sm.k[j * LK + col]) * sm.rb[j] * ex2(pre[(j / 16) * DKP + col] + sm.g[j * LG + col]);
+          else if (base < 2 * DKP)                           // (values beyond dv: whatever lies there, not stored)
+            w[e] = __bfloat162float(sm.q[j * LK + col - DKP]) * sm.beta[j];
           else
-            w[e] = j < n && col < DKP + dv ? __bfloat162float(v[(int64_t)j * CU + col]) : 0.f;
-          w[e] *= sm.beta[j];
+            w[e] = j < n && col < DKP + dv ? __bfloat162float(v[(int64_t)j * CU + col]) * sm.beta[j] : 0.f;
         }
         bv[x] = make_float2(w[0], w[1]);
       }

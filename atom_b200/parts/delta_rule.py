@@ -74,6 +74,14 @@ class ChannelDeltaRule(ProjectedMixer):
         rows, conv = proj["qkv"], cache.states.get("conv")
         la = linear(proj["a"], self.w_a2_weight, None, ws.get("dr.la", (T, H * dk), f32))
         gate = linear(proj["g"], self.w_g2_weight, None, ws.get("dr.gate", (T, H * dv), dt))
+        if step.max_q_len == 1 and T == step.num_seqs and not step.plan_for_any_batch and native.delta_step_supports(dk, dv):
+            # (every request brings one row: the rest is one kernel)
+            native.delta_step(y, rows, self.w_conv_weight, conv, la, self.w_A_log, self.w_dt_bias, proj["b"], gate, self.w_norm,
+                              self.norm_eps, y_scale, cache.states["S"], step.cu_q, step.state_slots, step.num_seqs, G, H, dk,
+                              dv, dk ** -0.5, UNIT_EPS, writes_cache)
+            if conv is not None and writes_cache and G != H:
+                native.conv_state_update(conv, rows, step.cu_q, step.state_slots, step.num_seqs)
+            return
         u = ws.get("dr.u", (T, self.channels), dt)
         rn = ws.get("dr.rn", (T, 2 * G), f32)
         beta = ws.get("dr.beta", (T, H), f32)

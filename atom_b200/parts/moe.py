@@ -61,7 +61,8 @@ class RoutedExperts(FeedForward):
         H, E, F = self.hidden_size, self.E, self.ff
         outputs = E + self.identity
         rows = (outputs, 1) if self.shared_gate else (outputs,)
-        p = {"router.weight": ParamSpec((sum(rows), H), rows=rows),
+        pad = -sum(rows) % 8                     # (the product's width in steps of 8)
+        p = {"router.weight": ParamSpec((sum(rows) + pad, H), rows=rows, pad=pad),
              "gate_up.weight": ParamSpec((E * 2 * F, H), rows=(F,) * (2 * E)),
              "down.weight": ParamSpec((E * H, F), rows=(H,) * E)}
         if self.correction:
@@ -111,6 +112,6 @@ class RoutedExperts(FeedForward):
             shared = linear(f, self.w_shared_down_weight, None, ws.get("moe.shared.out", (T, H), dt))
         out = ws.get("moe.out", (T, H), dt)
         native.moe_combine(out, y, pair_pos, top, None if on_input else wts, shared,
-                           logits[:, n_logits - 1:] if self.shared_gate else None, step.seq_of_token,
+                           logits[:, E + self.identity:E + self.identity + 1] if self.shared_gate else None, step.seq_of_token,
                            x if self.identity else None, ids if self.identity else None, E)
         return out

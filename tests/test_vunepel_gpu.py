@@ -97,6 +97,8 @@ DELTA_CASES = [  # heads, kv_heads, dim, vdim, taps, ranks, lens
     (4, 4, 64, 64, 4, (16, 24), (200, 129, 16)),
     (3, 1, 128, 128, 4, (16, 24), (193, 64, 63)),
     (1, 1, 1, 1, 2, (1, 1), (40, 3, 9)),
+    (2, 1, 32, 144, 4, (8, 8), (200, 100, 5)),
+    (2, 2, 60, 100, 3, (8, 8), (130, 3, 70)),
 ]
 EPS = 2e-5
 
@@ -134,13 +136,14 @@ def _delta_part(case, dtype, width=72):
 @pytest.mark.parametrize("case", DELTA_CASES)
 def test_delta_rule_part_under_every_cut(case, dtype, monkeypatch):
     """The state and the convolution's rows go from step to step in the request's slot, whatever the cut (also steps with
-    fewer rows than taps).  (bfloat16 runs long portions in chunks on the tensor cores where the sizes allow;
-    "bfloat16-rows" row by row there too.)"""
+    fewer rows than taps).  (bfloat16 runs long portions in chunks on the tensor cores and single rows in one kernel where
+    the sizes allow; "bfloat16-rows" row by row in separate kernels there too.)"""
     from atom_b200 import native
     if dtype.endswith("-rows"):
         if not native.delta_chunk_supports(case[2], case[3], torch.bfloat16):
             pytest.skip("these sizes run row by row anyway")
         monkeypatch.setattr(native, "DELTA_TC", False)
+        monkeypatch.setattr(native, "DELTA_STEP", False)
         dtype = "bfloat16"
     part, m, P, W = _delta_part(case, dtype)
     lens = dict(zip("abc", case[6]))
