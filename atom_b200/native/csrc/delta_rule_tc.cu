@@ -12,7 +12,7 @@
 //       inverse counterpart 2^-(sum up to the column) within the block, where that stays below 2^60; a block whose decays
 //       reach further forms 2^(G_i - G_j) for every pair instead.  Sums run within a block of 16 rows and over whole blocks,
 //       so that no difference is one of two large sums (a decay's logarithm counts as -32 at least: 2^-32 of a state is below
-//       its last bit).  T = (I + diag(beta) A_strictly_lower)^-1 is formed column by column in 32-bit, [W | U_v] is T times
+//       its last bit).  T = (I + diag(beta) A_strictly_lower)^-1 is formed in 32-bit, block by block, [W | U_v] is T times
 //       diag(beta) [K~ | V].
 //   delta_chunk_scan_kernel     a CTA per (request, head, 16 value columns) walks the chunks in order.  The transposed state
 //       (16 columns x key channels) lies in the accumulators of four warps, a quarter of the channels each, and is the left
@@ -295,23 +295,63 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
   __syncthreads();
 
   if (warp < 2) {
-    // T, a thread per column: once x_j stands, every later row loses beta_i A_ij x_j
-    float x[C];
+    // T: the blocks on the diagonal, a thread per column (once x_j stands, every later row loses beta_i A_ij x_j), then
+    // block diagonal by block diagonal  T_IJ = -T_II sum_K L_IK T_KJ  (the sum waits in T's unused block (J, I))
+    constexpr int LT = PrepSmem<DKP>::LT;
+    {
+      const int b = tid >> 4, c = tid & 15;
+      float x[16];
 #pragma unroll
-    for (int i = 0; i < C; ++i) x[i] = i == tid ? 1.f : 0.f;
+      for (int i = 0; i < 16; ++i) x[i] = i == c ? 1.f : 0.f;
 #pragma unroll
-    for (int j = 0; j < C - 1; ++j) {
+      for (int j = 0; j < 15; ++j) {
 #pragma unroll
-      for (int i4 = (j + 1) / 4; i4 < C / 4; ++i4) {
-        const float4 l = *reinterpret_cast<const float4*>(sm.a + j * LB + i4 * 4);      // (zero where i <= j)
-        x[4 * i4] = fmaf(-l.x, x[j], x[4 * i4]);
-        x[4 * i4 + 1] = fmaf(-l.y, x[j], x[4 * i4 + 1]);
-        x[4 * i4 + 2] = fmaf(-l.z, x[j], x[4 * i4 + 2]);
-        x[4 * i4 + 3] = fmaf(-l.w, x[j], x[4 * i4 + 3]);
+        for (int i4 = (j + 1) / 4; i4 < 4; ++i4) {
+          const float4 l = *reinterpret_cast<const float4*>(sm.a + (16 * b + j) * LB + 16 * b + i4 * 4);   // (zero where i <= j)
+          x[4 * i4] = fmaf(-l.x, x[j], x[4 * i4]);
+          x[4 * i4 + 1] = fmaf(-l.y, x[j], x[4 * i4 + 1]);
+          x[4 * i4 + 2] = fmaf(-l.z, x[j], x[4 * i4 + 2]);
+          x[4 * i4 + 3] = fmaf(-l.w, x[j], x[4 * i4 + 3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) sm.t[(16 * b + i) * LT + 16 * b + c] = x[i];
+    }
+    const int c = tid & 15, r = (tid >> 4) * 4;              // a column, four rows of a block
+#pragma unroll 1
+    for (int d = 1; d < 4; ++d) {
+      asm volatile("bar.sync 2, 64;\n" ::: "memory");
+#pragma unroll 1
+      for (int J = 0; J + d < 4; ++J) {
+        const int I = J + d;
+        float m[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+        for (int j = 16 * J; j < 16 * I; ++j) {
+          const float4 l = *reinterpret_cast<const float4*>(sm.a + j * LB + 16 * I + r);
+          const float y = sm.t[j * LT + 16 * J + c];
+          m[0] = fmaf(l.x, y, m[0]);
+          m[1] = fmaf(l.y, y, m[1]);
+          m[2] = fmaf(l.z, y, m[2]);
+          m[3] = fmaf(l.w, y, m[3]);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) sm.t[(16 * J + r + q) * LT + 16 * I + c] = m[q];
+      }
+      asm volatile("bar.sync 2, 64;\n" ::: "memory");
+#pragma unroll 1
+      for (int J = 0; J + d < 4; ++J) {
+        const int I = J + d;
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+        for (int k = 0; k < 16; ++k) {
+          const float y = sm.t[(16 * J + k) * LT + 16 * I + c];
+#pragma unroll
+          for (int q = 0; q < 4; ++q) o[q] = fmaf(-sm.t[(16 * I + r + q) * LT + 16 * I + k], y, o[q]);
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) sm.t[(16 * I + r + q) * LT + 16 * J + c] = o[q];
       }
     }
-#pragma unroll
-    for (int i = 0; i < C; ++i) sm.t[i * PrepSmem<DKP>::LT + tid] = x[i];
   } else {
     // meanwhile: Q~, K^ transposed, the whole chunk's decays
     const int w = tid - 64;
@@ -376,7 +416,7 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[I][x][e] = 0.f;
     const __nv_bfloat16* v = p.u + t0 * CU + 2 * (int64_t)G * dk + (int64_t)hd * dv - DKP;
-#pragma unroll
+#pragma unroll 1
     for (int ks = 0; ks < C / 8; ++ks) {
       float2 bv[4];
 #pragma unroll
@@ -396,7 +436,8 @@ __global__ void __launch_bounds__(PT, 2) delta_chunk_prepare_kernel(const Params
         bv[x] = make_float2(w[0], w[1]);
       }
 #pragma unroll
-      for (int I = ks / 2; I < 4; ++I) {
+      for (int I = 0; I < 4; ++I) {
+        if (I < ks / 2) continue;                            // (zero above the diagonal's blocks)
         uint32_t th[4], tl[4];
 #pragma unroll
         for (int e = 0; e < 4; ++e)
