@@ -229,7 +229,8 @@ PREBUILT_MIXED_HEADS = (
     {"ATOM_MH_NH": 4, "ATOM_MH_NKV": 2, "ATOM_MH_DK": 16, "ATOM_MH_DV": 32},
 )
 # Sizes of the windowed attention on the tensor cores that the build check compiles ahead of use.
-PREBUILT_WINDOW_HEADS = ({"ATOM_WA_DK": 128, "ATOM_WA_DV": 128}, {"ATOM_WA_DK": 64, "ATOM_WA_DV": 64})
+PREBUILT_WINDOW_HEADS = ({"ATOM_WA_DK": 128, "ATOM_WA_DV": 128}, {"ATOM_WA_DK": 64, "ATOM_WA_DV": 64},
+                         {"ATOM_WA_DK": 64, "ATOM_WA_DV": 128, "ATOM_WA_MAPS": 2})
 
 
 # Sizes of the attention over a window and pooled blocks on the tensor cores that the build check compiles ahead of use.

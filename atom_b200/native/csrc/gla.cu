@@ -225,6 +225,40 @@ __global__ void gla_gate_norm_kernel(T* __restrict__ y, int64_t ldy, const float
   }
 }
 
+// The same in bfloat16 for dv up to 128 in steps of 4: a lane four columns, all of a head's numbers read once.
+template <bool SIGMOID>
+__global__ void __launch_bounds__(256)
+gla_gate_norm_vec_kernel(__nv_bfloat16* __restrict__ y, int64_t ldy, const float* __restrict__ o,
+                         const __nv_bfloat16* __restrict__ g, int64_t ldg, const __nv_bfloat16* __restrict__ w, int H, int dv,
+                         float eps, const int* __restrict__ seq_of_token, float out_scale) {
+  atom::pdl_trigger();
+  atom::pdl_wait();
+  const int t = blockIdx.x;
+  if (seq_of_token[t] < 0) return;
+  const int warp = threadIdx.x >> 5, i = (threadIdx.x & 31) * 4, nwarps = blockDim.x >> 5;
+  const bool in = i < dv;
+  auto load4 = [&](const __nv_bfloat16* p) {
+    const uint2 q = in ? *reinterpret_cast<const uint2*>(p) : make_uint2(0u, 0u);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  };
+  const float4 w4 = load4(w + i);
+  for (int h = warp; h < H; h += nwarps) {
+    const float4 v = in ? *reinterpret_cast<const float4*>(o + ((int64_t)t * H + h) * dv + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 z = load4(g + (int64_t)t * ldg + (int64_t)h * dv + i);
+    const float ss = warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
+    const float f = rsqrtf(ss / (float)dv + eps) * out_scale;
+    auto act = [](float gg) { return (SIGMOID ? 1.f : gg) / (1.f + expf(-gg)); };
+    if (in) {
+      uint2 packed;
+      *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x * f * w4.x * act(z.x), v.y * f * w4.y * act(z.y));
+      *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z * f * w4.z * act(z.z), v.w * f * w4.w * act(z.w));
+      *reinterpret_cast<uint2*>(y + (int64_t)t * ldy + (int64_t)h * dv + i) = packed;
+    }
+  }
+}
+
 template <typename T, int KPT>
 static int launch_gla(float* out, const T* q, const T* k, const T* v, int64_t ld, float* z, int64_t ldz,
                       const void* zb, int zb_dtype, float inv_tau, float q_scale, float* state, float* sB, float* sA,
@@ -311,6 +345,17 @@ ATOM_EXPORT int atom_gla_gate_norm(void* y, int64_t ldy, const float* o, const v
   if (H <= 0 || dv <= 0 || (w_dtype != ATOM_F32 && w_dtype != ATOM_BF16) || (dtype != ATOM_F32 && dtype != ATOM_BF16))
     return ATOM_ERR_ARG;
   const int threads = H >= 8 ? 256 : 32 * H;
+  const uintptr_t all = (uintptr_t)y | (uintptr_t)o | (uintptr_t)g | (uintptr_t)w;
+  if (dtype == ATOM_BF16 && w_dtype == ATOM_BF16 && dv <= 128 && dv % 4 == 0 && ldy % 4 == 0 && ldg % 4 == 0 &&
+      ((uintptr_t)o % 16) == 0 && all % 8 == 0) {
+#define ATOM_GN(SIG)                                                                                                 \
+  atom::launch_pdl(atom::gla_gate_norm_vec_kernel<SIG>, dim3(T), dim3(threads), 0, stream, (__nv_bfloat16*)y, ldy, o, \
+                   (const __nv_bfloat16*)g, ldg, (const __nv_bfloat16*)w, H, dv, eps, seq_of_token, out_scale)
+    if (sigmoid) ATOM_GN(true);
+    else ATOM_GN(false);
+#undef ATOM_GN
+    return atom::check_launch();
+  }
 #define ATOM_GN(TT, SIG)                                                                                               \
   atom::launch_pdl(atom::gla_gate_norm_kernel<TT, SIG>, dim3(T), dim3(threads), 0, stream, (TT*)y, ldy, o, (const TT*)g, \
                    ldg, w, w_dtype, H, dv, eps, seq_of_token, out_scale)

@@ -306,10 +306,11 @@ def test_what_enters_the_recurrence(taps, dtype):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("gate", ["silu", "sigmoid"])
-def test_output_norm_per_head_with_its_gate(gate, dtype):
+@pytest.mark.parametrize("H,dv", [(5, 24), (9, 128), (3, 50), (2, 136), (8, 100)])
+def test_output_norm_per_head_with_its_gate(H, dv, gate, dtype):
     from atom_b200 import native
 
-    T, H, dv = 7, 5, 24
+    T = 7
     dt = _dt(dtype)
     g = torch.Generator().manual_seed(3)
     o = torch.randn(T, H * dv, generator=g)
