@@ -164,7 +164,7 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
                            int* __restrict__ status, const RopeExtras x) {
   atom::pdl_trigger();
   atom::pdl_wait();
-  extern __shared__ __align__(16) float cv_y[];      // [C], cos and sin of the rotated pairs
+  extern __shared__ __align__(16) float cv_y[];      // [C], cos and sin of the rotated pairs, [(H + G) dk / 8] sums of squares
   const int t = blockIdx.x;
   const int s = seq_of_token[t];
   if (s < 0) return;
@@ -185,6 +185,7 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
   const int half = rot_dims / 2;
   float* ang_c = cv_y + C;
   float* ang_s = ang_c + half;
+  float* squares = ang_s + half;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {      // (all heads of the token share the angles)
     float sn, cs;
     sincosf((float)p * freq[i], &sn, &cs);
@@ -241,31 +242,34 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
     }
     *reinterpret_cast<float4*>(cv_y + c) = make_float4(y[0], y[1], y[2], y[3]);
     *reinterpret_cast<float4*>(cv_y + c + 4) = make_float4(y[4], y[5], y[6], y[7]);
+    if (x.wq && c < (H + G) * dk) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+      squares[g] = ss;
+    }
   }
   __syncthreads();
   const int qk_end = (H + G) * dk;
-  if (x.wq) {
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int n = warp; n < H + G; n += blockDim.x >> 5) {
-      float ss = 0.f;
-      for (int i = lane; i < dk; i += 32) ss = fmaf(cv_y[n * dk + i], cv_y[n * dk + i], ss);
-      ss = warp_sum(ss);
-      const float f = rsqrtf(ss / (float)dk + x.norm_eps);
-      for (int i = lane; i < dk; i += 32) cv_y[n * dk + i] *= f * load_as_float(n < H ? x.wq : x.wk, x.norm_dtype, i);
-    }
-    __syncthreads();
-  }
   for (int g = threadIdx.x; g < groups; g += blockDim.x) {
     const int c = g * 8;
     __nv_bfloat16* dst;
     int i0 = 0;
     bool rotated = false;
     int64_t keep_at = -1;
-    float o[8];
+    float o[8], own[8];
+    float nf = 1.f;                                      // with a norm: the head's factor, and its weights
+    const void* wn = nullptr;
     if (c < qk_end) {
       const int n = c / dk;
       i0 = c - n * dk;
       rotated = i0 < rot_dims;
+      if (x.wq) {
+        wn = n < H ? x.wq : x.wk;
+        float ss = 0.f;
+        for (int q = 0; q < dk / 8; ++q) ss += squares[n * (dk / 8) + q];
+        nf = rsqrtf(ss / (float)dk + x.norm_eps);
+      }
       if (n < H) {
         dst = q_out + ((int64_t)t * H + n) * dk + i0;
       } else {
@@ -279,28 +283,44 @@ conv_rope_write_vec_kernel(__nv_bfloat16* __restrict__ q_out, const __nv_bfloat1
       keep_at = (int64_t)t * x.GV * dv + idx;
       dst = writes ? v_pages + (((int64_t)page * x.GV + gg) * page_size + slot) * dv + (idx - gg * dv) : nullptr;
     }
+    // eight numbers of the token's row (of the head's, from number i on), normed where there is a norm
+    auto load8 = [&](float (&v)[8], int at, int i) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = cv_y[at + e];
+      if (!wn) return;
+      if (x.norm_dtype == ATOM_BF16) {
+        const uint4 raw = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)wn + i);
+        const __nv_bfloat16* wv = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= nf * __bfloat162float(wv[e]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= nf * ((const float*)wn)[i + e];
+      }
+    };
+    load8(own, c, i0);
     if (rotated && x.neighbours) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const float a = cv_y[c + 2 * e], b = cv_y[c + 2 * e + 1];
+        const float a = own[2 * e], b = own[2 * e + 1];
         const float cs = ang_c[(i0 >> 1) + e], sn = ang_s[(i0 >> 1) + e];
         o[2 * e] = a * cs - b * sn;
         o[2 * e + 1] = b * cs + a * sn;
       }
     } else if (rotated) {
       const bool low = i0 < half;                      // the first of the pair: (a, b) = (own, + half); else (- half, own)
-      const float* av = cv_y + (low ? c : c - half);
-      const float* bv = cv_y + (low ? c + half : c);
+      float other[8];
+      load8(other, low ? c + half : c - half, low ? i0 + half : i0 - half);
       const int f0 = low ? i0 : i0 - half;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const float cs = ang_c[f0 + e], sn = ang_s[f0 + e];
-        const float a = av[e], b = bv[e];
+        const float a = low ? own[e] : other[e], b = low ? other[e] : own[e];
         o[e] = low ? a * cs - b * sn : b * cs + a * sn;
       }
     } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[e] = cv_y[c + e];
+      for (int e = 0; e < 8; ++e) o[e] = own[e];
       if (keep_at >= 0 && x.v_first) {
         const uint4 raw = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)x.v_first + keep_at);
         const __nv_bfloat16* fv = reinterpret_cast<const __nv_bfloat16*>(&raw);
@@ -534,14 +554,14 @@ ATOM_EXPORT int atom_conv_rope_write(void* q_out, const void* qkv, int dtype, in
                      rot_dims, positions, seq_of_token, cu_q, state_slots, block_table, max_pages, page_size,
                      (float*)k_pages, (float*)v_pages, num_pages, status, x);
   else if (dtype == ATOM_BF16 && dk % 8 == 0 && dv % 8 == 0 && rot_dims % (neighbours ? 8 : 16) == 0 && ld % 8 == 0 && taps <= 8 &&
-           (taps == 0 || w_dtype == ATOM_BF16) && ((H + G) * dk + GV * dv + rot_dims) * sizeof(float) <= 48 * 1024 &&
+           (taps == 0 || w_dtype == ATOM_BF16) && ((H + G) * dk + GV * dv + rot_dims + (H + G) * dk / 8) * sizeof(float) <= 48 * 1024 &&
            ((uintptr_t)qkv % 16) == 0 && ((uintptr_t)conv_w % 16) == 0 && ((uintptr_t)conv_state % 16) == 0 &&
            ((uintptr_t)bias % 16) == 0 && ((uintptr_t)v_first % 16) == 0 && ((uintptr_t)v_keep % 16) == 0 &&
-           ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0) {
+           ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)wq % 16) == 0 && ((uintptr_t)wk % 16) == 0 && ((uintptr_t)k_pages % 16) == 0 && ((uintptr_t)v_pages % 16) == 0) {
     const int C = (H + G) * dk + GV * dv;
     const int threads = C / 8 >= 256 ? 256 : ((C / 8 + 31) / 32) * 32;
 #define ATOM_CV(TAPS)                                                                                               \
-  atom::launch_pdl(atom::conv_rope_write_vec_kernel<TAPS>, dim3(T), dim3(threads), (C + rot_dims) * sizeof(float), stream, \
+  atom::launch_pdl(atom::conv_rope_write_vec_kernel<TAPS>, dim3(T), dim3(threads), (C + rot_dims + (H + G) * dk / 8) * sizeof(float), stream, \
                    (__nv_bfloat16*)q_out, (const __nv_bfloat16*)qkv, ld, H, G, dk, dv, (const __nv_bfloat16*)conv_w, \
                    (const __nv_bfloat16*)conv_state, freq, rot_dims, positions, seq_of_token, cu_q, state_slots,    \
                    block_table, max_pages, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages,  \

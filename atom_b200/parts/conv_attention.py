@@ -52,10 +52,13 @@ def window_plan(step, nh: int, nkv: int, dk: int, dv: int, window: Optional[int]
                 units = step.num_tokens * nh
             else:
                 units = (-(-step.num_tokens // native.WINDOW_TC_ROWS) + step.num_seqs - 1) * nh
-            # (two CTAs of one map fit an SM; steps with prompt portions fill it once before their keys are shared out: the
-            # shares cost a pass over 32-bit partial outputs of every row)
-            plan = (native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 and maps == 1 else 1,
-                                                  min_share=128), heads_rows)
+            # (two CTAs of one map fit an SM, one of two maps; steps with prompt portions fill it once before their keys
+            # are shared out: the shares cost a pass over 32-bit partial outputs of every row)
+            if step.max_q_len <= 1 and maps > 1:      # (one CTA to an SM: no second round)
+                nsplit = max(1, min(native.SM_COUNT // max(units, 1), -(-longest // 128), 64))
+            else:
+                nsplit = native.attention_mixed_splits(units, longest, per_sm=2 if step.max_q_len <= 1 else 1, min_share=128)
+            plan = (nsplit, heads_rows)
         else:
             plan = (0, False)
         step.plans[key] = plan
